@@ -7,6 +7,7 @@ from .gigopel import GigopelConfig
 from .sokirax import SokiraxConfig
 from .felolorn import FelolornConfig
 from .dinuzen import DinuzenConfig
+from .kulesun import KulesunConfig
 
 __all__ = ["ConfigError", "config_from_dict", "load_config", "register_architecture", "registered_architectures",
-           "BlockSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule", "Qwen3Config", "GigopelConfig", "SokiraxConfig", "FelolornConfig", "DinuzenConfig"]
+           "BlockSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule", "Qwen3Config", "GigopelConfig", "SokiraxConfig", "FelolornConfig", "DinuzenConfig", "KulesunConfig"]

@@ -60,6 +60,7 @@ MODULES: Dict[str, str] = {
     "recurrence": "recurrence.cu",
     "diag_recurrence": "diag_recurrence.cu",
     "diff_attention": "diff_attention.cu",
+    "mixed_head_attention": "mixed_head_attention.cu",
     "sampling": "sampling.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",
     "attention_fast": "attention_fast.cu",

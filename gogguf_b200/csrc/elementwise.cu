@@ -1039,17 +1039,21 @@ GG_API gg_rmsnorm_rows(const void* x, long long ldx, int dtype, const float* w, 
 
 // ----------------------------------------------------------------------------- soft cap
 // z <- cap * tanh(z / cap), in place, float32 (logits that are bounded smoothly).
-__global__ void softcap_kernel(float* z, float cap, long long n) {
+__global__ void softcap_kernel(float* z, float cap, float scale, long long n) {
     pdl_launch();
     pdl_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) z[i] = cap * tanhf(z[i] / cap);
+    if (i < n) {
+        const float v = z[i] * scale;
+        z[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
+    }
 }
 
-GG_API gg_softcap(float* z, float cap, long long n, cudaStream_t stream) {
+// z <- cap tanh(scale z / cap); cap 0: z <- scale z
+GG_API gg_softcap(float* z, float cap, float scale, long long n, cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (!(cap > 0.f)) return GG_ERR_ARG;
-    return gg_launch(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, z, cap, n);
+    if (!(cap >= 0.f)) return GG_ERR_ARG;
+    return gg_launch(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, z, cap, scale, n);
 }
 
 // ----------------------------------------------------------------------------- RMS norm in groups

@@ -10,16 +10,20 @@ from .build import KernelError, kernel, module
 
 
 def headwise_gemm_mma(x: torch.Tensor, ldx: int, hx: int, w: torch.Tensor, out: torch.Tensor, ldo: int, ho: int,
-                      m: int, alpha: float = 1.0) -> None:
+                      m: int, alpha: float = 1.0, gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h, :] = alpha * w[h] @ x[t, h, :] on the tensor cores; bfloat16 x and w [H, N, K], K, ldx and hx
-    multiples of 8, out bfloat16 or float32."""
+    multiples of 8, out bfloat16 or float32.  gate (rows of H * N logits in the output's dtype): the result is
+    multiplied by their sigmoid."""
     H, N, K = w.shape
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not w.is_contiguous():
         raise KernelError("headwise_gemm_mma takes bfloat16 operands, the weights contiguous [H, N, K]")
+    if gate is not None and (gate.dtype != out.dtype or gate.stride(-1) != 1 or gate.shape[-1] != H * N):
+        raise KernelError("headwise_gemm_mma: the gate has rows of H * N logits in the output's dtype")
     from .kernels import dtype_code
     kernel("latent_attention", "gg_headwise_gemm_mma")(
         x.data_ptr(), int(ldx), int(hx), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype), int(ldo), int(ho),
-        int(m), N, K, H, float(alpha), torch.cuda.current_stream().cuda_stream)
+        int(m), N, K, H, float(alpha), gate.data_ptr() if gate is not None else 0,
+        gate.stride(0) if gate is not None else 0, torch.cuda.current_stream().cuda_stream)
 
 
 def latent_attention_mma(qcat: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, cu_seqlens: torch.Tensor,
@@ -54,11 +58,14 @@ def mma_splits(n_seqs: int, n_tokens: int, heads: int, R: int, r: int, window: i
 def latent_prompt_mma(qd: torch.Tensor, qcat: torch.Tensor, kv: torch.Tensor, ckr: torch.Tensor, av: torch.Tensor,
                       cu_seqlens: torch.Tensor, seq_of_token: torch.Tensor, n_seqs: int, n_tokens: int, heads: int,
                       d: int, r: int, dv: int, R: int, scale: float, window: int, out_scale: float = 1.0,
-                      sink: Optional[torch.Tensor] = None) -> None:
+                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """Attention of a step whose sequences all start at position 0, in the expanded form: qd [T, >= heads (d + r)]
     (plain query parts), qcat [T, heads, R + r] (rotated parts at [..., R:]), kv [T, heads d + heads dv] (per-head
     plain keys, then values), ckr [T, R + r] (the shared rotated key part at [:, R:]); av [T, heads, dv] receives
-    out_scale times the heads' outputs.  All bfloat16."""
+    out_scale times the heads' outputs.  All bfloat16.  gate (rows of heads * dv logits): the outputs are multiplied by
+    their sigmoid."""
+    if gate is not None and (gate.dtype != torch.bfloat16 or gate.stride(-1) != 1 or gate.shape[-1] != heads * dv):
+        raise KernelError("latent_prompt_mma: the gate has bfloat16 rows of heads * dv logits")
     for t in (qd, qcat, kv, ckr, av):
         if t.dtype != torch.bfloat16 or t.stride(-1) != 1:
             raise KernelError("latent_prompt_mma takes bfloat16 rows")
@@ -66,6 +73,7 @@ def latent_prompt_mma(qd: torch.Tensor, qcat: torch.Tensor, kv: torch.Tensor, ck
         qd.data_ptr(), qd.stride(0), qcat.data_ptr(), kv.data_ptr(), kv.stride(0), ckr.data_ptr(), ckr.stride(0),
         av.data_ptr(), cu_seqlens.data_ptr(), seq_of_token.data_ptr(), int(n_seqs), int(n_tokens), heads, d, r, dv, R,
         float(scale), int(window), float(out_scale), sink.data_ptr() if sink is not None else 0,
+        gate.data_ptr() if gate is not None else 0, gate.stride(0) if gate is not None else 0,
         torch.cuda.current_stream().cuda_stream)
 
 
@@ -99,10 +107,11 @@ class _Fast:
                              ctx.n_seqs, T, H, R, self.r, self.scale, self.window, splits, part_o, part_ml,
                              max_new=max(int(ctx.max_new), 1), sink=self.sink)
 
-    def expand(self, olat: torch.Tensor, uv: torch.Tensor, av: torch.Tensor, m: int, alpha: float) -> None:
-        """av[t, h, :] = alpha * Wuv_h olat[t, h]."""
+    def expand(self, olat: torch.Tensor, uv: torch.Tensor, av: torch.Tensor, m: int, alpha: float,
+               gate: Optional[torch.Tensor] = None) -> None:
+        """av[t, h, :] = alpha * Wuv_h olat[t, h] (times the gate's sigmoid)."""
         dv = uv.shape[1]
-        headwise_gemm_mma(olat, self.H * self.R, self.R, uv, av, self.H * dv, dv, m, alpha)
+        headwise_gemm_mma(olat, self.H * self.R, self.R, uv, av, self.H * dv, dv, m, alpha, gate)
 
 
 def try_make(heads: int, nope_dim: int, latent_dim: int, rope_dim: int, row_stride: int, scale: float,

@@ -16,7 +16,7 @@
 template <typename TX, typename TW, typename TO, bool ACC>
 __global__ void __launch_bounds__(256) gemm_plain_kernel(const TX* x, const TW* __restrict__ w,
                                                          TO* __restrict__ out, int M, int N, int K,
-                                                         long long ldx, long long ldo) {
+                                                         long long ldx, long long ldo, const float* __restrict__ bias) {
     pdl_launch();
     pdl_wait();
     __shared__ float xs[BK][BM + 1];
@@ -69,6 +69,7 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(const TX* x, const TW* 
             const int n = n0 + tn + j;
             if (n >= N) continue;
             TO* o = out + (size_t)m * ldo + n;
+            if (bias != nullptr) acc[i][j] += bias[n];
             if (ACC) *o = from_f<TO>(to_f<TO>(*o) + acc[i][j]);
             else *o = from_f<TO>(acc[i][j]);
         }
@@ -77,14 +78,14 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(const TX* x, const TW* 
 
 template <typename TX, typename TW>
 static int launch(const void* x, const void* w, void* out, int out_dtype, int accumulate,
-                  int M, int N, int K, long long ldx, long long ldo, cudaStream_t stream) {
+                  int M, int N, int K, long long ldx, long long ldo, const float* bias, cudaStream_t stream) {
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     if (out_dtype == GG_F32) {
-        if (accumulate) gg_launch(gemm_plain_kernel<TX, TW, float, true>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (float*)out, M, N, K, ldx, ldo);
-        else gg_launch(gemm_plain_kernel<TX, TW, float, false>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (float*)out, M, N, K, ldx, ldo);
+        if (accumulate) gg_launch(gemm_plain_kernel<TX, TW, float, true>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (float*)out, M, N, K, ldx, ldo, bias);
+        else gg_launch(gemm_plain_kernel<TX, TW, float, false>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (float*)out, M, N, K, ldx, ldo, bias);
     } else if (out_dtype == GG_BF16) {
         if (accumulate) return GG_ERR_DTYPE;  // sums are kept in float32
-        gg_launch(gemm_plain_kernel<TX, TW, bf16, false>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (bf16*)out, M, N, K, ldx, ldo);
+        gg_launch(gemm_plain_kernel<TX, TW, bf16, false>, dim3(grid), dim3(256), 0, stream, 1, (const TX*)x, (const TW*)w, (bf16*)out, M, N, K, ldx, ldo, bias);
     } else {
         return GG_ERR_DTYPE;
     }
@@ -92,15 +93,16 @@ static int launch(const void* x, const void* w, void* out, int out_dtype, int ac
 }
 
 // x[M, K] with row stride ldx (elements), w[N, K] contiguous, out[M, N] with row stride ldo.
-// accumulate != 0: out += product (float32 out only; this is the residual add).
+// accumulate != 0: out += product (float32 out only; this is the residual add).  bias (may be null): [N] float32.
 GG_API gg_gemm_plain(const void* x, int x_dtype, const void* w, int w_dtype, void* out, int out_dtype,
-                     int accumulate, int M, int N, int K, long long ldx, long long ldo, cudaStream_t stream) {
+                     int accumulate, int M, int N, int K, long long ldx, long long ldo, const float* bias,
+                     cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || ldx < K || ldo < N) return GG_ERR_ARG;
     if ((M + BM - 1) / BM > 65535) return GG_ERR_ARG;
-    if (x_dtype == GG_F32 && w_dtype == GG_F32) return launch<float, float>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, stream);
-    if (x_dtype == GG_BF16 && w_dtype == GG_BF16) return launch<bf16, bf16>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, stream);
-    if (x_dtype == GG_BF16 && w_dtype == GG_F32) return launch<bf16, float>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, stream);
-    if (x_dtype == GG_F32 && w_dtype == GG_BF16) return launch<float, bf16>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, stream);
+    if (x_dtype == GG_F32 && w_dtype == GG_F32) return launch<float, float>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, bias, stream);
+    if (x_dtype == GG_BF16 && w_dtype == GG_BF16) return launch<bf16, bf16>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, bias, stream);
+    if (x_dtype == GG_BF16 && w_dtype == GG_F32) return launch<bf16, float>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, bias, stream);
+    if (x_dtype == GG_F32 && w_dtype == GG_BF16) return launch<float, bf16>(x, w, out, out_dtype, accumulate, M, N, K, ldx, ldo, bias, stream);
     return GG_ERR_DTYPE;
 }

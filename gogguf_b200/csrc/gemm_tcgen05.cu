@@ -93,7 +93,24 @@ struct NormIO {
     float eps;
     float* out_ssq;
     bf16* out_xhat;
+    const float* bias;       // [N] float32 or null: added to every row after the factor (all modes but SwiGLU and q/k/v)
 };
+
+// Bias values of `n` consecutive columns from c0 on (columns at or beyond N get 0), added to v.
+template <int n>
+__device__ __forceinline__ void add_bias(float* v, const float* __restrict__ bias, int c0, int N) {
+    if (c0 + n <= N && ((((uintptr_t)(bias + c0)) & 15) == 0)) {
+#pragma unroll
+        for (int j = 0; j < n / 4; ++j) {
+            const float4 b = reinterpret_cast<const float4*>(bias + c0)[j];
+            v[4 * j] += b.x; v[4 * j + 1] += b.y; v[4 * j + 2] += b.z; v[4 * j + 3] += b.w;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < n; ++j)
+            if (c0 + j < N) v[j] += bias[c0 + j];
+    }
+}
 
 // The q/k/v projection of an attention layer with what follows it fused into the epilogue (head size 128:
 // one head per 128-row weight tile of the decode form, two per tile of the CTA-pair form): per-head RMSNorm of q and k with one shared weight
@@ -341,6 +358,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
                     float4 v = make_float4(__uint_as_float(r[16 * q + 4 * j]), __uint_as_float(r[16 * q + 4 * j + 1]),
                                            __uint_as_float(r[16 * q + 4 * j + 2]), __uint_as_float(r[16 * q + 4 * j + 3]));
                     if (scaled) { v.x *= sc; v.y *= sc; v.z *= sc; v.w *= sc; }
+                    if (nio.bias != nullptr) add_bias<4>(&v.x, nio.bias, tn * BN + c0 + 16 * q + 4 * j, N);
                     v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
                     reinterpret_cast<float4*>(orow + c0 + 16 * q)[j] = v;
                     if (stats) {
@@ -373,6 +391,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
 #pragma unroll
             for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
         }
+        if (nio.bias != nullptr) add_bias<16>(reinterpret_cast<float*>(r), nio.bias, tn * BN + c0, N);
         store_row_chunk16(r, gi, tn * BN + c0, N, out, out_mode, ldo, nio, ss);
     }
 }
@@ -530,6 +549,7 @@ __device__ __forceinline__ void finish_token_block(float4 acc, int gj, int tile_
         const bool whole = gi0 + 4 <= N;
         const size_t o = (size_t)gj * ldo + gi0;
         float f[4] = {acc.x, acc.y, acc.z, acc.w};
+        if (nio.bias != nullptr) add_bias<4>(f, nio.bias, gi0, N);
         if (out_mode == OUT_BF16) {
             bf16* op = (bf16*)out + o;
             if (whole && (((uintptr_t)op) & 7) == 0) {
@@ -622,10 +642,10 @@ __global__ void __launch_bounds__(NUM_THREADS, MINB) gemm_tc_kernel(
     uint64_t* accum = empty + STAGES;
     uint64_t* recv_bar = accum + 1;
     // the tile goes through shared memory when K splits are added inside the cluster, for the fused
-    // activation, and (decode form) whenever a norm is folded into this product
+    // activation, and (decode form) whenever a norm is folded into this product or a bias goes with it
     // (only the decode form splits K or fuses the activation; the launcher sees to that)
     const bool staged = SWAP && (cluster_reduce || out_mode == OUT_SWIGLU || out_mode == OUT_QKV ||
-                                 (partial == nullptr && (nio.in_ssq != nullptr || nio.out_ssq != nullptr)));
+                                 (partial == nullptr && (nio.in_ssq != nullptr || nio.out_ssq != nullptr || nio.bias != nullptr)));
     uint32_t* tmem_slot = (uint32_t*)(recv_bar + 1);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
     // decode form with a folded norm: the factor of every token of the tile, computed by the epilogue warps while
@@ -802,6 +822,7 @@ __global__ void __launch_bounds__(NUM_THREADS, MINB) gemm_tc_kernel(
 #pragma unroll
                         for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
                     }
+                    if (nio.bias != nullptr) add_bias<16>(reinterpret_cast<float*>(r), nio.bias, gj0, N);
                     store_row_chunk16(r, gi, gj0, N, out, out_mode, ldo, nio, ss);
                 }
             }
@@ -1658,7 +1679,7 @@ GG_API gg_gemm_tc(const void* x, const void* w, void* out, int out_mode, int M, 
                   long long ldo, float* scratch, long long scratch_elems, int use_cluster, int* status,
                   cudaStream_t stream) {
     if (out_mode == OUT_QKV) return GG_ERR_ARG;
-    const NormIO none = {nullptr, 0, 0.f, 0.f, nullptr, nullptr};
+    const NormIO none = {nullptr, 0, 0.f, 0.f, nullptr, nullptr, nullptr};
     const QkvIO noq = {};
     return gemm_tc_impl(x, w, out, out_mode, M, N, K, ldx, ldo, scratch, scratch_elems, use_cluster, status, none, noq, stream);
 }
@@ -1672,13 +1693,15 @@ GG_API gg_gemm_tc(const void* x, const void* w, void* out, int out_mode, int M, 
 //   out_ssq != null (out_mode 2 only): after out += product the kernel also writes out_xhat[M, N]
 //     (bfloat16 copy of the updated rows, row stride N) and out_ssq[M, ceil(N / 128)], their partial sums
 //     of squares over blocks of 128 columns: the inputs of the next folded product.
+//   bias != null (not with out_mode 3): [N] float32, added to every row after the factor, before the output mode.
 GG_API gg_gemm_tc_norm(const void* x, const void* w, void* out, int out_mode, int M, int N, int K, long long ldx,
                        long long ldo, const float* in_ssq, int in_parts, float eps, float* out_ssq, void* out_xhat,
-                       float* scratch, long long scratch_elems, int* status, cudaStream_t stream) {
+                       const float* bias, float* scratch, long long scratch_elems, int* status, cudaStream_t stream) {
     if (in_ssq != nullptr && (in_parts != (K + 127) / 128 || !(eps > 0.f))) return GG_ERR_ARG;
+    if (bias != nullptr && out_mode == OUT_SWIGLU) return GG_ERR_ARG;
     if (out_ssq != nullptr && (out_mode != OUT_F32_ACC || out_xhat == nullptr)) return GG_ERR_ARG;
     if (out_mode == OUT_QKV) return GG_ERR_ARG;
-    const NormIO nio = {in_ssq, in_parts, 1.0f / (float)K, eps, out_ssq, (bf16*)out_xhat};
+    const NormIO nio = {in_ssq, in_parts, 1.0f / (float)K, eps, out_ssq, (bf16*)out_xhat, bias};
     const QkvIO noq = {};
     return gemm_tc_impl(x, w, out, out_mode, M, N, K, ldx, ldo, scratch, scratch_elems, 1, status, nio, noq, stream);
 }
@@ -1703,7 +1726,7 @@ GG_API gg_gemm_tc_qkv_rope(const void* x, const void* w, int M, int K, long long
                            int max_pages, int page_size, int n_pages, void* k_pool, void* v_pool, int nq, int nkv,
                            float* scratch, long long scratch_elems, int* status, cudaStream_t stream) {
     if (in_ssq != nullptr && (in_parts != (K + 127) / 128 || !(in_eps > 0.f))) return GG_ERR_ARG;
-    const NormIO nio = {in_ssq, in_parts, K > 0 ? 1.0f / (float)K : 0.f, in_eps, nullptr, nullptr};
+    const NormIO nio = {in_ssq, in_parts, K > 0 ? 1.0f / (float)K : 0.f, in_eps, nullptr, nullptr, nullptr};
     const QkvIO qio = {(bf16*)q_out, qw, kw, eps, cosv, sinv, positions, seq_of_token, page_table, max_pages, page_size,
                        (bf16*)k_pool, (bf16*)v_pool, nq, nkv, n_pages, status};
     const int N = (nq + 2 * nkv) * 128;

@@ -294,10 +294,10 @@ def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.T
                                               int(rows), n, float(eps), _stream())
 
 
-def softcap(z: torch.Tensor, cap: float, n: Optional[int] = None) -> None:
-    """z <- cap * tanh(z / cap) in place (float32)."""
+def softcap(z: torch.Tensor, cap: float, n: Optional[int] = None, scale: float = 1.0) -> None:
+    """z <- cap * tanh(scale * z / cap) in place (float32); cap 0: z <- scale * z."""
     _need(z, torch.float32, "logits")
-    kernel("elementwise", "gg_softcap")(_p(z), float(cap), int(z.numel() if n is None else n), _stream())
+    kernel("elementwise", "gg_softcap")(_p(z), float(cap), float(scale), int(z.numel() if n is None else n), _stream())
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, n_tokens: int, inter: int) -> None:
@@ -339,17 +339,21 @@ def feed_tokens(tokens: torch.Tensor, src: torch.Tensor, sampled: torch.Tensor, 
 
 # ------------------------------------------------------------------------------- matrix product
 def gemm_plain(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
-               m: Optional[int] = None) -> None:
-    """out[M, N] (+)= x[M, K] @ w[N, K]^T on the CUDA cores with float32 accumulation."""
+               m: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> None:
+    """out[M, N] (+)= x[M, K] @ w[N, K]^T (+ bias [N], float32) on the CUDA cores with float32 accumulation."""
     N, K = w.shape
     M = x.shape[0] if m is None else m
     if x.shape[-1] != K or out.shape[-1] != N:
         raise KernelError(f"gemm: x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)} disagree")
     if x.stride(-1) != 1 or out.stride(-1) != 1 or not w.is_contiguous():
         raise KernelError("gemm: operands must be row-major")
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        if bias.numel() != N:
+            raise KernelError("gemm: the bias has one number per output column")
     kernel("gemm_plain", "gg_gemm_plain")(_p(x), dtype_code(x.dtype), _p(w), dtype_code(w.dtype), _p(out),
                                            dtype_code(out.dtype), int(accumulate), M, N, K,
-                                           x.stride(0), out.stride(0), _stream())
+                                           x.stride(0), out.stride(0), _p(bias), _stream())
 
 
 # ------------------------------------------------------------------------------- attention
@@ -450,6 +454,98 @@ def diff_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tens
         _p(partial), int(max_new), _p(status_word(q.device)), _stream())
 
 
+def head_kv_prep(row: torch.Tensor, k_off: int, v_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                 positions: torch.Tensor, seq_of_token: torch.Tensor, page_table: torch.Tensor, page_size: int,
+                 n_tokens: int, kv_heads: int, d: int, dv: int, unit: bool, eps: float,
+                 first: Optional[torch.Tensor] = None, lam: float = 0.0, keep: Optional[torch.Tensor] = None) -> None:
+    """Keys (column k_off of the projection row) and values (column v_off) into the paged cache.  unit: each head's
+    values are divided by their root mean square (eps inside).  first (float32 [T, kv_heads * dv]): the values become
+    (1 - lam) v + lam first; keep (like first): this layer's values are left there, unmixed."""
+    if not (row.dtype == k_pool.dtype == v_pool.dtype) or row.stride(-1) != 1:
+        raise KernelError("head_kv_prep: rows and cache must share one dtype")
+    if k_pool.shape[-1] != d or v_pool.shape[-1] != dv or k_pool.shape[1] != kv_heads or v_pool.shape[1] != kv_heads:
+        raise KernelError("head_kv_prep: the pools do not fit the heads")
+    for t in (first, keep):
+        if t is not None:
+            _need(t, torch.float32, "first / keep")
+            if t.numel() < n_tokens * kv_heads * dv:
+                raise KernelError("head_kv_prep: first / keep hold kv_heads * dv numbers per token")
+    from .tcgen05_gemm import status_word
+    kernel("mixed_head_attention", "gg_head_kv_prep")(
+        _p(row), row.stride(0), dtype_code(row.dtype), int(k_off), int(v_off), _p(k_pool), _p(v_pool), _p(positions),
+        _p(seq_of_token), _p(page_table), page_table.shape[-1], int(page_size), k_pool.shape[0], int(n_tokens),
+        int(kv_heads), int(d), int(dv), int(bool(unit)), float(eps), _p(first), float(lam), _p(keep),
+        _p(status_word(row.device)), _stream())
+
+
+def _mixed_head_check(row, k_pool, v_pool, out, talk, H: int, G: int, d: int, dv: int, g_off: int) -> None:
+    if not (row.dtype == k_pool.dtype == v_pool.dtype == out.dtype) or row.stride(-1) != 1 or out.stride(-1) != 1:
+        raise KernelError("mixed_head_attention: rows, cache and output must share one dtype")
+    _need(talk, torch.float32, "talk")
+    if talk.numel() != H * H or k_pool.shape[-1] != d or v_pool.shape[-1] != dv or k_pool.shape[1] != G:
+        raise KernelError("mixed_head_attention: the mixing matrix or the pools do not fit the heads")
+    if row.shape[-1] < max(H * d, g_off + H) or out.shape[-1] < H * dv:
+        raise KernelError("mixed_head_attention: the rows are too short for the heads")
+
+
+def mixed_head_attention_plain(row: torch.Tensor, g_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
+                               talk: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
+                               page_table: torch.Tensor, page_size: int, n_tokens: int, heads: int, kv_heads: int, d: int,
+                               dv: int, scale: float, cap: float = 0.0, coef: float = 0.0, every: float = 1.0,
+                               one: bool = False, window: int = 0) -> None:
+    """Attention over the paged cache whose heads' weights are mixed by talk [heads, heads] (float32) before they meet
+    the values; q at column 0 of the projection row, the heads' gate logits at column g_off (negative: no gate).  cap:
+    scores bounded by cap tanh(s / cap); coef, every: the query temperature; one: one joins the softmax's denominator."""
+    _mixed_head_check(row, k_pool, v_pool, out, talk, heads, kv_heads, d, dv, g_off)
+    from .tcgen05_gemm import status_word
+    kernel("mixed_head_attention", "gg_mixed_head_attention_plain")(
+        _p(row), row.stride(0), int(g_off), _p(k_pool), _p(v_pool), _p(out), out.stride(0), dtype_code(row.dtype), _p(talk),
+        _p(positions), _p(seq_of_token), _p(page_table), page_table.shape[-1], int(page_size), k_pool.shape[0], int(n_tokens),
+        int(heads), int(kv_heads), int(d), int(dv), float(scale), float(cap), float(coef), float(every), float(bool(one)),
+        int(window), _p(status_word(row.device)), _stream())
+
+
+def mixed_head_mma_takes(heads: int, kv_heads: int, d: int, dv: int, page_size: int) -> bool:
+    """Does the tensor-core form of attention with mixed heads take these sizes (bfloat16 tensors)?"""
+    from .build import module
+    return bool(module("mixed_head_attention").lib.gg_mixed_head_mma_takes(int(heads), int(kv_heads), int(d), int(dv),
+                                                                          int(page_size)))
+
+
+def mixed_head_splits(n_tokens: int, n_seqs: int, heads: int, kv_heads: int, max_ctx: int) -> int:
+    """Into how many shares a step's key tiles are cut (see `diff_attention_splits`)."""
+    tpt = max(1, 64 // (heads // kv_heads))
+    ctas = max(n_seqs, -(-n_tokens // tpt)) * kv_heads * ((kv_heads + 1) // 2)
+    tiles = -(-max_ctx // 64)
+    if ctas >= 148 or tiles < 4:
+        return 1
+    return int(max(1, min(32, 296 // max(ctas, 1), tiles // 2)))
+
+
+def mixed_head_attention_mma(row: torch.Tensor, g_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
+                             talk: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
+                             cu_seqlens: torch.Tensor, page_table: torch.Tensor, page_size: int, n_tokens: int, n_seqs: int,
+                             heads: int, kv_heads: int, d: int, dv: int, scale: float, u: torch.Tensor, ml: torch.Tensor,
+                             cap: float = 0.0, coef: float = 0.0, every: float = 1.0, one: bool = False, window: int = 0,
+                             nsplit: int = 1, max_new: int = 0) -> None:
+    """`mixed_head_attention_plain` on the tensor cores (mma.sync) for bfloat16 tensors.  Scratch (float32): u of
+    n_tokens * heads * nsplit * kv_heads * dv numbers, ml of n_tokens * heads * nsplit * 2.  max_new: the most rows one
+    sequence brings, where the caller knows it."""
+    _mixed_head_check(row, k_pool, v_pool, out, talk, heads, kv_heads, d, dv, g_off)
+    _need(row, torch.bfloat16, "row")
+    _need(u, torch.float32, "u")
+    _need(ml, torch.float32, "ml")
+    if u.numel() < n_tokens * heads * nsplit * kv_heads * dv or ml.numel() < n_tokens * heads * nsplit * 2:
+        raise KernelError("mixed_head_attention_mma: the scratch is too small")
+    from .tcgen05_gemm import status_word
+    kernel("mixed_head_attention", "gg_mixed_head_attention_mma")(
+        _p(row), row.stride(0), int(g_off), _p(k_pool), _p(v_pool), _p(out), out.stride(0), _p(talk), _p(positions),
+        _p(seq_of_token), _p(cu_seqlens), _p(page_table), page_table.shape[-1], int(page_size), k_pool.shape[0],
+        int(n_tokens), int(n_seqs), int(heads), int(kv_heads), int(d), int(dv), float(scale), float(cap), float(coef),
+        float(every), float(bool(one)), int(window), int(nsplit), _p(u), _p(ml), int(max_new), _p(status_word(row.device)),
+        _stream())
+
+
 def diff_attention_partial_elems(n_tokens: int, heads: int, dv: int, nsplit: int) -> int:
     return n_tokens * heads * nsplit * 2 * (2 + dv)
 
@@ -469,11 +565,13 @@ def diff_attention_splits(n_tokens: int, n_seqs: int, heads: int, kv_heads: int,
 def latent_prep(q: torch.Tensor, dkv: torch.Tensor, norm_weight: torch.Tensor, eps: float, cos: torch.Tensor,
                 sin: torch.Tensor, rot_dims: int, positions: torch.Tensor, seq_of_token: torch.Tensor,
                 page_table: torch.Tensor, page_size: int, pool: Optional[torch.Tensor], qcat: torch.Tensor,
-                n_tokens: int, heads: int, d: int, r: int, R: int, dense: Optional[torch.Tensor] = None) -> None:
+                n_tokens: int, heads: int, d: int, r: int, R: int, dense: Optional[torch.Tensor] = None,
+                pairing: str = "adjacent") -> None:
     """Norm of the latent, rotation of the shared key part and of the queries' rotated parts, cache write.
     q [T, heads * (d + r)] and dkv [T, R + r] may be column ranges of one buffer (row strides are passed);
     pool [page][page_size][row]; qcat [T, heads, R + r] receives the rotated parts at [..., R:]; dense (optional,
-    contiguous [T, R + r] in the cache's dtype) receives the rows the cache gets, token by token."""
+    contiguous [T, R + r] in the cache's dtype) receives the rows the cache gets, token by token.
+    pairing: "adjacent" (2i with 2i + 1) or "halves" (i with i + rot_dims / 2)."""
     if q.dtype != dkv.dtype or (pool is not None and pool.dtype != q.dtype):
         raise KernelError("latent_prep: q, dkv and the cache must share one dtype")
     if q.stride(-1) != 1 or dkv.stride(-1) != 1 or not qcat.is_contiguous():
@@ -486,19 +584,23 @@ def latent_prep(q: torch.Tensor, dkv: torch.Tensor, norm_weight: torch.Tensor, e
         _p(q), q.stride(0), _p(dkv), dkv.stride(0), dtype_code(q.dtype), _p(norm_weight), float(eps), _p(cos), _p(sin),
         int(rot_dims), _p(positions), _p(seq_of_token), _p(page_table), page_table.shape[-1], int(page_size),
         pool.shape[0] if pool is not None else 0, _p(pool), pool.shape[-1] if pool is not None else R + r,
-        _p(qcat), dtype_code(qcat.dtype), n_tokens, heads, d, r, R, _p(dense), _p(status_word(q.device)), _stream())
+        _p(qcat), dtype_code(qcat.dtype), n_tokens, heads, d, r, R, _p(dense), int(pairing == "halves"), _p(status_word(q.device)), _stream())
 
 
 def headwise_gemm(x: torch.Tensor, ldx: int, hx: int, w: torch.Tensor, out: torch.Tensor, ldo: int, ho: int,
-                  m: int, alpha: float = 1.0) -> None:
+                  m: int, alpha: float = 1.0, gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h, :] = alpha * w[h] @ x[t, h, :] for w [H, N, K]; x[t, h] starts at t * ldx + h * hx elements
-    into x, out[t, h] at t * ldo + h * ho into out."""
+    into x, out[t, h] at t * ldo + h * ho into out.  gate (rows of H * N logits in the output's dtype): the result is
+    multiplied by their sigmoid."""
     H, N, K = w.shape
+    if gate is not None and (gate.dtype != out.dtype or gate.stride(-1) != 1 or gate.shape[-1] != H * N):
+        raise KernelError("headwise_gemm: the gate has rows of H * N logits in the output's dtype")
     if not w.is_contiguous():
         raise KernelError("headwise_gemm: the weights must be contiguous [H, N, K]")
     kernel("latent_attention", "gg_headwise_gemm")(_p(x), dtype_code(x.dtype), int(ldx), int(hx), _p(w),
                                                     dtype_code(w.dtype), _p(out), dtype_code(out.dtype), int(ldo),
-                                                    int(ho), int(m), N, K, H, float(alpha), _stream())
+                                                    int(ho), int(m), N, K, H, float(alpha), _p(gate),
+                                                    gate.stride(0) if gate is not None else 0, _stream())
 
 
 def latent_attention_plain(qcat: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,

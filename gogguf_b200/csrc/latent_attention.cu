@@ -23,14 +23,14 @@
 // ----------------------------------------------------------------------------- prep
 // One block per token.  dkv[t] = [latent (R) | key part (r)] as the down projection left it; q[t] holds H heads
 // of [plain (d) | rot (r)].  Writes pool row [rms(latent) * w | rotate(key part)] and qcat[t, h, R : R + r] =
-// rotate(q rot part).  The rotation pairs element 2i with 2i+1 for i < dims / 2 and leaves the rest as it is;
-// cos/sin[t, i] are the step's tables.  Padding tokens (seq_of_token < 0) write zeros to qcat and no cache.
+// rotate(q rot part).  The rotation pairs element 2i with 2i+1 (halves != 0: i with i + dims / 2) for i < dims / 2 and
+// leaves the rest as it is; cos/sin[t, i] are the step's tables.  Padding tokens (seq_of_token < 0) write zeros to qcat and no cache.
 template <typename T, typename TQ>
 __global__ void __launch_bounds__(256) latent_prep_kernel(
     const T* q, long long ldq, const T* dkv, long long lddkv, const float* __restrict__ normw, float eps,
     const float* cosv, const float* sinv, int dims, const int* __restrict__ positions,
     const int* __restrict__ seq_of_token, const int* __restrict__ page_table, int max_pages, int page_size,
-    T* pool, int pool_row, TQ* qcat, int H, int d, int r, int R, const PageBounds pb, T* dense) {
+    T* pool, int pool_row, TQ* qcat, int H, int d, int r, int R, const PageBounds pb, T* dense, int halves) {
     pdl_launch();
     pdl_wait();
     __shared__ float red[33];
@@ -44,18 +44,22 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(
     }
     const float* cs = cosv + (size_t)t * half;
     const float* sn = sinv + (size_t)t * half;
+    auto turned = [&](const T* src, int e) {             // element e of a rotated run that starts at src
+        float v = to_f<T>(src[e]);
+        if (e < dims) {
+            const bool first = halves ? e < half : !(e & 1);
+            const int i = halves ? (first ? e : e - half) : e >> 1;
+            const float o = to_f<T>(src[halves ? (first ? e + half : e - half) : e ^ 1]);
+            v = first ? v * cs[i] - o * sn[i] : v * cs[i] + o * sn[i];
+        }
+        return v;
+    };
     // rotated part of every query head
     const T* qt = q + (size_t)t * ldq;
     for (int i = threadIdx.x; i < H * r; i += blockDim.x) {
         const int h = i / r, e = i % r;
         const T* src = qt + (size_t)h * (d + r) + d;
-        float v = to_f<T>(src[e]);
-        if (e < dims) {
-            const float o = to_f<T>(src[e ^ 1]);
-            const float c = cs[e >> 1], s = sn[e >> 1];
-            v = (e & 1) ? v * c + o * s : v * c - o * s;
-        }
-        qc[(size_t)h * (R + r) + R + e] = from_f<TQ>(v);
+        qc[(size_t)h * (R + r) + R + e] = from_f<TQ>(turned(src, e));
     }
     if (pool == nullptr && dense == nullptr) return;
     const T* dk = dkv + (size_t)t * lddkv;
@@ -76,31 +80,26 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(
         if (drow != nullptr) drow[i] = v;
     }
     for (int e = threadIdx.x; e < r; e += blockDim.x) {
-        float v = to_f<T>(dk[R + e]);
-        if (e < dims) {
-            const float o = to_f<T>(dk[R + (e ^ 1)]);
-            const float c = cs[e >> 1], s = sn[e >> 1];
-            v = (e & 1) ? v * c + o * s : v * c - o * s;
-        }
+        const float v = turned(dk + R, e);
         if (row != nullptr) row[R + e] = from_f<T>(v);
         if (drow != nullptr) drow[R + e] = from_f<T>(v);
     }
 }
 
 // q, dkv and the pool share `dtype`; qcat has `q_dtype`.  pool may be null (a layer that reads another's cache).
-// dense (may be null): [T, R + r] in `dtype`, the rows the cache gets, token by token.
+// dense (may be null): [T, R + r] in `dtype`, the rows the cache gets, token by token.  halves: how pairs are formed.
 GG_API gg_latent_prep(const void* q, long long ldq, const void* dkv, long long lddkv, int dtype, const float* normw,
                       float eps, const float* cosv, const float* sinv, int dims, const int* positions,
                       const int* seq_of_token, const int* page_table, int max_pages, int page_size, int n_pages,
                       void* pool, int pool_row, void* qcat, int q_dtype, int ntok, int H, int d, int r, int R,
-                      void* dense, int* status, cudaStream_t stream) {
+                      void* dense, int halves, int* status, cudaStream_t stream) {
     if (ntok <= 0) return 0;
     if (H <= 0 || d <= 0 || r < 0 || R <= 0 || dims < 0 || dims > r || (dims & 1) || pool_row < R + r || page_size <= 0)
         return GG_ERR_ARG;
     const PageBounds pb{n_pages, status};
 #define GG_PREP(T, TQ) gg_launch(latent_prep_kernel<T, TQ>, dim3(ntok), dim3(256), 0, stream, 1, (const T*)q, ldq, \
         (const T*)dkv, lddkv, normw, eps, cosv, sinv, dims, positions, seq_of_token, page_table, max_pages, page_size, \
-        (T*)pool, pool_row, (TQ*)qcat, H, d, r, R, pb, (T*)dense)
+        (T*)pool, pool_row, (TQ*)qcat, H, d, r, R, pb, (T*)dense, halves)
     if (dtype == GG_F32 && q_dtype == GG_F32) GG_PREP(float, float);
     else if (dtype == GG_BF16 && q_dtype == GG_F32) GG_PREP(bf16, float);
     else if (dtype == GG_BF16 && q_dtype == GG_BF16) GG_PREP(bf16, bf16);
@@ -112,13 +111,18 @@ GG_API gg_latent_prep(const void* q, long long ldq, const void* dkv, long long l
 // ----------------------------------------------------------------------------- per-head products
 // out[t, h, n] = alpha * sum_k x[t, h, k] * w[h, n, k] for h < H: H small products that share the token axis.
 // x[t, h, k] is at x + t * ldx + h * hx + k, out[t, h, n] at out + t * ldo + h * ho + n, w[h] is [N, K] row-major.
-// The sum over k runs in a fixed order that does not depend on the number of tokens.
+// The sum over k runs in a fixed order that does not depend on the number of tokens.  gate (may be null): a logit per
+// output, in the output's type, at gate + t * ldg + h * N + n; the output is multiplied by its sigmoid.
 #define HB 64
 #define HK 16
+template <typename TG>
+__device__ __forceinline__ float gate_factor(const TG* gate, size_t at) { return 1.0f / (1.0f + expf(-to_f<TG>(gate[at]))); }
+
 template <typename TX, typename TW, typename TO>
 __global__ void __launch_bounds__(256) headwise_gemm_kernel(const TX* x, long long ldx, long long hx,
                                                             const TW* __restrict__ w, TO* out, long long ldo,
-                                                            long long ho, int M, int N, int K, float alpha) {
+                                                            long long ho, int M, int N, int K, float alpha,
+                                                            const TO* gate, long long ldg) {
     pdl_launch();
     pdl_wait();
     __shared__ float xs[HK][HB + 1];
@@ -170,19 +174,23 @@ __global__ void __launch_bounds__(256) headwise_gemm_kernel(const TX* x, long lo
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tn + j;
-            if (n < N) out[(size_t)m * ldo + (size_t)h * ho + n] = from_f<TO>(acc[i][j] * alpha);
+            if (n >= N) continue;
+            float v = acc[i][j] * alpha;
+            if (gate != nullptr) v *= gate_factor(gate, (size_t)m * ldg + (size_t)h * N + n);
+            out[(size_t)m * ldo + (size_t)h * ho + n] = from_f<TO>(v);
         }
     }
 }
 
 GG_API gg_headwise_gemm(const void* x, int x_dtype, long long ldx, long long hx, const void* w, int w_dtype,
                         void* out, int out_dtype, long long ldo, long long ho, int M, int N, int K, int H,
-                        float alpha, cudaStream_t stream) {
+                        float alpha, const void* gate, long long ldg,
+                            cudaStream_t stream) {
     if (M <= 0 || N <= 0 || H <= 0) return 0;
     if (K <= 0 || H > 65535 || (M + HB - 1) / HB > 65535) return GG_ERR_ARG;
     dim3 grid((N + HB - 1) / HB, (M + HB - 1) / HB, H);
 #define GG_HW(TX, TW, TO) gg_launch(headwise_gemm_kernel<TX, TW, TO>, dim3(grid), dim3(256), 0, stream, 1, \
-        (const TX*)x, ldx, hx, (const TW*)w, (TO*)out, ldo, ho, M, N, K, alpha)
+        (const TX*)x, ldx, hx, (const TW*)w, (TO*)out, ldo, ho, M, N, K, alpha, (const TO*)gate, ldg)
     const int code = x_dtype * 4 + w_dtype * 2 + out_dtype;
     switch (code) {
         case 0: GG_HW(float, float, float); break;
@@ -336,7 +344,8 @@ __device__ __forceinline__ void zero16(void* smem) { *reinterpret_cast<uint4*>(s
 template <typename TO>
 __global__ void __launch_bounds__(128) headwise_mma_kernel(const bf16* x, long long ldx, long long hx,
                                                            const bf16* __restrict__ w, TO* out, long long ldo,
-                                                           long long ho, int M, int N, int K, float alpha) {
+                                                           long long ho, int M, int N, int K, float alpha,
+                                                           const TO* gate, long long ldg) {
     pdl_launch();
     __shared__ __align__(16) bf16 xs[64 * HM_LD];
     __shared__ __align__(16) bf16 ws[64 * HM_LD];
@@ -384,14 +393,21 @@ __global__ void __launch_bounds__(128) headwise_mma_kernel(const bf16* x, long l
             const int m = m0 + warp * 16 + g + half * 8;
             if (m >= M) continue;
             TO* o = out + (size_t)m * ldo + (size_t)h * ho + n;
-            if (n < N) o[0] = from_f<TO>(acc[nt][2 * half] * alpha);
-            if (n + 1 < N) o[1] = from_f<TO>(acc[nt][2 * half + 1] * alpha);
+            float v0 = acc[nt][2 * half] * alpha, v1 = acc[nt][2 * half + 1] * alpha;
+            if (gate != nullptr) {
+                const size_t at = (size_t)m * ldg + (size_t)h * N + n;
+                if (n < N) v0 *= gate_factor(gate, at);
+                if (n + 1 < N) v1 *= gate_factor(gate, at + 1);
+            }
+            if (n < N) o[0] = from_f<TO>(v0);
+            if (n + 1 < N) o[1] = from_f<TO>(v1);
         }
     }
 }
 
 GG_API gg_headwise_gemm_mma(const void* x, long long ldx, long long hx, const void* w, void* out, int out_dtype,
-                            long long ldo, long long ho, int M, int N, int K, int H, float alpha, cudaStream_t stream) {
+                            long long ldo, long long ho, int M, int N, int K, int H, float alpha, const void* gate,
+                                long long ldg, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || H <= 0) return 0;
     if (K <= 0 || (K % 8) || (ldx % 8) || (hx % 8) || (((uintptr_t)x) & 15) || (((uintptr_t)w) & 15) || H > 65535 ||
         (M + 63) / 64 > 65535)
@@ -399,7 +415,7 @@ GG_API gg_headwise_gemm_mma(const void* x, long long ldx, long long hx, const vo
     dim3 grid((N + 63) / 64, (M + 63) / 64, H);
     GG_DISPATCH_DTYPE(out_dtype, TO,
         gg_launch(headwise_mma_kernel<TO>, dim3(grid), dim3(128), 0, stream, 1, (const bf16*)x, ldx, hx,
-                  (const bf16*)w, (TO*)out, ldo, ho, M, N, K, alpha));
+                  (const bf16*)w, (TO*)out, ldo, ho, M, N, K, alpha, (const TO*)gate, ldg));
     return gg_last_error();
 }
 
@@ -754,7 +770,8 @@ template <int DVT>
 __global__ void __launch_bounds__(128) latent_prompt_mma_kernel(
     const bf16* qd, long long ldq, const bf16* qcat, const bf16* kv, long long ldkv, const bf16* ckr, long long ldc,
     bf16* av, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_of_token, int n_seqs, int H, int d, int r,
-    int dv, int R, float scale_log2, int window, float out_scale, const float* __restrict__ sink) {
+    int dv, int R, float scale_log2, int window, float out_scale, const float* __restrict__ sink, const bf16* gate,
+    long long ldg) {
     pdl_launch();
     extern __shared__ __align__(16) unsigned char smraw[];
     constexpr int KT = 64;
@@ -933,7 +950,14 @@ __global__ void __launch_bounds__(128) latent_prompt_mma_kernel(
 #pragma unroll
         for (int nt = 0; nt < DVT / 8; ++nt) {
             const int c = nt * 8 + 2 * q4;
-            if (c < dv) *reinterpret_cast<uint32_t*>(orow + c) = pack_bf16(o[nt][2 * i] * inv, o[nt][2 * i + 1] * inv);
+            if (c >= dv) continue;
+            float v0 = o[nt][2 * i] * inv, v1 = o[nt][2 * i + 1] * inv;
+            if (gate != nullptr) {
+                const size_t at = (size_t)(t0 + prow[i]) * ldg + (size_t)h * dv + c;
+                v0 *= gate_factor(gate, at);
+                v1 *= gate_factor(gate, at + 1);
+            }
+            *reinterpret_cast<uint32_t*>(orow + c) = pack_bf16(v0, v1);
         }
     }
 }
@@ -947,11 +971,12 @@ GG_API gg_latent_prompt_mma_takes(int d, int r, int dv) {
 
 // qd [T, >= H (d + r)] (row stride ldq; head h's plain query at h (d + r)), qcat [T, H, R + r] (rotated query parts
 // at [..., R:]), kv [T, H d + H dv] (row stride ldkv), ckr [T, R + r] (row stride ldc; rotated key part at R),
-// av [T, H, dv]; every sequence of the step starts at position 0.
+// av [T, H, dv]; every sequence of the step starts at position 0.  gate (may be null): a bfloat16 logit per output,
+// at gate + t * ldg + h * dv + i; the output is multiplied by its sigmoid.
 GG_API gg_latent_prompt_mma(const void* qd, long long ldq, const void* qcat, const void* kv, long long ldkv,
                             const void* ckr, long long ldc, void* av, const int* cu_seqlens, const int* seq_of_token,
                             int n_seqs, int ntok, int H, int d, int r, int dv, int R, float scale, int window,
-                            float out_scale, const float* sink, cudaStream_t stream) {
+                            float out_scale, const float* sink, const void* gate, long long ldg, cudaStream_t stream) {
     if (ntok <= 0 || n_seqs <= 0) return 0;
     if (!gg_latent_prompt_mma_takes(d, r, dv) || H <= 0 || H > 65535 || (ldq % 8) || (ldkv % 8) || (ldc % 8) ||
         ((R + r) % 8) || (R % 8) || ((H * d) % 8) ||
@@ -970,7 +995,7 @@ GG_API gg_latent_prompt_mma(const void* qd, long long ldq, const void* qcat, con
         }
         return gg_launch(kern, dim3(grid), dim3(128), smem, stream, 1, (const bf16*)qd, ldq, (const bf16*)qcat, (const bf16*)kv,
                          ldkv, (const bf16*)ckr, ldc, (bf16*)av, cu_seqlens, seq_of_token, n_seqs, H, d, r, dv, R, sl2, window,
-                         out_scale, sink);
+                         out_scale, sink, (const bf16*)gate, ldg);
     }
     auto kern = latent_prompt_mma_kernel<128>;
     static bool set2 = false;
@@ -980,7 +1005,8 @@ GG_API gg_latent_prompt_mma(const void* qd, long long ldq, const void* qcat, con
         set2 = true;
     }
     return gg_launch(kern, dim3(grid), dim3(128), smem, stream, 1, (const bf16*)qd, ldq, (const bf16*)qcat, (const bf16*)kv, ldkv,
-                     (const bf16*)ckr, ldc, (bf16*)av, cu_seqlens, seq_of_token, n_seqs, H, d, r, dv, R, sl2, window, out_scale, sink);
+                     (const bf16*)ckr, ldc, (bf16*)av, cu_seqlens, seq_of_token, n_seqs, H, d, r, dv, R, sl2, window, out_scale, sink,
+                     (const bf16*)gate, ldg);
 }
 
 GG_API gg_latent_attention_checked() { return gg_debug_bounds(); }

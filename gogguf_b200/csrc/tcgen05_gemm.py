@@ -30,11 +30,11 @@ def check_status(device: torch.device) -> None:
     v = int(t.item())
     if v != 0:
         t.zero_()
-        if 41 <= v <= 51:
+        if 41 <= v <= 53:
             who = {41: "attention_plain", 42: "attn_decode", 43: "attn_prefill", 44: "attn_decode_tma",
                    45: "attn_prefill_tc", 46: "qk_norm_rope_cache", 47: "qk_norm_rope_cache (16-byte form)",
                    48: "the q/k/v product's cache write", 49: "latent_prep", 50: "diff_qk_prep",
-                   51: "diff_attention"}[v]
+                   51: "diff_attention", 52: "head_kv_prep", 53: "mixed_head_attention"}[v]
             raise KernelError(f"debug build: kernel {who} met a page-table index or page id out of range (code {v}); "
                               "it read page 0 (a reader) or wrote nothing (a writer), results of that step are invalid")
         raise KernelError(f"a bounded wait inside a kernel ran out (code {v}: 1 TMA producer, 2 MMA issuer, "
@@ -106,8 +106,10 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: boo
 def gemm_tc_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False,
                  m: Optional[int] = None, swiglu: bool = False, in_ssq: Optional[torch.Tensor] = None,
                  eps: float = 0.0, out_ssq: Optional[torch.Tensor] = None,
-                 out_xhat: Optional[torch.Tensor] = None, scratch: Optional[torch.Tensor] = None) -> None:
-    """`gemm_tc` with an RMSNorm folded in on either side (K splits inside clusters).
+                 out_xhat: Optional[torch.Tensor] = None, scratch: Optional[torch.Tensor] = None,
+                 bias: Optional[torch.Tensor] = None) -> None:
+    """`gemm_tc` with an RMSNorm folded in on either side (K splits inside clusters).  bias (float32 [N], not with
+    swiglu): added to every row after the norm's factor.
 
     in_ssq [M, ceil(K / 128)]: x is the bfloat16 copy of raw residual rows and w carries the norm's weight;
     every output row is multiplied by 1 / sqrt(sum(in_ssq[row]) / K + eps).  out_ssq [M, ceil(N / 128)] and
@@ -145,12 +147,14 @@ def gemm_tc_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
                 or out_xhat.dtype != torch.bfloat16 or not out_xhat.is_contiguous() or out_xhat.shape[-1] != N \
                 or out_ssq.numel() < M * ((N + 127) // 128) or out_xhat.numel() < M * N:
             raise KernelError("gemm_tc_norm: out_ssq is float32 [M, ceil(N / 128)], out_xhat bfloat16 [M, N]")
+    if bias is not None and (swiglu or bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != N):
+        raise KernelError("gemm_tc_norm: a bias is float32 [N] and does not go with the fused SwiGLU")
     st = status_word(x.device)
     kernel("gemm_tcgen05", "gg_gemm_tc_norm")(
         x.data_ptr(), w.data_ptr(), out.data_ptr(), mode, M, N, K, x.stride(0), out.stride(0),
         in_ssq.data_ptr() if in_ssq is not None else 0, in_parts, float(eps),
         out_ssq.data_ptr() if out_ssq is not None else 0, out_xhat.data_ptr() if out_xhat is not None else 0,
-        scratch.data_ptr() if scratch is not None else 0, scratch.numel() if scratch is not None else 0,
+        bias.data_ptr() if bias is not None else 0, scratch.data_ptr() if scratch is not None else 0, scratch.numel() if scratch is not None else 0,
         st.data_ptr(), torch.cuda.current_stream().cuda_stream)
 
 
@@ -194,7 +198,7 @@ def gemm_tc_qkv_rope(x: torch.Tensor, w: torch.Tensor, m: int, q_out: torch.Tens
 
 
 def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable]:
-    """A callable f(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None) for this
+    """A callable f(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None) for this
     weight, or None if its sizes are not taken (K must be a multiple of 8 so that rows start on 16-byte
     boundaries for TMA).  swiglu=True: the weight is interleaved gate/up (see `interleave_gate_up`) and
     out is [M, N / 2].  The keyword arguments are those of `gemm_tc_norm`; a call that has to fall back
@@ -207,13 +211,13 @@ def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable
 
     split_room: Dict[int, int] = {}      # tokens -> floats of scratch with which the prefill form splits K
 
-    def run(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None):
+    def run(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None):
         folded = in_ssq is not None or out_ssq is not None
         if x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
             if swiglu or folded:
                 raise KernelError("fused product: activations must be 16-byte aligned rows")
             from . import kernels as Kn
-            Kn.gemm_plain(x, weight, out, accumulate, m)
+            Kn.gemm_plain(x, weight, out, accumulate, m, bias=bias)
             return
         M = x.shape[0] if m is None else m
         scratch = None
@@ -223,8 +227,8 @@ def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable
                 need = split_room[M] = pair_scratch_elems(M, N, K)
             if need:
                 scratch = ws.get("gemm_partial_tiles", (need,), torch.float32)
-        if folded:
-            gemm_tc_norm(x, weight, out, accumulate, m, swiglu, in_ssq, eps, out_ssq, out_xhat, scratch)
+        if folded or bias is not None:
+            gemm_tc_norm(x, weight, out, accumulate, m, swiglu, in_ssq, eps, out_ssq, out_xhat, scratch, bias)
         else:
             gemm_tc(x, weight, out, accumulate, m, scratch, cluster=True, swiglu=swiglu)
 

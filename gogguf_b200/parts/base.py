@@ -110,7 +110,8 @@ class RowStats:
 
 
 class Linear:
-    """y = x W^T for a weight W[N, K]; float32 accumulation, optional add into a float32 output.
+    """y = x W^T (+ bias) for a weight W[N, K]; float32 accumulation, optional add into a float32 output.  The bias
+    [N] is kept in float32 and added to the float32 sums inside the product.
 
     The bfloat16 path uses the tcgen05 tensor-core kernel when the sizes allow it and the plain CUDA
     core kernel otherwise (and always in the 32-bit path and for a matrix stored in 32-bit).
@@ -119,7 +120,8 @@ class Linear:
     `emit=stats` asks an accumulating product to write the statistics of the rows it updates.
     """
 
-    def __init__(self, weight: torch.Tensor, rt: Runtime, swiglu: bool = False):
+    def __init__(self, weight: torch.Tensor, rt: Runtime, swiglu: bool = False,
+                 bias: Optional[torch.Tensor] = None):
         self.rt = rt
         self.weight = rt.matrix(weight)
         self.out_features, self.in_features = self.weight.shape
@@ -129,6 +131,9 @@ class Linear:
         if rt.fast and rt.dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16:
             from ..csrc import tcgen05_gemm
             self._fast = tcgen05_gemm.make_linear(self.weight, swiglu=swiglu)
+        self.bias = rt.vector(bias) if bias is not None else None
+        if self.bias is not None and (swiglu or self.bias.numel() != self.out_features):
+            raise ValueError("Linear: a bias has one number per output and does not go with the fused SwiGLU form")
         if swiglu and self._fast is None:
             raise ValueError("Linear: the fused SwiGLU form needs the tensor-core kernel")
 
@@ -182,6 +187,8 @@ class Linear:
             kw.update(out_ssq=emit.ssq, out_xhat=emit.xhat)
             emit.fresh = True
         if self._fast is not None and x.dtype == torch.bfloat16:
+            if self.bias is not None:
+                kw.update(bias=self.bias)
             self._fast(x, out, accumulate, m, ws, **kw)
         else:
-            K.gemm_plain(x, self.weight, out, accumulate, m)
+            K.gemm_plain(x, self.weight, out, accumulate, m, bias=self.bias)

@@ -36,7 +36,8 @@ class LinearHead:
     """logits = W h in float32; W is the embedding matrix when the spec says `tied_to`
     (pkg/model/qwen3/model.go:578-610, pkg/model/qwen3/tensors.go:36-48).  ``tensor`` of the spec names the
     stored matrix under the part's prefix (default "weight").  ``softcap`` (optional, c > 0): the logits are
-    bounded smoothly, c tanh(logits / c), in float32."""
+    bounded smoothly, c tanh(logits / c), in float32.  ``scale`` (default 1): a factor on the logits, in float32,
+    before any bound."""
 
     @classmethod
     def tensors(cls, spec: PartSpec) -> Dict[str, TensorDecl]:
@@ -48,6 +49,7 @@ class LinearHead:
         self.vocab = int(spec["vocab_size"])
         cap = spec.get("softcap")
         self.softcap = float(cap) if cap else 0.0
+        self.scale = float(spec.get("scale", 1.0))
         if self.softcap < 0.0:
             raise ValueError("head: softcap must be positive")
         if spec.get("tied_to") is not None:
@@ -59,6 +61,6 @@ class LinearHead:
 
     def forward(self, h: torch.Tensor, logits: torch.Tensor, ctx: StepContext, m: Optional[int] = None) -> None:
         self.proj(h, logits, m=m, ws=ctx.ws)
-        if self.softcap:
+        if self.softcap or self.scale != 1.0:
             rows = logits.shape[0] if m is None else m
-            K.softcap(logits, self.softcap, rows * self.vocab)
+            K.softcap(logits, self.softcap, rows * self.vocab, self.scale)

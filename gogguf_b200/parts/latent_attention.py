@@ -17,17 +17,21 @@ product and run attention in the ordinary per-head form, which costs a third of 
 compute the same sums, so a position's result does not depend on how its sequence was cut into steps beyond
 rounding.
 
-The rotation is the adjacent-pair kind (`rope_adjacent`), applied to the first `rotary_dim` elements of the
-rot part; `rope_dim` may be 0 (no rotated part, no position encoding: `position` is then left out).
+The rotation is applied to the first `rotary_dim` elements of the rot part; how its pairs are formed (adjacent
+elements or halves) is what the position encoding says in `pairing`.  `rope_dim` may be 0 (no rotated part, no
+position encoding: `position` is then left out).
 
-Two options.  `q_latent_dim` (Rq): the queries go through a latent of their own, c_q = N(W_dq h; w_q) (RMS norm with
+Three options.  `q_latent_dim` (Rq): the queries go through a latent of their own, c_q = N(W_dq h; w_q) (RMS norm with
 a plain weight, `latent_norm_eps`), q = W_uq c_q; W_dq and the key/value down projection run as one product.
 `sink`: a stored number per head whose exponential joins the softmax's denominator; it has no key and no value, is
-not scaled, and counts once.
+not scaled, and counts once.  `output_gate`: the concatenated heads are multiplied, element by element, by
+sigmoid(W_g h) before the output projection; W_g shares the first product, the multiplication happens in float32 where
+the heads' outputs are made.
 
 Spec parameters: hidden_size, num_heads, nope_dim, rope_dim, value_dim, latent_dim, scale, window,
-latent_norm_eps, position, q_latent_dim, sink, and optionally `names` (local tensor names of q, down, latent_norm,
-up_k, up_v, out; with a query latent q_down, q_latent_norm and q (the up projection); with a sink, sink).
+latent_norm_eps, position, q_latent_dim, sink, output_gate, and optionally `names` (local tensor names of q, down, latent_norm,
+up_k, up_v, out; with a query latent q_down, q_latent_norm and q (the up projection); with a sink, sink; with an
+output gate, gate).
 """
 from __future__ import annotations
 
@@ -46,7 +50,7 @@ PROMPT_FORM_MIN_TOKENS = 32      # whole prompts of at least this many tokens ta
 
 _NAMES = dict(q="q_proj.weight", down="kv_down_proj.weight", latent_norm="kv_norm.weight", up_k="k_up_proj.weight",
               up_v="v_up_proj.weight", out="o_proj.weight", q_down="q_down_proj.weight", q_latent_norm="q_norm.weight",
-              sink="sink")
+              sink="sink", gate="gate_proj.weight")
 
 
 def _names(spec: PartSpec) -> Dict[str, str]:
@@ -69,6 +73,8 @@ class LatentAttentionMixer:
             extra[n["q_latent_norm"]] = TensorDecl(shape=(Rq,), init="ones_normal")
         if spec.get("sink"):
             extra[n["sink"]] = TensorDecl(shape=(H,), init="small_normal")
+        if spec.get("output_gate"):
+            extra[n["gate"]] = TensorDecl(shape=(H * dv, W))
         return {
             **extra,
             n["q"]: TensorDecl(shape=(H * (d + r), Rq or W)),
@@ -93,11 +99,13 @@ class LatentAttentionMixer:
         self.eps = float(spec["latent_norm_eps"])
         self.position = None
         self.rot = 0
+        self.pairing = "adjacent"
         if self.r > 0:
             pos = dict(spec["position"])
             self.position = lookup(POSITIONS, pos["kind"], "position encoding")(pos, rt)
-            if getattr(self.position, "pairing", None) != "adjacent":
-                raise ValueError("latent attention rotates adjacent pairs; its position encoding must be of that kind")
+            self.pairing = getattr(self.position, "pairing", None)
+            if self.pairing not in ("adjacent", "halves"):
+                raise ValueError("latent attention rotates adjacent pairs or halves; its position encoding must say which")
             self.rot = int(pos.get("rotary_dim", self.r))
             if self.rot > self.r or self.rot % 2:
                 raise ValueError(f"latent attention: rotary_dim={self.rot} must be even and at most rope_dim={self.r}")
@@ -108,10 +116,15 @@ class LatentAttentionMixer:
         # from the normed query latent by a product of their own
         wq = rt.matrix(weights[n["q_down"] if self.Rq else n["q"]])
         wdown = rt.matrix(weights[n["down"]])
-        if wq.dtype != wdown.dtype:
-            wq, wdown = wq.float(), wdown.float()
-        # one product for the queries and the down projection: rows [all q heads | latent | shared key part]
-        self.q_down = Linear(torch.cat([wq, wdown], dim=0), rt)
+        first = [wq, wdown]
+        self.gated = bool(spec.get("output_gate"))
+        if self.gated:
+            first.append(rt.matrix(weights[n["gate"]]))
+        if len({w.dtype for w in first}) != 1:
+            first = [w.float() for w in first]
+        # one product for the queries and the down projection: rows [all q heads | latent | shared key part], then
+        # the output gate's
+        self.q_down = Linear(torch.cat(first, dim=0), rt)
         self.nq = self.Rq or H * (d + r)
         self.q_up = Linear(weights[n["q"]], rt) if self.Rq else None
         self.q_latent_norm = rt.vector(weights[n["q_latent_norm"]]) if self.Rq else None
@@ -126,13 +139,20 @@ class LatentAttentionMixer:
         self.kv_up = None
         if rt.fast and rt.dtype == torch.bfloat16 and self.uk_t.dtype == torch.bfloat16:
             from ..csrc import fast_latent
-            self._fast = fast_latent.try_make(H, d, R, r, H * (d + r) if self.Rq else self.nq + R + r, self.scale,
+            self._fast = fast_latent.try_make(H, d, R, r, H * (d + r) if self.Rq else self.q_down.out_features, self.scale,
                                               self.window, self.sink)
             # whole prompts: keys and values of all heads by one product, attention in the expanded form
             if (self._fast is not None and fast_latent.prompt_takes(d, r, dv) and R % 8 == 0 and (H * d) % 8 == 0
                     and (H * dv) % 8 == 0):
                 kv_up = Linear(torch.cat([rt.matrix(weights[n["up_k"]]), rt.matrix(weights[n["up_v"]])], dim=0), rt)
                 self.kv_up = kv_up if kv_up.tensor_core else None
+
+    def absorb_norm(self, norm) -> bool:
+        """Take the block's pre-norm into the first product; `forward` then gets RowStats as `h`."""
+        if not self.q_down.can_fold or norm.size != self.hidden:
+            return False
+        self.q_down.fold_input_norm(norm.weight, norm.eps)
+        return True
 
     def scale_output(self, mult: float) -> bool:
         """Multiply what this part adds to the residual by `mult`: the factor goes onto the heads' outputs in
@@ -151,10 +171,11 @@ class LatentAttentionMixer:
         # the tensor-core kernel takes bfloat16 queries; the plain kernels keep the absorbed query and the
         # latent output in float32 whatever the compute dtype
         mid = torch.bfloat16 if self._fast is not None else torch.float32
-        width = self.nq + R + r
+        width = self.q_down.out_features
         qd = ctx.ws.get("lat_q_down", (T, width), dt)
         self.q_down(h, qd, ws=ctx.ws)
-        dkv = qd[:, self.nq:]
+        dkv = qd[:, self.nq:self.nq + R + r]
+        gate = qd[:, self.nq + R + r:] if self.gated else None
         if self.Rq:
             # queries through their own latent: norm of the first Rq columns, then the up projection
             cq = ctx.ws.get("lat_q_latent", (T, self.Rq), dt)
@@ -173,16 +194,17 @@ class LatentAttentionMixer:
             ckr = ctx.ws.get("lat_rows_dense", (T, R + r), dt)
             K.latent_prep(qh, dkv, self.latent_norm, self.eps, cos, sin, self.rot,
                           ctx.positions, ctx.seq_of_token, table, cache.page_size,
-                          cache.pool if writes_cache else None, qcat, T, H, d, r, R, dense=ckr)
+                          cache.pool if writes_cache else None, qcat, T, H, d, r, R, dense=ckr,
+                          pairing=self.pairing)
             kv = ctx.ws.get("lat_keys_values", (T, H * (d + dv)), dt)
             self.kv_up(ckr[:, :R], kv, ws=ctx.ws)
             fast_latent.latent_prompt_mma(qd, qcat, kv, ckr, av, ctx.cu_seqlens, ctx.seq_of_token, ctx.n_seqs, T, H, d, r,
-                                          dv, R, self.scale, self.window, self.out_scale, self.sink)
+                                          dv, R, self.scale, self.window, self.out_scale, self.sink, gate)
             self.o(av, residual, accumulate=True, ws=ctx.ws)
             return
         K.latent_prep(qh, dkv, self.latent_norm, self.eps, cos, sin, self.rot,
                       ctx.positions, ctx.seq_of_token, table, cache.page_size, cache.pool if writes_cache else None,
-                      qcat, T, H, d, r, R)
+                      qcat, T, H, d, r, R, pairing=self.pairing)
         if self._fast is not None:
             self._fast.absorb(qd, width, d + r, self.uk_t, qcat, T)
         else:
@@ -194,7 +216,7 @@ class LatentAttentionMixer:
             K.latent_attention_plain(qcat, cache.pool, olat, ctx.positions, ctx.seq_of_token, table,
                                      cache.page_size, T, H, R, r, self.scale, self.window, self.sink)
         if self._fast is not None:
-            self._fast.expand(olat, self.uv, av, T, self.out_scale)
+            self._fast.expand(olat, self.uv, av, T, self.out_scale, gate)
         else:
-            K.headwise_gemm(olat, H * R, R, self.uv, av, H * dv, dv, T, alpha=self.out_scale)
+            K.headwise_gemm(olat, H * R, R, self.uv, av, H * dv, dv, T, alpha=self.out_scale, gate=gate)
         self.o(av, residual, accumulate=True, ws=ctx.ws)

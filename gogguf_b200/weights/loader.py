@@ -42,7 +42,8 @@ class TensorDecl:
 
     init: "normal" (N(0, std)), "ones_normal" (1 + N(0, norm_std)), "zeros_normal" (N(0, norm_std)),
     "small_normal" (N(0, 0.5)), "unit_interval" (sigmoid of N(0, 1): numbers inside (0, 1)), "mean" ((1 + N(0,
-    norm_std)) / n for a vector of n: the coefficients of an average) or "zeros";
+    norm_std)) / n for a vector of n: the coefficients of an average), "near_identity" (a square matrix: the identity
+    plus N(0, 1 / n) elements), "half" (0.5 + N(0, norm_std)) or "zeros";
     used only by the random-weights mode.  optional: may be absent (for
     instance a separate head matrix of a model with tied embeddings).
     """
@@ -167,6 +168,10 @@ def random_tensors(expected: Mapping[str, TensorDecl], seed: int, std: float, no
                 t.sigmoid_()
             elif d.init == "mean":               # coefficients of an average
                 t.mul_(norm_std).add_(1.0).div_(float(d.shape[-1]))
+            elif d.init == "near_identity":      # a mixing matrix of heads
+                t.div_(float(d.shape[-1])).add_(torch.eye(d.shape[-1], device=dev))
+            elif d.init == "half":               # the share of a mix
+                t.mul_(norm_std).add_(0.5)
             else:
                 raise ValueError(f"tensor {name!r}: unknown init {d.init!r}")
         out[name] = t.to(dtype)
