@@ -506,9 +506,9 @@ __global__ void __launch_bounds__(MC_WARPS * 32) mixed_head_combine_kernel(
     const float* __restrict__ talk, const int* __restrict__ seq_of_token, int H, int G, int dv, int nsplit, float one) {
     pdl_launch();
     pdl_wait();
-    extern __shared__ float mc_sm[];
-    float* f = mc_sm;                                   // [H][nsplit]: share z's factor for head g
-    float* red = f + H * nsplit;                        // [MC_WARPS][4][128]
+    extern __shared__ __align__(16) float mc_sm[];
+    float* red = mc_sm;                                 // [MC_WARPS][4][128] (first: it is written 16 bytes at a time)
+    float* f = red + MC_WARPS * 4 * 128;                // [H][nsplit]: share z's factor for head g
     const int t = blockIdx.x, gv = blockIdx.y, hpg = H / G;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     bf16* o = out + (size_t)t * ldo + (size_t)gv * hpg * dv;
