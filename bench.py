@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L] [--impl ours|reference]
                     [--shape 8b|14b|32b] [--workload] [--prefill-lengths 256,1024] [--decode-contexts 16384,32768]
-    python bench.py --compare gigopel|sokirax|felolorn|dinuzen [--compare-sizes 2k,4k]   (another workload, see the end of this text)
+    python bench.py --compare gigopel|sokirax|felolorn|dinuzen|kulesun [--compare-sizes 2k,4k]   (another workload, see the end of this text)
 
 A "step" is one decode step of a batch: every sequence goes on by one token, sampled greedily on the
 device.  The timed region is exactly K steps after W warm-up steps, timed with CUDA events on the
@@ -46,6 +46,12 @@ unit, Mamba-2; routed experts with identity experts and a gated shared expert): 
 layers cycle through attention, RG-LRU, Mamba-2 and attention on borrowed keys, beside the all-experts Felolorn model
 (its closest relative: norms after the parts, recurrences behind short convolutions, routed experts with a
 correction) and the same Qwen3.  It prints {"compare": "dinuzen", "sizes": {...}}.
+
+`--compare kulesun` measures the Kulesun design (norms on both sides of every part; latent attention with a gate on
+the heads' outputs, and attention whose heads' weights are mixed; gated dense feed-forwards): one model per size whose
+layers cycle through two latent layers and one attention layer, beside the dense Sokirax model (the same arrangement
+of norms and the same feed-forward around other mixers), the dense Gigopel model (latent attention of the same sizes)
+and the same Qwen3.  It prints {"compare": "kulesun", "sizes": {...}}.
 
 Peaks come from MEASURED_PEAKS.json beside this file when the driver wrote it, else from the
 fallback figures of an earlier measurement on this pool.  The weights (16 GB) are far larger than
@@ -290,6 +296,30 @@ def dinuzen_config(z):
                 initializer_range=0.02, layers=layers)
 
 
+# Kulesun at the same widths and depths: Gigopel's latent sizes (without a window), attention heads of 128 as Dinuzen's,
+# Sokirax's dense feed-forward
+KULESUN_SIZES = {
+    "2k": dict(width=2048, heads=16, dim=64, rot_dim=32, vdim=64, kv_rank=256, att_heads=16, att_kv_heads=4, att_dim=128,
+               ff=8192, layers=8, vocab=65536),
+    "4k": dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, att_heads=32, att_kv_heads=8, att_dim=128,
+               ff=16384, layers=8, vocab=65536),
+}
+
+
+def kulesun_config(z):
+    """Layers cycle through latent attention, latent attention and attention with mixed heads."""
+    lat = dict(heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["vdim"], kv_rank=z["kv_rank"],
+               scale=(z["dim"] + z["rot_dim"]) ** -0.5,
+               rot=dict(base=500000.0, dims=z["rot_dim"], scaling=dict(factor=4.0, original=8192, fast=16.0, slow=2.0)))
+    att = dict(heads=z["att_heads"], kv_heads=z["att_kv_heads"], dim=z["att_dim"], vdim=z["att_dim"], scale=z["att_dim"] ** -0.5,
+               softcap=30.0, v_mix=True, q_temp=dict(coef=0.1, every=4096))
+    mlp = dict(kind="dense", ff=(2 * z["ff"] // 3) // 128 * 128)
+    return dict(architecture="Kulesun", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), initializer_range=0.02,
+                embedding=dict(scale=z["width"] ** 0.5), logit_scale=0.5,
+                layers=[dict(type="attention", mixer=att, mlp=mlp) if i % 3 == 2 else dict(type="latent_attention", mixer=lat, mlp=mlp)
+                        for i in range(z["layers"])])
+
+
 def qwen3_like(z):
     """Qwen3 at the same width, depth, head count and feed-forward parameter count (3 matrices instead of 2), with
     full attention (its cache of a 2,048-token context is read whole; Gigopel reads its window)."""
@@ -440,12 +470,34 @@ def compare_run(a):
         per_seq = (n[0] + n[3]) * t * G * (2 * d + dv) * 2 + n[2] * 2 * inner * z["ssm_state"] * 4 + n[1] * 2 * W * 4
         return flops, wbytes, per_seq
 
+    def kul_numbers(z, t):
+        """The same figures for a Kulesun model whose layers cycle through two latent layers and an attention layer.
+        Attention's own arithmetic is counted as the definition has it: a score product and a value product per head, and
+        the mixing of the heads' weights at every key left out."""
+        W, H, d, r, dv, R = z["width"], z["heads"], z["dim"], z["rot_dim"], z["vdim"], z["kv_rank"]
+        AH, AG, ad = z["att_heads"], z["att_kv_heads"], z["att_dim"]
+        n_att = len(range(2, z["layers"], 3))
+        n_lat = z["layers"] - n_att
+        lat = H * (d + r) * W + (R + r) * W + H * (d + dv) * R + 2 * W * H * dv
+        att = (AH + 2 * AG) * ad * W + AH * W + W * AH * ad
+        ff = 3 * W * ((2 * z["ff"] // 3) // 128 * 128)
+        keys = t * (t + 1) // 2
+        flops = 2 * t * (n_lat * lat + n_att * att + z["layers"] * ff) + 2 * z["vocab"] * W
+        flops += keys * (n_lat * 2 * H * (d + r + dv) + n_att * 2 * 2 * AH * ad)
+        wbytes = (n_lat * lat + n_att * att + z["layers"] * ff) * 2 + z["vocab"] * W * 2
+        per_seq = t * 2 * (n_lat * (R + r) + n_att * 2 * AG * ad)
+        return flops, wbytes, per_seq
+
     out = {}
     T = PROMPT_LEN
     design = a.compare
     for name in [x for x in a.compare_sizes.split(",") if x.strip()]:
         z = GIGOPEL_SIZES[name]
-        if design == "dinuzen":
+        if design == "kulesun":
+            zs, zk = SOKIRAX_SIZES[name], KULESUN_SIZES[name]
+            arms = [("kulesun_dense", kulesun_config(zk)), ("sokirax_dense", sokirax_config(zs, "dense")),
+                    ("gigopel_dense", gigopel_config(z, "dense")), ("qwen3_like", qwen3_like(z))]
+        elif design == "dinuzen":
             zs, zf, zd = SOKIRAX_SIZES[name], FELOLORN_SIZES[name], DINUZEN_SIZES[name]
             arms = [("dinuzen_experts", dinuzen_config(zd)), ("felolorn_experts", felolorn_config(zf)),
                     ("qwen3_like", qwen3_like(z))]
@@ -468,11 +520,16 @@ def compare_run(a):
             per_seq = 0
             if arm == "qwen3_like":
                 flops, wbytes = qwen_numbers(cd, z, T)
+            elif arm == "kulesun_dense":
+                flops, wbytes, per_seq = kul_numbers(zk, T)
+            elif arm == "gigopel_dense" and design == "kulesun":
+                flops, wbytes = gig_numbers(z, "dense", T)
+                per_seq = min(T, z["window"]) * z["layers"] * (z["kv_rank"] + z["rot_dim"]) * 2
             elif arm == "dinuzen_experts":
                 flops, wbytes, per_seq = din_numbers(zd, T)
             elif arm == "felolorn_experts":
                 flops, wbytes, per_seq = fel_numbers(zf, T)
-            elif design in ("sokirax", "felolorn"):
+            elif design in ("sokirax", "felolorn", "kulesun"):
                 flops, wbytes, per_seq = sok_numbers(zs, "dense" if arm.endswith("dense") else "moe", T)
             else:
                 flops, wbytes = gig_numbers(z, "dense" if arm.endswith("dense") else "moe", T)
@@ -490,7 +547,7 @@ def compare_run(a):
                     rb -= z["layers"] * (z["experts"] - used) * 3 * z["width"] * z["expert_ff"] * 2
                 if arm == "qwen3_like":
                     rb += b * T * 2 * z["layers"] * 8 * 128 * 2
-                elif design in ("sokirax", "felolorn", "dinuzen"):
+                elif design in ("sokirax", "felolorn", "dinuzen", "kulesun"):
                     rb += b * per_seq
                 else:
                     rb += b * min(T, z["window"]) * z["layers"] * (z["kv_rank"] + z["rot_dim"]) * 2
@@ -529,7 +586,7 @@ def main():
                     "decode_by_context)")
     ap.add_argument("--prefill-lengths", default="", help="comma separated prompt lengths: time one prefill step of each "
                     "(printed on stderr, added to the line as prefill_sweep)")
-    ap.add_argument("--compare", default="", choices=["", "gigopel", "sokirax", "felolorn", "dinuzen"],
+    ap.add_argument("--compare", default="", choices=["", "gigopel", "sokirax", "felolorn", "dinuzen", "kulesun"],
                     help="another workload: the named design beside Qwen3 at equal size (prefill and decode), see the top")
     ap.add_argument("--compare-sizes", default="2k,4k", help="which of the comparison's layer sizes to run")
     a = ap.parse_args()

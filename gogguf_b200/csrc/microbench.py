@@ -529,9 +529,83 @@ def dinuzen(sizes=((16, 4, 64, 128, 2048, 32, 64, 128, 8), (32, 8, 128, 128, 409
         torch.cuda.empty_cache()
 
 
+def kulesun(sizes=((16, 4, 128, 128, 2048), (32, 8, 128, 128, 4096))) -> None:
+    """The kernels the Kulesun design added, at layer sizes (heads, kv heads, d, dv, width): attention with mixed heads
+    (csrc/mixed_head_attention.cu) on a prompt of 2,048 tokens against the bf16 tensor peak (two products per head, as
+    the definition has it) and in decode steps against the copy bandwidth; the writer of keys and values; the products
+    with a bias."""
+    from . import kernels as K
+    from . import tcgen05_gemm as TG
+    dev = "cuda:0"
+    hbm, tflops, src = _peaks()
+    print(f"peaks ({src}): {hbm:.0f} GB/s copy, {tflops:.0f} TFLOP/s bf16")
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    for H, G, d, dv, W in sizes:
+        T, ps = 2048, 64
+        pages = T // ps
+        kpool = (torch.randn(pages * 64, G, ps, d, device=dev) * 0.5).to(torch.bfloat16)
+        vpool = torch.randn(pages * 64, G, ps, dv, device=dev).to(torch.bfloat16)
+        width = (H + G) * d + G * dv + H
+        row = torch.randn(T, width, device=dev).to(torch.bfloat16)
+        o = torch.empty(T, H * dv, device=dev, dtype=torch.bfloat16)
+        talk = torch.eye(H, device=dev) + torch.randn(H, H, device=dev) / H
+        pos, sot = i32(list(range(T))), i32([0] * T)
+        table = i32([list(range(pages))])
+        kw = dict(cap=30.0, coef=0.1, every=4096.0, one=True)
+        run = mixed_head_runner(H, G, d, dv, width - H, talk, kw, ps)
+        for n in (256, 2048):
+            cu = i32([0, n])
+            us = _time_graph(lambda i: run(row[:n], kpool, vpool, o[:n], pos[:n], sot[:n], cu, table, n, 1, n, n), reps=10)
+            flops = 2 * H * (d + dv) * (n * (n + 1) // 2)
+            print(f"mixed-head attention prompt  H={H} G={G} d={d} dv={dv} T={n}: {us:8.1f} us  {flops / us / 1e6:6.1f} TFLOP/s "
+                  f"({flops / us / 1e6 / tflops:.3f} of the bf16 peak)", flush=True)
+        for B in (8, 64):
+            tb = i32([[(b * pages + j) for j in range(pages)] for b in range(B)])
+            posb, sotb, cub = i32([T - 1] * B), i32(list(range(B))), i32(list(range(B + 1)))
+            us = _time_graph(lambda i: run(row[:B], kpool, vpool, o[:B], posb, sotb, cub, tb, B, B, 1, T))
+            nbytes = B * T * G * (d + dv) * 2
+            print(f"mixed-head attention decode  batch {B:2d} ctx {T}: {us:8.1f} us  {nbytes / us / 1e3:7.1f} GB/s "
+                  f"({nbytes / us / 1e3 / hbm:.2f} of the copy bandwidth)", flush=True)
+        first = torch.randn(T, G * dv, device=dev)
+        us = _time_graph(lambda i: K.head_kv_prep(row, H * d, (H + G) * d, kpool, vpool, pos, sot, table, ps, T, G, d, dv, True, 1e-6,
+                                                  first, 0.3), reps=10)
+        nbytes = T * G * ((d + dv) * 4 + dv * 4)
+        print(f"keys and values into the cache T={T}: {us:6.1f} us  {nbytes / us / 1e3 / hbm:.2f} of the copy bandwidth", flush=True)
+        us = _time_graph(lambda i: K.head_kv_prep(row[:8], H * d, (H + G) * d, kpool, vpool, pos, sot, table, ps, 8, G, d, dv, True, 1e-6,
+                                                  first, 0.3))
+        print(f"keys and values into the cache, 8 rows: {us:6.1f} us", flush=True)
+        # ---- a product with and without a bias
+        w = (torch.randn(W, W, device=dev) * 0.02).to(torch.bfloat16)
+        b = torch.randn(W, device=dev)
+        for m in (8, T):
+            x = torch.randn(m, W, device=dev).to(torch.bfloat16)
+            y = torch.zeros(m, W, device=dev)
+            t = [_time_graph(lambda i: TG.gemm_tc_norm(x, w, y, accumulate=True, bias=bb)) for bb in (None, b)]
+            print(f"product {W} x {W}, {m} rows, added into float32: {t[0]:6.1f} us, with a bias {t[1]:6.1f} us", flush=True)
+        del kpool, vpool
+        torch.cuda.empty_cache()
+
+
+def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps):
+    """A callable that runs attention with mixed heads as the mixer would for a step of those sizes; scratch is made on
+    the first call of a size, so that the calls can be captured."""
+    from . import kernels as K
+    scratch = {}
+
+    def run(row, kpool, vpool, o, pos, sot, cu, table, T, n_seqs, max_new, max_ctx):
+        ns = K.mixed_head_splits(T, n_seqs, H, G, max_ctx) if max_new <= 4 else 1
+        if T not in scratch:
+            scratch[T] = (torch.empty(T * H * ns * G * dv, device=row.device), torch.empty(T * H * ns * 2, device=row.device))
+        u, ml = scratch[T]
+        K.mixed_head_attention_mma(row, g_off, kpool, vpool, o, talk, pos, sot, cu, table, ps, T, n_seqs, H, G, d, dv, d ** -0.5, u, ml,
+                                   nsplit=ns, max_new=max_new, **kw)
+
+    return run
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "gemm_layer", "attn", "prefill_attn", "sample", "latent", "retention", "recurrence", "dinuzen"])
+    ap.add_argument("what", choices=["gemm", "gemm_layer", "attn", "prefill_attn", "sample", "latent", "retention", "recurrence", "dinuzen", "kulesun"])
     ap.add_argument("--m", default="1,8,64", help="token counts (gemm), batch sizes (attn) or prompt lengths (prefill_attn)")
     ap.add_argument("--ctx", default="2048", help="attn: cached positions per sequence (comma separated)")
     ap.add_argument("--scratch", action="store_true", help="attn: splits merged by a second kernel instead of inside clusters")
@@ -546,8 +620,8 @@ def main() -> None:
     if a.what == "recurrence":
         recurrence()
         return
-    if a.what == "dinuzen":
-        dinuzen()
+    if a.what in ("dinuzen", "kulesun"):
+        {"dinuzen": dinuzen, "kulesun": kulesun}[a.what]()
         return
     if a.what == "attn":
         for c in a.ctx.split(","):

@@ -9,7 +9,8 @@ import torch
 
 import plain_kulesun as plain
 from helpers import random_tokens, read_folder, rel_err
-from kulesun_cases import CASES, attn, draw_case, latent, layer, make_folder, model, plain_logits, rot, write_case
+from kulesun_cases import (CASES, attn, draw_case, latent, layer, make_folder, model, plain_logits, rot, rounded_logits,
+                           write_case)
 from test_gpu_felolorn import close, load, run_cut
 
 pytestmark = pytest.mark.gpu
