@@ -61,6 +61,7 @@ MODULES: Dict[str, str] = {
     "diag_recurrence": "diag_recurrence.cu",
     "diff_attention": "diff_attention.cu",
     "mixed_head_attention": "mixed_head_attention.cu",
+    "mixed_head_prompt": "mixed_head_prompt.cu",
     "sampling": "sampling.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",
     "attention_fast": "attention_fast.cu",
@@ -72,6 +73,7 @@ _HEADERS = ["common.cuh"]
 # further files a module's source includes (they take part in its hash)
 _INCLUDES: Dict[str, List[str]] = {
     "attention_fast.cu": ["tma_util.cuh"],
+    "mixed_head_prompt.cu": ["tma_util.cuh"],
     "gemm_tcgen05.cu": ["tma_util.cuh"],
     "gemm_tcgen05_static.cu": ["gemm_tcgen05.cu", "gemm_tcgen05_static.h", "tma_util.cuh"],
     "diagnostics.cu": ["tma_util.cuh"],

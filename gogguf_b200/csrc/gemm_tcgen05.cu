@@ -327,7 +327,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
         return;
     }
     float ss = 0.f;          // running sum of squares of the updated row over 128 columns
-    if (out_mode == OUT_F32_ACC && tn * BN + BN <= N && ((((uintptr_t)out) | ((uintptr_t)nio.out_xhat)) & 15) == 0 &&
+    if (out_mode == OUT_F32_ACC && tn * BN + BN <= N && ((((uintptr_t)out) | ((uintptr_t)nio.out_xhat) | ((uintptr_t)nio.bias)) & 15) == 0 &&
         (ldo & 3) == 0 && (N & 7) == 0) {
         // Adding into the residual reads what is there: one thread's 16 columns at a time, every group would
         // wait a whole trip to L2 for its 64 bytes (about 20 us per tile, in the open after a product's last
@@ -347,6 +347,14 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
             uint32_t r[64];
 #pragma unroll
             for (int q = 0; q < 4; ++q) tmem_ld16(taddr + (uint32_t)(c0 + 16 * q), r + 16 * q);
+            if (nio.bias != nullptr && live) {           // the same 64 numbers for every row: from L1
+                const float4* bp = reinterpret_cast<const float4*>(nio.bias + tn * BN + c0);
+#pragma unroll
+                for (int j = 0; j < 16; ++j) {
+                    const float4 b = __ldg(bp + j);
+                    old[j].x += b.x; old[j].y += b.y; old[j].z += b.z; old[j].w += b.w;
+                }
+            }
             tmem_ld_wait();
             if (!live) continue;
 #pragma unroll
@@ -358,7 +366,6 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
                     float4 v = make_float4(__uint_as_float(r[16 * q + 4 * j]), __uint_as_float(r[16 * q + 4 * j + 1]),
                                            __uint_as_float(r[16 * q + 4 * j + 2]), __uint_as_float(r[16 * q + 4 * j + 3]));
                     if (scaled) { v.x *= sc; v.y *= sc; v.z *= sc; v.w *= sc; }
-                    if (nio.bias != nullptr) add_bias<4>(&v.x, nio.bias, tn * BN + c0 + 16 * q + 4 * j, N);
                     v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
                     reinterpret_cast<float4*>(orow + c0 + 16 * q)[j] = v;
                     if (stats) {

@@ -546,6 +546,40 @@ def mixed_head_attention_mma(row: torch.Tensor, g_off: int, k_pool: torch.Tensor
         _stream())
 
 
+def mixed_head_prompt_takes(heads: int, kv_heads: int, d: int, dv: int, page_size: int) -> bool:
+    """Does the tcgen05 form of attention with mixed heads take these sizes (bfloat16 tensors)?"""
+    from .build import module
+    return bool(module("mixed_head_prompt").lib.gg_mixed_head_prompt_takes(int(heads), int(kv_heads), int(d), int(dv),
+                                                                          int(page_size)))
+
+
+def mixed_head_attention_prompt(row: torch.Tensor, g_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
+                                talk: torch.Tensor, seq_of_token: torch.Tensor, cu_seqlens: torch.Tensor, ctx_lens: torch.Tensor,
+                                page_table: torch.Tensor, page_size: int, n_tokens: int, n_seqs: int, heads: int, kv_heads: int,
+                                d: int, dv: int, scale: float, u: torch.Tensor, ml: torch.Tensor, cap: float = 0.0,
+                                coef: float = 0.0, every: float = 1.0, one: bool = False, window: int = 0,
+                                value_heads: Optional[int] = None) -> None:
+    """`mixed_head_attention_mma` for prompts, on the tcgen05 tensor cores (128 query rows of a head per CTA).
+    value_heads: kv heads' values per CTA, 1 or 2 (default: 2 where there are several)."""
+    _mixed_head_check(row, k_pool, v_pool, out, talk, heads, kv_heads, d, dv, g_off)
+    _need(row, torch.bfloat16, "row")
+    _need(u, torch.float32, "u")
+    _need(ml, torch.float32, "ml")
+    if u.numel() < n_tokens * heads * kv_heads * dv or ml.numel() < n_tokens * heads * 2:
+        raise KernelError("mixed_head_attention_prompt: the scratch is too small")
+    if value_heads is None:
+        value_heads = 2 if kv_heads > 1 else 1
+    from .tcgen05_gemm import status_word
+    kernel("mixed_head_prompt", "gg_mixed_head_prompt")(
+        _p(row), row.stride(0), _p(k_pool), _p(v_pool), _p(u), _p(ml), _p(cu_seqlens), _p(ctx_lens), _p(seq_of_token),
+        _p(page_table), page_table.shape[-1], int(page_size), k_pool.shape[0], int(n_tokens), int(n_seqs),
+        n_tokens // 128 + n_seqs, int(heads), int(kv_heads), int(d), int(dv), float(scale), float(cap), float(coef), float(every),
+        int(window), int(value_heads), _p(status_word(row.device)), _stream())
+    kernel("mixed_head_attention", "gg_mixed_head_combine")(
+        _p(u), _p(ml), _p(row), row.stride(0), int(g_off), _p(out), out.stride(0), _p(talk), _p(seq_of_token), int(n_tokens),
+        int(heads), int(kv_heads), int(dv), 1, float(bool(one)), _stream())
+
+
 def diff_attention_partial_elems(n_tokens: int, heads: int, dv: int, nsplit: int) -> int:
     return n_tokens * heads * nsplit * 2 * (2 + dv)
 

@@ -549,10 +549,13 @@ def kulesun(sizes=((16, 4, 128, 128, 2048), (32, 8, 128, 128, 4096))) -> None:
         row = torch.randn(T, width, device=dev).to(torch.bfloat16)
         o = torch.empty(T, H * dv, device=dev, dtype=torch.bfloat16)
         talk = torch.eye(H, device=dev) + torch.randn(H, H, device=dev) / H
-        pos, sot = i32(list(range(T))), i32([0] * T)
+        pos, sot, i32_t = i32(list(range(T))), i32([0] * T), i32([0, T])
         table = i32([list(range(pages))])
         kw = dict(cap=30.0, coef=0.1, every=4096.0, one=True)
         run = mixed_head_runner(H, G, d, dv, width - H, talk, kw, ps)
+        one_head = mixed_head_runner(H, G, d, dv, width - H, talk, kw, ps, value_heads=1)
+        us = _time_graph(lambda i: one_head(row, kpool, vpool, o, pos, sot, i32_t, table, T, 1, T, T), reps=10)
+        print(f"   (one kv head's values per CTA, T={T}: {us:8.1f} us)", flush=True)
         for n in (256, 2048):
             cu = i32([0, n])
             us = _time_graph(lambda i: run(row[:n], kpool, vpool, o[:n], pos[:n], sot[:n], cu, table, n, 1, n, n), reps=10)
@@ -586,14 +589,22 @@ def kulesun(sizes=((16, 4, 128, 128, 2048), (32, 8, 128, 128, 4096))) -> None:
         torch.cuda.empty_cache()
 
 
-def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps):
+def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps, value_heads=None):
     """A callable that runs attention with mixed heads as the mixer would for a step of those sizes; scratch is made on
     the first call of a size, so that the calls can be captured."""
     from . import kernels as K
     scratch = {}
 
     def run(row, kpool, vpool, o, pos, sot, cu, table, T, n_seqs, max_new, max_ctx):
-        ns = K.mixed_head_splits(T, n_seqs, H, G, max_ctx) if max_new <= 4 else 1
+        if max_new > 4:
+            if T not in scratch:
+                scratch[T] = (torch.empty(T * H * G * dv, device=row.device), torch.empty(T * H * 2, device=row.device),
+                              torch.tensor([max_ctx], dtype=torch.int32, device=row.device))
+            u, ml, ends = scratch[T]
+            K.mixed_head_attention_prompt(row, g_off, kpool, vpool, o, talk, sot, cu, ends, table, ps, T, n_seqs, H, G, d, dv, d ** -0.5,
+                                          u, ml, value_heads=value_heads, **kw)
+            return
+        ns = K.mixed_head_splits(T, n_seqs, H, G, max_ctx)
         if T not in scratch:
             scratch[T] = (torch.empty(T * H * ns * G * dv, device=row.device), torch.empty(T * H * ns * 2, device=row.device))
         u, ml = scratch[T]

@@ -569,6 +569,23 @@ GG_API gg_mixed_head_mma_takes(int H, int G, int d, int dv, int page_size) {
             H % G == 0 && H / G <= MH_ROWS && H <= 512 && G <= 4096) ? 1 : 0;
 }
 
+// u [ntok][H][nsplit][G][dv] and ml [ntok][H][nsplit][2] (float32: unnormalised results of the shares of the keys on every
+// kv head's values, their references in log2 units and sums) -> out [ntok, H dv] (bfloat16, row stride ldo): the shares put
+// together, divided by the softmax's sum (with `one` joining it), the heads mixed by talk [H][H], gated by the logits at
+// row + t ld + g_off (g_off negative: no gate).
+GG_API gg_mixed_head_combine(const float* u, const float* ml, const void* row, long long ld, int g_off, void* out, long long ldo,
+                             const float* talk, const int* seq_of_token, int ntok, int H, int G, int dv, int nsplit, float one,
+                             cudaStream_t stream) {
+    if (ntok <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || dv <= 0 || dv > 128 || dv % 4 || nsplit < 1 || ldo < (long long)H * dv || (((uintptr_t)u) & 15))
+        return GG_ERR_ARG;
+    const size_t smem = ((size_t)H * nsplit + MC_WARPS * 4 * 128) * sizeof(float);
+    if (smem > 220 * 1024) return GG_ERR_ARG;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_combine_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return gg_launch(mixed_head_combine_kernel, dim3(ntok, G), dim3(MC_WARPS * 32), smem, stream, 1, u, ml, (const bf16*)row, ld,
+                     g_off, (bf16*)out, ldo, talk, seq_of_token, H, G, dv, nsplit, one);
+}
+
 template <int D, int DV, int NV, bool WK>
 static int mh_launch(const bf16* row, long long ld, const bf16* k_pool, const bf16* v_pool, float* u, float* ml,
                      const int* positions, const int* seq_of_token, const int* cu_seqlens, const int* page_table,
@@ -618,10 +635,7 @@ GG_API gg_mixed_head_attention_mma(const void* row, long long ld, int g_off, con
 #undef MH_GO
 #undef MH_ARGS
     if (rc != 0) return rc;
-    const size_t smem = ((size_t)H * nsplit + MC_WARPS * 4 * 128) * sizeof(float);
-    if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_combine_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return gg_launch(mixed_head_combine_kernel, dim3(ntok, G), dim3(MC_WARPS * 32), smem, stream, 1, (const float*)u,
-                     (const float*)ml, (const bf16*)row, ld, g_off, (bf16*)out, ldo, talk, seq_of_token, H, G, dv, nsplit, one);
+    return gg_mixed_head_combine(u, ml, row, ld, g_off, out, ldo, talk, seq_of_token, ntok, H, G, dv, nsplit, one, stream);
 }
 
 // 1 if this library was built with checked page tables (the debug build), else 0.

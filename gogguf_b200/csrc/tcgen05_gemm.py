@@ -38,7 +38,8 @@ def check_status(device: torch.device) -> None:
             raise KernelError(f"debug build: kernel {who} met a page-table index or page id out of range (code {v}); "
                               "it read page 0 (a reader) or wrote nothing (a writer), results of that step are invalid")
         raise KernelError(f"a bounded wait inside a kernel ran out (code {v}: 1 TMA producer, 2 MMA issuer, "
-                          "3 epilogue of a product, 11-12 decode attention, 21-28 prefill attention); "
+                          "3 epilogue of a product, 11-12 decode attention, 21-28 prefill attention, 61-68 prefill attention "
+                          "with mixed heads); "
                           "results of that step are invalid")
 
 

@@ -19,7 +19,7 @@ values are the ones later layers mix in, "mix"), extra_one, talking (False: T is
 head_gate, window (absent: none), names.
 
 Temperature, scores, softmax, mixing and gate are float32 in both compute paths.  In the bfloat16 path head sizes of up
-to 128 run on the tensor cores; GOGGUF_B200_MIXED_HEAD_MMA=0 keeps the plain kernel, their twin.
+to 128 run on the tensor cores (prompts on tcgen05, short stretches and decode steps on mma.sync); GOGGUF_B200_MIXED_HEAD_MMA=0 keeps the plain kernel, their twin.
 """
 from __future__ import annotations
 
@@ -35,6 +35,8 @@ from ..csrc import kernels as K
 from ..weights.loader import TensorDecl
 from .base import Linear, Runtime, StepContext
 from .registry import register_mixer
+
+PROMPT_FORM_MIN_TOKENS = 48      # steps whose longest stretch of new tokens has at least this many take the tcgen05 form
 
 FIRST_VALUES = "mixed_head_first_values"      # workspace: the source layer's values of the step's tokens
 
@@ -143,7 +145,13 @@ class MixedHeadAttentionMixer:
                        cache.page_size, T, G, d, dv, self.unit, self.eps, first, self.lam, keep)
         o = ctx.ws.get("mixed_head_out", (T, H * dv), self.rt.dtype)
         kw = dict(cap=self.cap, coef=self.coef, every=self.every, one=self.one, window=self.window)
-        if self._mma and K.mixed_head_mma_takes(H, G, d, dv, cache.page_size):
+        if (self._mma and ctx.max_new >= PROMPT_FORM_MIN_TOKENS
+                and K.mixed_head_prompt_takes(H, G, d, dv, cache.page_size)):
+            u = ctx.ws.get("mixed_head_u", (T * H * G * dv,), torch.float32)
+            ml = ctx.ws.get("mixed_head_ml", (T * H * 2,), torch.float32)
+            K.mixed_head_attention_prompt(row, self.g_off, cache.k, cache.v, o, self.talk, ctx.seq_of_token, ctx.cu_seqlens,
+                                          ctx.ctx_lens, table, cache.page_size, T, ctx.n_seqs, H, G, d, dv, self.scale, u, ml, **kw)
+        elif self._mma and K.mixed_head_mma_takes(H, G, d, dv, cache.page_size):
             # steps of few rows over long contexts (decode steps): the key tiles are shared out over several CTAs
             nsplit = K.mixed_head_splits(T, ctx.n_seqs, H, G, int(ctx.max_ctx)) if ctx.max_new <= 4 else 1
             u = ctx.ws.get("mixed_head_u", (T * H * nsplit * G * dv,), torch.float32)

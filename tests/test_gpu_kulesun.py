@@ -141,6 +141,44 @@ def _mixed_reference(q, k, v, gate, talk, pos, lens, scale, cap, coef, every, on
     return torch.stack(out)
 
 
+def _prompt_form(K, row, g_off, kf, vf, talk, pos, lens, sot, cu, table, H, G, d, dv, scale, want, nv, kw, tol=1.2e-2):
+    """The tcgen05 form on a step of stretches `lens` against the wanted rows."""
+    T, ends = len(pos), []
+    for n in lens:
+        ends.append(pos[sum(lens[:len(ends) + 1]) - 1] + 1)
+    o = torch.empty(T, H * dv, dtype=torch.bfloat16, device=DEV)
+    u = torch.full((T * H * G * dv,), 1e30, device=DEV)
+    ml = torch.full((T * H * 2,), 1e30, device=DEV)
+    K.mixed_head_attention_prompt(row.to(DEV), g_off, kf.to(DEV), vf.to(DEV), o, talk.to(DEV), sot, cu, _i32(ends), table, PS, T,
+                                  len(lens), H, G, d, dv, scale, u, ml, value_heads=nv, **kw)
+    from gogguf_b200.csrc.tcgen05_gemm import check_status
+    check_status(torch.device(DEV))
+    assert rel_err(o, want) < tol, ("prompt form", lens, nv, rel_err(o, want))
+
+
+@pytest.mark.parametrize("cap,factor", [(0.0, 1.0), (0.0, 30.0), (60.0, 12.0), (30.0, 1.0), (30.0, 25.0), (2.0, 3.0)])
+def test_prompt_form_with_scores_of_every_size(cap, factor):
+    """Small and large scores: bounds that serve as their own reference and bounds that are too wide for it, no bound,
+    maxima that grow from page to page, scores beyond the polynomial's range."""
+    K = _K()
+    H, G, d, dv, n = 4, 2, 64, 128, 300
+    g = _gen(int(cap * 10 + factor))
+    kf = torch.randn(5, G, PS, d, generator=g)
+    kf = (kf * torch.linspace(0.2, 1.5, 5).reshape(5, 1, 1, 1)).to(torch.bfloat16)      # later pages score higher
+    vf = torch.randn(5, G, PS, dv, generator=g).to(torch.bfloat16)
+    row = torch.randn(n, H * d + 8, generator=g).to(torch.bfloat16)
+    talk = torch.eye(H) + torch.randn(H, H, generator=g) / H
+    ks, vs = (torch.cat([f[p].permute(1, 0, 2) for p in range(5)]).double() for f in (kf, vf))
+    pos = list(range(n))
+    kw = dict(cap=cap, coef=0.2, every=30.0, one=True)
+    scale = factor / math.sqrt(d)
+    want = _mixed_reference(row[:, :H * d].double().reshape(n, H, d), [ks], [vs], row[:, H * d:H * d + H].double(), talk.double(), pos,
+                            [n], scale, cap, 0.2, 30.0, True).reshape(n, H * dv)
+    cu, sot = _batch((n,))
+    for nv in (1, 2):
+        _prompt_form(K, row, H * d, kf, vf, talk, pos, [n], sot, cu, _i32([list(range(5))]), H, G, d, dv, scale, want, nv, kw)
+
+
 @pytest.mark.parametrize("H,G,d,dv,cap,temp,one,gated", [
     (4, 2, 64, 64, 20.0, (0.3, 16.0), True, True), (6, 2, 12, 20, 5.0, (0.5, 7.0), True, True),
     (8, 1, 32, 128, 0.0, None, True, True), (3, 3, 128, 40, 10.0, (1.0, 1.0), True, False),
@@ -190,6 +228,8 @@ def test_attention_with_mixed_heads_alone(H, G, d, dv, cap, temp, one, gated):
                 K.mixed_head_attention_mma(row.to(DEV), g_off, kf.to(DEV), vf.to(DEV), o, talk.to(DEV), _i32(pos), sot, cu, table,
                                            PS, T, 3, H, G, d, dv, scale, u, ml, nsplit=ns, max_new=mx, **kw)
                 assert rel_err(o, want) < 1.2e-2, (lens, ns, mx, rel_err(o, want))
+            for nv in (1, 2):
+                _prompt_form(K, row, g_off, kf, vf, talk, pos, lens, sot, cu, table, H, G, d, dv, scale, want, nv, kw)
         done = [x + n for x, n in zip(done, lens)]
     cu, sot = _batch((1, 1))
     sot[1] = -1
