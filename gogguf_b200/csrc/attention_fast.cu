@@ -887,7 +887,8 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
     // and a late warp that then waits for a P V which needs its own arrival would never leave
     uint64_t* p_ready = bars + 13;                  // [2]
     uint64_t* pv_done = bars + 15;
-    uint32_t* tmem_slot = (uint32_t*)(bars + 16);
+    uint64_t* o_done = bars + 16;                   // every P V is complete
+    uint32_t* tmem_slot = (uint32_t*)(bars + 17);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
     // no early release of the next kernel here: see the note on dependent launches in common.cuh
@@ -897,6 +898,7 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
         for (int i = 0; i < 2; ++i) { tma::mbar_init(&k_full[i], 1); tma::mbar_init(&k_empty[i], 1); }
         for (int i = 0; i < 3; ++i) { tma::mbar_init(&v_full[i], 1); tma::mbar_init(&v_empty[i], 1); }
         tma::mbar_init(&s_full[0], 1); tma::mbar_init(&s_full[1], 1); tma::mbar_init(pv_done, 1);
+        tma::mbar_init(o_done, 1);
         tma::mbar_init(&p_ready[0], 4);       // one arrival per softmax warp
         tma::mbar_init(&p_ready[1], 4);
         *abort_flag = 0;
@@ -998,6 +1000,7 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
                 tc5::commit(pv_done);
                 tc5::commit(&v_empty[vs]);
             }
+            if (ok) tc5::commit(o_done);
         }
     } else if (active) {
         const int row = threadIdx.x;                       // query row of the tile = tensor-memory lane
@@ -1105,10 +1108,9 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
             __syncwarp();
             if (lane == 0) tma::mbar_arrive(&p_ready[j & 1]);
         }
-        // The last P V.  The scores of the last page say that the P V of two pages before is complete; the one
-        // in between has not been waited for, and a wait by parity can only tell neighbouring phases apart.
-        if (ok && ntiles > 1) ok = tma::mbar_wait(pv_done, (uint32_t)((ntiles - 2) & 1), abort_flag, status, 28);
-        if (ok && tma::mbar_wait(pv_done, (uint32_t)((ntiles - 1) & 1), abort_flag, status, 28)) {
+        // The last P V, on a barrier of its own that completes once: a warp that comes late to a wait by parity could find
+        // two phases gone, which looks like none.
+        if (ok && tma::mbar_wait(o_done, 0, abort_flag, status, 28)) {
             tc5::fence_after();
             const float ls = attn_sink_sum(l, m_used, sink, h);
             const float inv = ls > 0.f ? out_scale / ls : 0.f;

@@ -62,6 +62,7 @@ MODULES: Dict[str, str] = {
     "diff_attention": "diff_attention.cu",
     "mixed_head_attention": "mixed_head_attention.cu",
     "mixed_head_prompt": "mixed_head_prompt.cu",
+    "mixed_head_decode": "mixed_head_decode.cu",
     "sampling": "sampling.cu",
     "gemm_tcgen05": "gemm_tcgen05.cu",
     "attention_fast": "attention_fast.cu",

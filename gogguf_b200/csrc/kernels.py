@@ -560,7 +560,7 @@ def mixed_head_attention_prompt(row: torch.Tensor, g_off: int, k_pool: torch.Ten
                                 coef: float = 0.0, every: float = 1.0, one: bool = False, window: int = 0,
                                 value_heads: Optional[int] = None) -> None:
     """`mixed_head_attention_mma` for prompts, on the tcgen05 tensor cores (128 query rows of a head per CTA).
-    value_heads: kv heads' values per CTA, 1 or 2 (default: 2 where there are several)."""
+    value_heads: kv heads' values per CTA: 1, 2 or, for dv <= 64, 4 (default: as many as there are)."""
     _mixed_head_check(row, k_pool, v_pool, out, talk, heads, kv_heads, d, dv, g_off)
     _need(row, torch.bfloat16, "row")
     _need(u, torch.float32, "u")
@@ -568,7 +568,7 @@ def mixed_head_attention_prompt(row: torch.Tensor, g_off: int, k_pool: torch.Ten
     if u.numel() < n_tokens * heads * kv_heads * dv or ml.numel() < n_tokens * heads * 2:
         raise KernelError("mixed_head_attention_prompt: the scratch is too small")
     if value_heads is None:
-        value_heads = 2 if kv_heads > 1 else 1
+        value_heads = 4 if kv_heads > 2 and dv <= 64 else min(kv_heads, 2)
     from .tcgen05_gemm import status_word
     kernel("mixed_head_prompt", "gg_mixed_head_prompt")(
         _p(row), row.stride(0), _p(k_pool), _p(v_pool), _p(u), _p(ml), _p(cu_seqlens), _p(ctx_lens), _p(seq_of_token),
@@ -578,6 +578,43 @@ def mixed_head_attention_prompt(row: torch.Tensor, g_off: int, k_pool: torch.Ten
     kernel("mixed_head_attention", "gg_mixed_head_combine")(
         _p(u), _p(ml), _p(row), row.stride(0), int(g_off), _p(out), out.stride(0), _p(talk), _p(seq_of_token), int(n_tokens),
         int(heads), int(kv_heads), int(dv), 1, float(bool(one)), _stream())
+
+
+def mixed_head_decode_takes(heads: int, kv_heads: int, d: int, dv: int, page_size: int) -> bool:
+    """Does the form for few rows over long contexts take these sizes (bfloat16 tensors)?"""
+    from .build import module
+    return bool(module("mixed_head_decode").lib.gg_mixed_head_decode_takes(int(heads), int(kv_heads), int(d), int(dv),
+                                                                          int(page_size)))
+
+
+def mixed_head_decode_splits(n_tokens: int, kv_heads: int, max_ctx: int) -> int:
+    """Into how many shares the pages of a (token, kv head) are cut: towards three CTAs a multiprocessor."""
+    return int(max(1, min(32, 444 // max(n_tokens * kv_heads, 1), -(-max_ctx // 64))))
+
+
+def mixed_head_attention_decode(row: torch.Tensor, g_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
+                                talk: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
+                                page_table: torch.Tensor, page_size: int, n_tokens: int, heads: int, kv_heads: int, d: int,
+                                dv: int, scale: float, scores: torch.Tensor, ml: torch.Tensor, part: torch.Tensor,
+                                nsplit: int, cap: float = 0.0, coef: float = 0.0, every: float = 1.0, one: bool = False,
+                                window: int = 0) -> None:
+    """`mixed_head_attention_mma` for steps of few rows over long contexts: keys and values are each read once.  Scratch
+    (float32): scores [n_tokens, heads, positions], positions a multiple of 64 that holds the longest sequence; ml of
+    n_tokens * heads * nsplit * 2 numbers, part of n_tokens * heads * nsplit * dv."""
+    _mixed_head_check(row, k_pool, v_pool, out, talk, heads, kv_heads, d, dv, g_off)
+    _need(row, torch.bfloat16, "row")
+    for t, n in ((scores, n_tokens * heads), (ml, n_tokens * heads * nsplit * 2), (part, n_tokens * heads * nsplit * dv)):
+        _need(t, torch.float32, "scratch")
+        if t.numel() < n:
+            raise KernelError("mixed_head_attention_decode: the scratch is too small")
+    if scores.dim() != 3 or tuple(scores.shape[:2]) != (n_tokens, heads):
+        raise KernelError("mixed_head_attention_decode: scores is [n_tokens, heads, positions]")
+    from .tcgen05_gemm import status_word
+    kernel("mixed_head_decode", "gg_mixed_head_decode")(
+        _p(row), row.stride(0), int(g_off), _p(k_pool), _p(v_pool), _p(out), out.stride(0), _p(talk), _p(positions),
+        _p(seq_of_token), _p(page_table), page_table.shape[-1], int(page_size), k_pool.shape[0], int(n_tokens), int(heads),
+        int(kv_heads), int(d), int(dv), float(scale), float(cap), float(coef), float(every), float(bool(one)), int(window),
+        int(nsplit), _p(scores), scores.shape[-1], _p(ml), _p(part), _p(status_word(row.device)), _stream())
 
 
 def diff_attention_partial_elems(n_tokens: int, heads: int, dv: int, nsplit: int) -> int:

@@ -604,12 +604,12 @@ def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps, value_heads=None):
             K.mixed_head_attention_prompt(row, g_off, kpool, vpool, o, talk, sot, cu, ends, table, ps, T, n_seqs, H, G, d, dv, d ** -0.5,
                                           u, ml, value_heads=value_heads, **kw)
             return
-        ns = K.mixed_head_splits(T, n_seqs, H, G, max_ctx)
+        ns = K.mixed_head_decode_splits(T, G, max_ctx)
         if T not in scratch:
-            scratch[T] = (torch.empty(T * H * ns * G * dv, device=row.device), torch.empty(T * H * ns * 2, device=row.device))
-        u, ml = scratch[T]
-        K.mixed_head_attention_mma(row, g_off, kpool, vpool, o, talk, pos, sot, cu, table, ps, T, n_seqs, H, G, d, dv, d ** -0.5, u, ml,
-                                   nsplit=ns, max_new=max_new, **kw)
+            scratch[T] = (torch.empty(T, H, -(-max_ctx // 64) * 64, device=row.device), torch.empty(T * H * ns * 2, device=row.device),
+                          torch.empty(T * H * ns * dv, device=row.device))
+        K.mixed_head_attention_decode(row, g_off, kpool, vpool, o, talk, pos, sot, table, ps, T, H, G, d, dv, d ** -0.5, *scratch[T], ns,
+                                      **kw)
 
     return run
 

@@ -563,6 +563,66 @@ __global__ void __launch_bounds__(MC_WARPS * 32) mixed_head_combine_kernel(
     }
 }
 
+// The same for one share (prompts): a warp per token and kv head, a lane four columns, a block the tokens of one kv head, so
+// that the rows of T it needs sit in shared memory, HC heads of the kv head at a time.
+template <int HC>
+__global__ void __launch_bounds__(MC_WARPS * 32) mixed_head_combine_rows_kernel(
+    const float* u, const float* ml, const bf16* row, long long ld, int g_off, bf16* out, long long ldo,
+    const float* __restrict__ talk, const int* __restrict__ seq_of_token, int ntok, int H, int G, int dv, float one) {
+    pdl_launch();
+    extern __shared__ __align__(16) float cr_sm[];
+    const int gv = blockIdx.y, hpg = H / G;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* tk = cr_sm;                                  // [H][HC]
+    float* f = tk + H * HC + warp * H;                  // [H] of this warp's token
+    const int t = blockIdx.x * MC_WARPS + warp, c = 4 * lane;
+    const bool have = t < ntok, live = have && seq_of_token[have ? t : 0] >= 0;
+    pdl_wait();
+    if (live) {
+        for (int h = lane; h < H; h += 32) {
+            const float m = ml[((size_t)t * H + h) * 2], l = ml[((size_t)t * H + h) * 2 + 1];
+            const float M = one > 0.f ? fmaxf(m, 0.f) : m;
+            const float e = mh_ex2(m - M);
+            f[h] = e / (l * e + (one > 0.f ? one * mh_ex2(-M) : 0.f));
+        }
+    }
+    for (int h0 = 0; h0 < hpg; h0 += HC) {
+        __syncthreads();
+        for (int i = threadIdx.x; i < H * HC; i += blockDim.x) {
+            const int g = i / HC, k = i - g * HC;
+            tk[i] = h0 + k < hpg ? talk[(size_t)(gv * hpg + h0 + k) * H + g] : 0.f;
+        }
+        __syncthreads();
+        if (!have || c >= dv) continue;
+        float acc[HC][4];
+#pragma unroll
+        for (int k = 0; k < HC; ++k) acc[k][0] = acc[k][1] = acc[k][2] = acc[k][3] = 0.f;
+        if (live) {
+            const float* ub = u + ((size_t)t * H * G + gv) * dv + c;
+#pragma unroll 4
+            for (int g = 0; g < H; ++g) {
+                const float4 v = *reinterpret_cast<const float4*>(ub + (size_t)g * G * dv);
+                const float fg = f[g];
+#pragma unroll
+                for (int k = 0; k < HC; ++k) {
+                    const float w = tk[g * HC + k] * fg;
+                    acc[k][0] = fmaf(w, v.x, acc[k][0]); acc[k][1] = fmaf(w, v.y, acc[k][1]);
+                    acc[k][2] = fmaf(w, v.z, acc[k][2]); acc[k][3] = fmaf(w, v.w, acc[k][3]);
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < HC; ++k) {
+            if (h0 + k >= hpg) break;
+            const int h = gv * hpg + h0 + k;
+            float s = 1.f;
+            if (live && g_off >= 0) s = 1.0f / (1.0f + mh_ex2(-MH_LOG2E * __bfloat162float(row[(size_t)t * ld + g_off + h])));
+            const uint32_t a = mh_pack(acc[k][0] * s, acc[k][1] * s), b = mh_pack(acc[k][2] * s, acc[k][3] * s);
+            *reinterpret_cast<uint2*>(out + (size_t)t * ldo + (size_t)h * dv + c) = make_uint2(a, b);
+        }
+    }
+}
+
 // 1 if the tensor-core form takes these sizes (bfloat16 only), else 0.
 GG_API gg_mixed_head_mma_takes(int H, int G, int d, int dv, int page_size) {
     return (d > 0 && d <= 128 && d % 8 == 0 && dv > 0 && dv <= 128 && dv % 8 == 0 && page_size == MH_KEYS && G > 0 &&
@@ -579,6 +639,15 @@ GG_API gg_mixed_head_combine(const float* u, const float* ml, const void* row, l
     if (ntok <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || dv <= 0 || dv > 128 || dv % 4 || nsplit < 1 || ldo < (long long)H * dv || (((uintptr_t)u) & 15))
         return GG_ERR_ARG;
+    if (nsplit == 1 && ntok >= 64 && (ldo % 4) == 0 && (((uintptr_t)out) & 7) == 0) {
+        const int hc = H / G > 2 ? 4 : (H / G > 1 ? 2 : 1);
+        const size_t sm = (size_t)H * (hc + MC_WARPS) * sizeof(float);
+        if (sm <= 48 * 1024) {
+            auto kern = hc == 4 ? mixed_head_combine_rows_kernel<4> : (hc == 2 ? mixed_head_combine_rows_kernel<2> : mixed_head_combine_rows_kernel<1>);
+            return gg_launch(kern, dim3((ntok + MC_WARPS - 1) / MC_WARPS, G), dim3(MC_WARPS * 32), sm, stream, 1, u, ml, (const bf16*)row,
+                             ld, g_off, (bf16*)out, ldo, talk, seq_of_token, ntok, H, G, dv, one);
+        }
+    }
     const size_t smem = ((size_t)H * nsplit + MC_WARPS * 4 * 128) * sizeof(float);
     if (smem > 220 * 1024) return GG_ERR_ARG;
     if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_combine_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

@@ -20,6 +20,7 @@
 #include "tma_util.cuh"
 
 #define MHP_PAGE 64
+#define MHP_MODEST 57.0f          // a bound (log2 units) below this keeps the sum of 64 weights below 2^64
 #define MHP_LOG2E 1.4426950408889634f
 
 namespace {
@@ -66,13 +67,16 @@ struct PromptSizes {
     static constexpr int TMEM = COLS <= 256 ? 256 : 512;
 };
 
-template <int D, int DV, int NV>
-__global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 : 1) mixed_head_prompt_kernel(
+// PAIR: two softmax warpgroups take turns, the even pages and the odd ones, each with a score buffer of its own (only for
+// scores that need no running reference).
+template <int D, int DV, int NV, bool PAIR>
+__global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 : 1) mixed_head_prompt_kernel(
     const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     float* __restrict__ u, float* __restrict__ ml, const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens,
     const int* __restrict__ seq_of_token, const int* __restrict__ page_table, int max_pages, int n_seqs, int H, int G, int d,
     int dv, float scale, float cap, float coef, float every, int window, int n_pages, int* __restrict__ status) {
     typedef PromptSizes<D, DV, NV> Z;
+    constexpr int SW = PAIR ? 8 : 4;                // softmax warps; then the TMA warp and the MMA warp
     extern __shared__ __align__(1024) uint8_t smem[];
     uint8_t* Qs = smem;
     uint8_t* Ks = Qs + Z::Q_BYTES;                  // two stages
@@ -86,7 +90,8 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
     uint64_t* s_full = bars + 9;                    // [2]
     uint64_t* p_ready = bars + 11;                  // [2]: a softmax warp may be a page ahead of another
     uint64_t* pv_done = bars + 13;
-    uint32_t* tmem_slot = (uint32_t*)(bars + 14);
+    uint64_t* u_done = bars + 14;                   // every P V is complete
+    uint32_t* tmem_slot = (uint32_t*)(bars + 15);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
     // no early release of the next kernel: see the note on dependent launches in common.cuh
@@ -100,11 +105,12 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
             tma::mbar_init(&p_ready[i], 4);         // one arrival per softmax warp
         }
         tma::mbar_init(pv_done, 1);
+        tma::mbar_init(u_done, 1);
         *abort_flag = 0;
         tma::mbar_fence_init();
         tma::prefetch_map(&tmQ); tma::prefetch_map(&tmK); tma::prefetch_map(&tmV);
     }
-    if (warp == 5) tc5::alloc(tmem_slot, Z::TMEM);
+    if (warp == SW + 1) tc5::alloc(tmem_slot, Z::TMEM);
     tc5::fence_before();
     __syncthreads();
     tc5::fence_after();
@@ -134,7 +140,7 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
     const int ntiles = active ? kt_last - kt_first + 1 : 0;
     const uint32_t S_t = tmem_base, U_t = tmem_base + 128;
 
-    if (warp == 4) {
+    if (warp == SW) {
         if (lane == 0 && active) {
             const int* pt = page_table + (size_t)b * max_pages;
             tma::mbar_expect_tx(q_full, Z::Q_BYTES);
@@ -161,7 +167,7 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
                 }
             }
         }
-    } else if (warp == 5) {
+    } else if (warp == SW + 1) {
         if (lane == 0 && active) {
             const uint32_t idesc_qk = tc5::idesc_bf16(128, 64, 0), idesc_pv = tc5::idesc_bf16(128, DV, 1);
             const uint32_t q_a = tma::smem_u32(Qs), k_a = tma::smem_u32(Ks), v_a = tma::smem_u32(Vs);
@@ -202,20 +208,22 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
                 tc5::commit(pv_done);
                 tc5::commit(&v_empty[s]);
             }
+            if (ok) tc5::commit(u_done);
         }
     } else if (active) {
-        const int row = threadIdx.x;                       // query row of the tile = tensor-memory lane
-        const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
+        const int row = threadIdx.x & 127;                 // query row of the tile = tensor-memory lane
+        const int wg = PAIR ? warp >> 2 : 0;
+        const uint32_t lane_off = (uint32_t)((warp & 3) * 32) << 16;
         const int p = pos0 + row;
         const float tau = coef == 0.f ? 1.0f : 1.0f + coef * logf(floorf((float)(p + 1) / every) + 1.0f);
         const float fac = scale * tau * (cap > 0.f ? 1.0f / cap : MHP_LOG2E);
         const float cap_log2 = cap * MHP_LOG2E;
         const f2 fac2 = pk2(fac, fac);
         // the reference in use (log2 units); a bound that keeps 64 weights below 2^64 needs none
-        float ref = (cap > 0.f && cap_log2 < 57.0f) ? 0.f : -INFINITY;
+        float ref = (cap > 0.f && cap_log2 < MHP_MODEST) ? 0.f : -INFINITY;
         float l = 0.f;
         bool ok = true;
-        for (int j = 0; j < ntiles; ++j) {
+        for (int j = wg; j < ntiles; j += PAIR ? 2 : 1) {
             if (!tma::mbar_wait(&s_full[j & 1], (uint32_t)((j >> 1) & 1), abort_flag, status, 67)) { ok = false; break; }
             tc5::fence_after();
             uint32_t sr[64];
@@ -283,42 +291,46 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
                 return la + lb;
             };
             float lpage = 0.f;
-            bool again = ref == -INFINITY;
-            if (!__any_sync(0xffffffffu, again)) {
+            if (PAIR) {
                 lpage = exponentials();
-                again = !(lpage < 1.8446744e19f);
-            }
-            if (__any_sync(0xffffffffu, again)) {
-                float m8[8];
-#pragma unroll
-                for (int k = 0; k < 8; ++k) m8[k] = __uint_as_float(sr[k]);
-#pragma unroll
-                for (int c = 8; c < 64; ++c) m8[c & 7] = fmaxf(m8[c & 7], __uint_as_float(sr[c]));
-                const float mx = fmaxf(fmaxf(fmaxf(m8[0], m8[1]), fmaxf(m8[2], m8[3])), fmaxf(fmaxf(m8[4], m8[5]), fmaxf(m8[6], m8[7])));
-                const bool grow = mx > ref + 8.0f || (ref == -INFINITY && mx != -INFINITY);
-                if (__any_sync(0xffffffffu, grow)) {
-                    float corr = 1.0f;
-                    if (grow) {
-                        corr = ref == -INFINITY ? 0.f : mhp_ex2(ref - mx);
-                        ref = mx;
-                        l *= corr;
-                    }
-                    if (j > 0) {                           // P V of the page before must be complete before U is rescaled
-                        if (!tma::mbar_wait(pv_done, (uint32_t)((j - 1) & 1), abort_flag, status, 68)) { ok = false; break; }
-                        tc5::fence_after();
-#pragma unroll 1
-                        for (int c0 = 0; c0 < nv * DV; c0 += 32) {
-                            uint32_t orow[32];
-                            tc5::ld32(U_t + lane_off + c0, orow);
-                            tc5::wait_ld();
-#pragma unroll
-                            for (int c = 0; c < 32; ++c) orow[c] = __float_as_uint(__uint_as_float(orow[c]) * corr);
-                            tc5::st32(U_t + lane_off + c0, orow);
-                        }
-                        tc5::wait_st();
-                    }
+            } else {
+                bool again = ref == -INFINITY;
+                if (!__any_sync(0xffffffffu, again)) {
+                    lpage = exponentials();
+                    again = !(lpage < 1.8446744e19f);
                 }
-                lpage = exponentials();
+                if (__any_sync(0xffffffffu, again)) {
+                    float m8[8];
+    #pragma unroll
+                    for (int k = 0; k < 8; ++k) m8[k] = __uint_as_float(sr[k]);
+    #pragma unroll
+                    for (int c = 8; c < 64; ++c) m8[c & 7] = fmaxf(m8[c & 7], __uint_as_float(sr[c]));
+                    const float mx = fmaxf(fmaxf(fmaxf(m8[0], m8[1]), fmaxf(m8[2], m8[3])), fmaxf(fmaxf(m8[4], m8[5]), fmaxf(m8[6], m8[7])));
+                    const bool grow = mx > ref + 8.0f || (ref == -INFINITY && mx != -INFINITY);
+                    if (__any_sync(0xffffffffu, grow)) {
+                        float corr = 1.0f;
+                        if (grow) {
+                            corr = ref == -INFINITY ? 0.f : mhp_ex2(ref - mx);
+                            ref = mx;
+                            l *= corr;
+                        }
+                        if (j > 0) {                           // P V of the page before must be complete before U is rescaled
+                            if (!tma::mbar_wait(pv_done, (uint32_t)((j - 1) & 1), abort_flag, status, 68)) { ok = false; break; }
+                            tc5::fence_after();
+    #pragma unroll 1
+                            for (int c0 = 0; c0 < nv * DV; c0 += 32) {
+                                uint32_t orow[32];
+                                tc5::ld32(U_t + lane_off + c0, orow);
+                                tc5::wait_ld();
+    #pragma unroll
+                                for (int c = 0; c < 32; ++c) orow[c] = __float_as_uint(__uint_as_float(orow[c]) * corr);
+                                tc5::st32(U_t + lane_off + c0, orow);
+                            }
+                            tc5::wait_st();
+                        }
+                    }
+                    lpage = exponentials();
+                }
             }
             l += lpage;
             // P over this thread's own row of the scores it has read: the P V that read the P of two pages ago from this
@@ -329,26 +341,30 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
             __syncwarp();
             if (lane == 0) tma::mbar_arrive(&p_ready[j & 1]);
         }
-        // (a wait by parity can only tell neighbouring phases apart: the last two P V in turn)
-        if (ok && ntiles > 1) ok = tma::mbar_wait(pv_done, (uint32_t)((ntiles - 2) & 1), abort_flag, status, 68);
-        if (ok && tma::mbar_wait(pv_done, (uint32_t)((ntiles - 1) & 1), abort_flag, status, 68)) {
+        ok = ok && tma::mbar_wait(u_done, 0, abort_flag, status, 68);
+        const size_t at = (size_t)(tok0 + row0 + row) * H + h;
+        if (PAIR) {
+            // the odd pages' sums join the even pages' (both warpgroups come here, whatever happened to their waits)
+            float* sums = reinterpret_cast<float*>(smem);   // (Q is not read any more: its last reader is complete, or nothing is)
+            if (wg == 1) sums[row] = l;
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (wg == 0) l += sums[row];
+        }
+        if (ok) {
             tc5::fence_after();
-            const size_t at = (size_t)(tok0 + row0 + row) * H + h;
-            if (row < rows && v0 == 0) { ml[at * 2] = ref; ml[at * 2 + 1] = l; }
+            if (row < rows && v0 == 0 && wg == 0) { ml[at * 2] = ref; ml[at * 2 + 1] = l; }
+            // (a pair of warpgroups shares the runs of 32 columns out between its two)
 #pragma unroll 1
-            for (int n = 0; n < nv; ++n) {
-                float* dst = u + (at * G + v0 + n) * dv;
-#pragma unroll 1
-                for (int c0 = 0; c0 < DV; c0 += 32) {
-                    uint32_t orow[32];
-                    tc5::ld32(U_t + lane_off + (uint32_t)(n * DV + c0), orow);
-                    tc5::wait_ld();
-                    if (row < rows) {
+            for (int c0 = 32 * wg; c0 < nv * DV; c0 += PAIR ? 64 : 32) {
+                const int n = c0 / DV, e0 = c0 % DV;
+                float* dst = u + (at * G + v0 + n) * dv + e0;
+                uint32_t orow[32];
+                tc5::ld32(U_t + lane_off + (uint32_t)c0, orow);
+                tc5::wait_ld();
+                if (row < rows) {
 #pragma unroll
-                        for (int c = 0; c < 32; c += 4)
-                            if (c0 + c < dv)
-                                *reinterpret_cast<uint4*>(dst + c0 + c) = make_uint4(orow[c], orow[c + 1], orow[c + 2], orow[c + 3]);
-                    }
+                    for (int c = 0; c < 32; c += 4)
+                        if (e0 + c < dv) *reinterpret_cast<uint4*>(dst + c) = make_uint4(orow[c], orow[c + 1], orow[c + 2], orow[c + 3]);
                 }
             }
         }
@@ -360,18 +376,18 @@ __global__ void __launch_bounds__(192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 :
         while (clock64() - t0 < 2000000LL) { }
         __syncthreads();
     }
-    if (warp == 5) {
+    if (warp == SW + 1) {
         tc5::fence_after();
         tc5::dealloc(tmem_base, Z::TMEM);
     }
 }
 
-template <int D, int DV, int NV>
-int launch_prompt(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, float* u, float* ml, const int* cu_seqlens,
+template <int D, int DV, int NV, bool PAIR>
+int launch_prompt_form(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, float* u, float* ml, const int* cu_seqlens,
                   const int* ctx_lens, const int* seq_of_token, const int* page_table, int max_pages, int n_seqs, int max_tiles,
                   int H, int G, int d, int dv, float scale, float cap, float coef, float every, int window, int n_pages,
                   int* status, cudaStream_t stream) {
-    auto kern = mixed_head_prompt_kernel<D, DV, NV>;
+    auto kern = mixed_head_prompt_kernel<D, DV, NV, PAIR>;
     constexpr int smem = PromptSizes<D, DV, NV>::SMEM;
     static bool configured = false;                        // per instantiation
     if (!configured) {
@@ -379,9 +395,18 @@ int launch_prompt(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMa
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return gg_launch(kern, dim3(H * ((G + NV - 1) / NV), max_tiles), dim3(192), smem, stream, 1, tq, tk, tv, u, ml, cu_seqlens,
+    return gg_launch(kern, dim3(H * ((G + NV - 1) / NV), max_tiles), dim3(PAIR ? 320 : 192), smem, stream, 1, tq, tk, tv, u, ml, cu_seqlens,
                      ctx_lens, seq_of_token, page_table, max_pages, n_seqs, H, G, d, dv, scale, cap, coef, every, window, n_pages,
                      status);
+}
+
+template <int D, int DV, int NV, typename... Args>
+int launch_prompt(bool no_reference, Args... args) {
+    // forms that fill tensor memory have the multiprocessor to themselves: a second softmax warpgroup has room there
+    if constexpr (PromptSizes<D, DV, NV>::TMEM == 512) {
+        if (no_reference) return launch_prompt_form<D, DV, NV, true>(args...);
+    }
+    return launch_prompt_form<D, DV, NV, false>(args...);
 }
 
 }  // namespace
@@ -393,7 +418,7 @@ GG_API gg_mixed_head_prompt_takes(int H, int G, int d, int dv, int page_size) {
 
 // row [ntok, ld] bfloat16 with q [H][d] at column 0; pools k [page][G][64][d], v [..][dv]; u [ntok][H][G][dv] and
 // ml [ntok][H][2] float32; max_tiles >= sum over sequences of ceil(new tokens / 128).  cap 0: scores not bounded; coef 0: no
-// temperature; window <= 0: none.  value_heads: kv heads' values per CTA (1 or 2).  A wait that runs out leaves one of the
+// temperature; window <= 0: none.  value_heads: kv heads' values per CTA (1 or 2; 4 for dv <= 64).  A wait that runs out leaves one of the
 // codes 61-68 in the status word.
 GG_API gg_mixed_head_prompt(const void* row, long long ld, const void* k_pool, const void* v_pool, float* u, float* ml,
                             const int* cu_seqlens, const int* ctx_lens, const int* seq_of_token, const int* page_table,
@@ -403,7 +428,7 @@ GG_API gg_mixed_head_prompt(const void* row, long long ld, const void* k_pool, c
     if (ntok <= 0 || n_seqs <= 0 || max_tiles <= 0) return 0;
     if (!gg_mixed_head_prompt_takes(H, G, d, dv, page_size) || max_tiles > 65535 || n_pages <= 0 || status == nullptr || u == nullptr ||
         ml == nullptr || (ld % 8) || ld < (long long)H * d || cap < 0.f || (coef != 0.f && !(every > 0.f)) ||
-        (value_heads != 1 && value_heads != 2) ||
+        (value_heads != 1 && value_heads != 2 && !(value_heads == 4 && dv <= 64)) ||
         (((uintptr_t)row | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)u) & 15))
         return GG_ERR_ARG;
     CUtensorMap tq, tk, tv;
@@ -414,9 +439,10 @@ GG_API gg_mixed_head_prompt(const void* row, long long ld, const void* k_pool, c
     if ((rc = tma::make_map_bf16(&tq, row, (unsigned long long)ntok, H * d, ld, 128)) != 0) return rc;
     if ((rc = tma::make_map_bf16(&tk, k_pool, rows, d, d, MHP_PAGE)) != 0) return rc;
     if ((rc = tma::make_map_bf16(&tv, v_pool, rows, dv, dv, MHP_PAGE)) != 0) return rc;
+#define MHP_ARGS cap > 0.f && cap * MHP_LOG2E < MHP_MODEST, tq, tk, tv, u, ml, cu_seqlens, ctx_lens, seq_of_token, page_table, \
+        max_pages, n_seqs, max_tiles, H, G, d, dv, scale, cap, coef, every, window, n_pages, status, stream
 #define MHP_GO(D_, V_) (value_heads == 2 ? launch_prompt<D_, V_, 2>(MHP_ARGS) : launch_prompt<D_, V_, 1>(MHP_ARGS))
-#define MHP_ARGS tq, tk, tv, u, ml, cu_seqlens, ctx_lens, seq_of_token, page_table, max_pages, n_seqs, max_tiles, H, G, d, dv, scale, \
-        cap, coef, every, window, n_pages, status, stream
+    if (value_heads == 4) return d <= 64 ? launch_prompt<64, 64, 4>(MHP_ARGS) : launch_prompt<128, 64, 4>(MHP_ARGS);
     if (d <= 64) return dv <= 64 ? MHP_GO(64, 64) : MHP_GO(64, 128);
     return dv <= 64 ? MHP_GO(128, 64) : MHP_GO(128, 128);
 #undef MHP_ARGS

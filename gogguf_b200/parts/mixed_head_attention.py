@@ -37,6 +37,7 @@ from .base import Linear, Runtime, StepContext
 from .registry import register_mixer
 
 PROMPT_FORM_MIN_TOKENS = 48      # steps whose longest stretch of new tokens has at least this many take the tcgen05 form
+DECODE_FORM_MAX_TOKENS = 4       # ... and steps that bring at most this many to each sequence the form for few rows
 
 FIRST_VALUES = "mixed_head_first_values"      # workspace: the source layer's values of the step's tokens
 
@@ -151,9 +152,17 @@ class MixedHeadAttentionMixer:
             ml = ctx.ws.get("mixed_head_ml", (T * H * 2,), torch.float32)
             K.mixed_head_attention_prompt(row, self.g_off, cache.k, cache.v, o, self.talk, ctx.seq_of_token, ctx.cu_seqlens,
                                           ctx.ctx_lens, table, cache.page_size, T, ctx.n_seqs, H, G, d, dv, self.scale, u, ml, **kw)
+        elif (self._mma and ctx.max_new <= DECODE_FORM_MAX_TOKENS
+                and K.mixed_head_decode_takes(H, G, d, dv, cache.page_size)):
+            nsplit = K.mixed_head_decode_splits(T, G, int(ctx.max_ctx))
+            scores = ctx.ws.get("mixed_head_scores", (T, H, -(-int(ctx.max_ctx) // 64) * 64), torch.float32)
+            ml = ctx.ws.get("mixed_head_ml", (T * H * nsplit * 2,), torch.float32)
+            part = ctx.ws.get("mixed_head_part", (T * H * nsplit * dv,), torch.float32)
+            K.mixed_head_attention_decode(row, self.g_off, cache.k, cache.v, o, self.talk, ctx.positions, ctx.seq_of_token, table,
+                                          cache.page_size, T, H, G, d, dv, self.scale, scores, ml, part, nsplit, **kw)
         elif self._mma and K.mixed_head_mma_takes(H, G, d, dv, cache.page_size):
-            # steps of few rows over long contexts (decode steps): the key tiles are shared out over several CTAs
-            nsplit = K.mixed_head_splits(T, ctx.n_seqs, H, G, int(ctx.max_ctx)) if ctx.max_new <= 4 else 1
+            # (steps of few rows over long contexts: the key tiles are shared out over several CTAs)
+            nsplit = K.mixed_head_splits(T, ctx.n_seqs, H, G, int(ctx.max_ctx)) if ctx.max_new <= DECODE_FORM_MAX_TOKENS else 1
             u = ctx.ws.get("mixed_head_u", (T * H * nsplit * G * dv,), torch.float32)
             ml = ctx.ws.get("mixed_head_ml", (T * H * nsplit * 2,), torch.float32)
             K.mixed_head_attention_mma(row, self.g_off, cache.k, cache.v, o, self.talk, ctx.positions, ctx.seq_of_token,

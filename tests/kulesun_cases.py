@@ -125,8 +125,9 @@ def draw_case(seed: int) -> dict:
         else:
             share = r.random() < 0.8
             g = G if share else r.choice([1, 2, 4])
-            m = attn(g * r.choice([1, 2, 4, 5]), g, r.choice([4, 8, 20, 32, 64, 128]), vdim if share else r.choice([8, 20, 64]),
-                     r.choice([0.1, 0.3, 1.0]), r.choice([None, 5.0, 30.0]),
+            dim = r.choice([4, 8, 20, 32, 64, 128])
+            m = attn(g * r.choice([1, 2, 4, 5]), g, dim, vdim if share else r.choice([8, 20, 64]),
+                     round(r.choice([0.3, 1.0, 2.0]) * dim ** -0.5, 4), r.choice([None, 5.0, 30.0]),
                      r.choice([None, (0.5, 4.0), (0.1, 100.0), (2.0, 1.0)]), v_mix=share)
         layers.append(layer(m, ff))
     return model(r.choice([53, 211, 641]), width, r.choice([1e-6, 1e-5, 3e-4]), layers, r.choice([1.0, 7.0]),

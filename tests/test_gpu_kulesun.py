@@ -228,18 +228,29 @@ def test_attention_with_mixed_heads_alone(H, G, d, dv, cap, temp, one, gated):
                 K.mixed_head_attention_mma(row.to(DEV), g_off, kf.to(DEV), vf.to(DEV), o, talk.to(DEV), _i32(pos), sot, cu, table,
                                            PS, T, 3, H, G, d, dv, scale, u, ml, nsplit=ns, max_new=mx, **kw)
                 assert rel_err(o, want) < 1.2e-2, (lens, ns, mx, rel_err(o, want))
-            for nv in (1, 2):
+            if max(lens) <= 3 and K.mixed_head_decode_takes(H, G, d, dv, PS):
+                for ns in (1, 3, 8):
+                    o = torch.empty(T, H * dv, dtype=torch.bfloat16, device=DEV)
+                    scores = torch.full((T, H, 8 * PS), 1e30, device=DEV)
+                    ml, part = torch.full((T * H * ns * 2,), 1e30, device=DEV), torch.full((T * H * ns * dv,), 1e30, device=DEV)
+                    K.mixed_head_attention_decode(row.to(DEV), g_off, kf.to(DEV), vf.to(DEV), o, talk.to(DEV), _i32(pos), sot, table, PS,
+                                                  T, H, G, d, dv, scale, scores, ml, part, ns, **kw)
+                    assert rel_err(o, want) < 6e-3, (lens, ns, rel_err(o, want))
+            for nv in (1, 2) + ((4,) if dv <= 64 else ()):
                 _prompt_form(K, row, g_off, kf, vf, talk, pos, lens, sot, cu, table, H, G, d, dv, scale, want, nv, kw)
         done = [x + n for x, n in zip(done, lens)]
     cu, sot = _batch((1, 1))
     sot[1] = -1
-    for which in ("plain", "mma"):
+    for which in ("plain", "mma", "decode"):
         o = torch.full((2, H * dv), 5.0, dtype=torch.bfloat16, device=DEV)
         row = torch.randn(2, width, generator=g).to(torch.bfloat16).to(DEV)
         args = (row, g_off, kf.to(DEV), vf.to(DEV), o, talk.to(DEV), _i32([done[0], 0]), sot)
         if which == "plain":
             K.mixed_head_attention_plain(*args, table[:2].contiguous(), PS, 2, H, G, d, dv, scale, **kw)
-        elif K.mixed_head_mma_takes(H, G, d, dv, PS):
+        elif which == "decode" and K.mixed_head_decode_takes(H, G, d, dv, PS):
+            K.mixed_head_attention_decode(*args, table[:2].contiguous(), PS, 2, H, G, d, dv, scale, torch.empty(2, H, 8 * PS, device=DEV),
+                                          torch.empty(4 * H, device=DEV), torch.empty(2 * H * dv, device=DEV), 1, **kw)
+        elif which == "mma" and K.mixed_head_mma_takes(H, G, d, dv, PS):
             K.mixed_head_attention_mma(*args, cu, table[:2].contiguous(), PS, 2, 2, H, G, d, dv, scale,
                                        torch.empty(2 * H * G * dv, device=DEV), torch.empty(4 * H, device=DEV), max_new=1, **kw)
         else:
@@ -269,6 +280,11 @@ def test_scores_that_are_all_far_below_the_one():
                                    torch.empty(H * ns * dv, device=DEV), torch.empty(H * ns * 2, device=DEV), one=True, nsplit=ns,
                                    max_new=1)
         assert 0 < float(want.abs().max()) < 1e-4 and rel_err(o, want) < 1.2e-2
+        K.mixed_head_attention_decode(q.to(torch.bfloat16).to(DEV), -1, kf.to(torch.bfloat16).to(DEV), vf.to(torch.bfloat16).to(DEV), o,
+                                      torch.eye(H, device=DEV), _i32([n - 1]), sot, _i32([[0, 1, 2, 3]]), PS, 1, H, G, d, dv, 1.0,
+                                      torch.empty(1, H, 256, device=DEV), torch.empty(H * ns * 2, device=DEV),
+                                      torch.empty(H * ns * dv, device=DEV), ns, one=True)
+        assert rel_err(o, want) < 6e-3
 
 
 @pytest.mark.parametrize("dt,qdt", [(torch.float32, torch.float32), (torch.bfloat16, torch.float32), (torch.bfloat16, torch.bfloat16)])
