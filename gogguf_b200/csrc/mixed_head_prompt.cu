@@ -67,16 +67,18 @@ struct PromptSizes {
     static constexpr int TMEM = COLS <= 256 ? 256 : 512;
 };
 
-// PAIR: two softmax warpgroups take turns, the even pages and the odd ones, each with a score buffer of its own (only for
-// scores that need no running reference).
-template <int D, int DV, int NV, bool PAIR>
-__global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 : 1) mixed_head_prompt_kernel(
+// GROUPS softmax warpgroups.  One: any scores.  Two (scores that need no running reference): both take every page, 32 of
+// its 64 keys each.  Four: two such pairs take turns, the even pages and the odd ones, each with a score buffer of its own.
+template <int D, int DV, int NV, int GROUPS>
+__global__ void __launch_bounds__(GROUPS * 128 + 64, PromptSizes<D, DV, NV>::TMEM == 256 ? 2 : 1) mixed_head_prompt_kernel(
     const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     float* __restrict__ u, float* __restrict__ ml, const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens,
     const int* __restrict__ seq_of_token, const int* __restrict__ page_table, int max_pages, int n_seqs, int H, int G, int d,
     int dv, float scale, float cap, float coef, float every, int window, int n_pages, int* __restrict__ status) {
     typedef PromptSizes<D, DV, NV> Z;
-    constexpr int SW = PAIR ? 8 : 4;                // softmax warps; then the TMA warp and the MMA warp
+    constexpr int SW = GROUPS * 4;                  // softmax warps; then the TMA warp and the MMA warp
+    constexpr bool PAIR = GROUPS > 1;               // no reference is kept
+    constexpr int STEP = GROUPS == 4 ? 2 : 1, NK = PAIR ? 32 : 64;      // pages from one of a thread's to its next, keys of it
     extern __shared__ __align__(1024) uint8_t smem[];
     uint8_t* Qs = smem;
     uint8_t* Ks = Qs + Z::Q_BYTES;                  // two stages
@@ -102,7 +104,7 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
             tma::mbar_init(&k_full[i], 1); tma::mbar_init(&k_empty[i], 1);
             tma::mbar_init(&v_full[i], 1); tma::mbar_init(&v_empty[i], 1);
             tma::mbar_init(&s_full[i], 1);
-            tma::mbar_init(&p_ready[i], 4);         // one arrival per softmax warp
+            tma::mbar_init(&p_ready[i], PAIR ? 8 : 4);       // one arrival per softmax warp of the page
         }
         tma::mbar_init(pv_done, 1);
         tma::mbar_init(u_done, 1);
@@ -201,7 +203,8 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk) {
                         const uint64_t bb = tc5::smem_desc(v_a + s * Z::V_STAGE + n * Z::V_HEAD + kk * 2048, Z::KBOX, 1024);
-                        tc5::mma_a_tmem(U_t + (uint32_t)(n * DV), S_t + (uint32_t)(s * 64 + kk * 8), bb, idesc_pv,
+                        // (16 keys of P are 8 columns; each group's lie over the scores it alone has read)
+                        tc5::mma_a_tmem(U_t + (uint32_t)(n * DV), S_t + (uint32_t)(s * 64 + (PAIR ? (kk >> 1) * 32 + (kk & 1) * 8 : kk * 8)), bb, idesc_pv,
                                         (j > 0 || kk > 0) ? 1u : 0u);
                     }
                 }
@@ -212,7 +215,7 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
         }
     } else if (active) {
         const int row = threadIdx.x & 127;                 // query row of the tile = tensor-memory lane
-        const int wg = PAIR ? warp >> 2 : 0;
+        const int wg = warp >> 2, half = PAIR ? wg & 1 : 0;      // (of a page's keys)
         const uint32_t lane_off = (uint32_t)((warp & 3) * 32) << 16;
         const int p = pos0 + row;
         const float tau = coef == 0.f ? 1.0f : 1.0f + coef * logf(floorf((float)(p + 1) / every) + 1.0f);
@@ -223,12 +226,12 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
         float ref = (cap > 0.f && cap_log2 < MHP_MODEST) ? 0.f : -INFINITY;
         float l = 0.f;
         bool ok = true;
-        for (int j = wg; j < ntiles; j += PAIR ? 2 : 1) {
+        for (int j = GROUPS == 4 ? wg >> 1 : 0; j < ntiles; j += STEP) {
             if (!tma::mbar_wait(&s_full[j & 1], (uint32_t)((j >> 1) & 1), abort_flag, status, 67)) { ok = false; break; }
             tc5::fence_after();
-            uint32_t sr[64];
-            tc5::ld32(S_t + lane_off + (uint32_t)((j & 1) * 64), sr);
-            tc5::ld32(S_t + lane_off + (uint32_t)((j & 1) * 64) + 32, sr + 32);
+            uint32_t sr[NK];
+            tc5::ld32(S_t + lane_off + (uint32_t)((j & 1) * 64 + half * 32), sr);
+            if (!PAIR) tc5::ld32(S_t + lane_off + (uint32_t)((j & 1) * 64) + 32, sr + (NK - 32));
             tc5::wait_ld();
             auto pair = [&](int e) { return pk2(__uint_as_float(sr[2 * e]), __uint_as_float(sr[2 * e + 1])); };
             auto put = [&](int e, f2 v) {
@@ -238,28 +241,33 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
                 sr[2 * e + 1] = __float_as_uint(c);
             };
 #pragma unroll
-            for (int e = 0; e < 32; ++e) put(e, mul2(pair(e), fac2));
+            for (int e = 0; e < NK / 2; ++e) put(e, mul2(pair(e), fac2));
             if (cap > 0.f) {
                 float mx4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], fabsf(__uint_as_float(sr[c])));
+                for (int c = 0; c < NK; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], fabsf(__uint_as_float(sr[c])));
                 const bool wide = !(fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) <= 1.0f);
                 if (!__any_sync(0xffffffffu, wide)) {
-                    const float c0 = 0.9999999403953552f * cap_log2, c1 = -0.33332857489585876f * cap_log2,
-                                c2 = 0.13325397670269012f * cap_log2, c3 = -0.05346517637372017f * cap_log2,
-                                c4 = 0.020305519923567772f * cap_log2, c5 = -0.006217069923877716f * cap_log2,
-                                c6 = 0.0010455535957589746f * cap_log2;
-                    const f2 k0 = pk2(c0, c0), k1 = pk2(c1, c1), k2 = pk2(c2, c2), k3 = pk2(c3, c3), k4 = pk2(c4, c4),
-                             k5 = pk2(c5, c5), k6 = pk2(c6, c6);
+                    const float cf[7] = {0.9999999403953552f, -0.33332857489585876f, 0.13325397670269012f, -0.05346517637372017f,
+                                         0.020305519923567772f, -0.006217069923877716f, 0.0010455535957589746f};
+                    constexpr int RUN = 8;                 // pairs side by side: the chains of multiply-adds overlap
 #pragma unroll
-                    for (int e = 0; e < 32; ++e) {
-                        const f2 x = pair(e), t = mul2(x, x);
-                        const f2 q = fma2(t, fma2(t, fma2(t, fma2(t, fma2(t, fma2(t, k6, k5), k4), k3), k2), k1), k0);
-                        put(e, mul2(x, q));
+                    for (int e0 = 0; e0 < NK / 2; e0 += RUN) {
+                        f2 t[RUN], q[RUN];
+#pragma unroll
+                        for (int e = 0; e < RUN; ++e) { t[e] = mul2(pair(e0 + e), pair(e0 + e)); q[e] = pk2(cf[6] * cap_log2, cf[6] * cap_log2); }
+#pragma unroll
+                        for (int k = 5; k >= 0; --k) {
+                            const f2 ck = pk2(cf[k] * cap_log2, cf[k] * cap_log2);
+#pragma unroll
+                            for (int e = 0; e < RUN; ++e) q[e] = fma2(t[e], q[e], ck);
+                        }
+#pragma unroll
+                        for (int e = 0; e < RUN; ++e) put(e0 + e, mul2(pair(e0 + e), q[e]));
                     }
                 } else {
 #pragma unroll
-                    for (int c = 0; c < 64; ++c) {
+                    for (int c = 0; c < NK; ++c) {
                         const float t = mhp_ex2(__uint_as_float(sr[c]) * (2.0f * MHP_LOG2E));
                         sr[c] = __float_as_uint(cap_log2 - __fdividef(2.0f * cap_log2, t + 1.0f));
                     }
@@ -268,20 +276,20 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
             const int key0 = (kt_first + j) * MHP_PAGE;
             if ((key0 + MHP_PAGE - 1 > pos0) || (window > 0 && key0 < pos0 + 127 - window + 1)) {
 #pragma unroll
-                for (int c = 0; c < 64; ++c) {
-                    const int kidx = key0 + c;
+                for (int c = 0; c < NK; ++c) {
+                    const int kidx = key0 + half * 32 + c;
                     if (!(kidx <= p && (window <= 0 || kidx > p - window))) sr[c] = 0xff800000u;
                 }
             }
-            uint32_t pb[32];
+            uint32_t pb[NK / 2];
             auto exponentials = [&]() -> float {           // P against the reference in use; returns the page's sum
                 const float mu = ref == -INFINITY ? 0.f : ref;
                 const f2 nmu = pk2(-mu, -mu);
                 f2 l4[4] = {pk2(0.f, 0.f), pk2(0.f, 0.f), pk2(0.f, 0.f), pk2(0.f, 0.f)};
 #pragma unroll
-                for (int e = 0; e < 32; ++e) {
+                for (int e = 0; e < NK / 2; ++e) {
                     float x0, x1;
-                    un2(add2(pair(e), nmu), x0, x1);
+                    un2(PAIR ? pair(e) : add2(pair(e), nmu), x0, x1);
                     const float p0 = mhp_ex2(x0), p1 = mhp_ex2(x1);
                     l4[e & 3] = add2(l4[e & 3], pk2(p0, p1));
                     pb[e] = mhp_bf2(p0, p1);
@@ -301,10 +309,10 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
                 }
                 if (__any_sync(0xffffffffu, again)) {
                     float m8[8];
-    #pragma unroll
+#pragma unroll
                     for (int k = 0; k < 8; ++k) m8[k] = __uint_as_float(sr[k]);
-    #pragma unroll
-                    for (int c = 8; c < 64; ++c) m8[c & 7] = fmaxf(m8[c & 7], __uint_as_float(sr[c]));
+#pragma unroll
+                    for (int c = 8; c < NK; ++c) m8[c & 7] = fmaxf(m8[c & 7], __uint_as_float(sr[c]));
                     const float mx = fmaxf(fmaxf(fmaxf(m8[0], m8[1]), fmaxf(m8[2], m8[3])), fmaxf(fmaxf(m8[4], m8[5]), fmaxf(m8[6], m8[7])));
                     const bool grow = mx > ref + 8.0f || (ref == -INFINITY && mx != -INFINITY);
                     if (__any_sync(0xffffffffu, grow)) {
@@ -317,12 +325,12 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
                         if (j > 0) {                           // P V of the page before must be complete before U is rescaled
                             if (!tma::mbar_wait(pv_done, (uint32_t)((j - 1) & 1), abort_flag, status, 68)) { ok = false; break; }
                             tc5::fence_after();
-    #pragma unroll 1
+#pragma unroll 1
                             for (int c0 = 0; c0 < nv * DV; c0 += 32) {
                                 uint32_t orow[32];
                                 tc5::ld32(U_t + lane_off + c0, orow);
                                 tc5::wait_ld();
-    #pragma unroll
+#pragma unroll
                                 for (int c = 0; c < 32; ++c) orow[c] = __float_as_uint(__uint_as_float(orow[c]) * corr);
                                 tc5::st32(U_t + lane_off + c0, orow);
                             }
@@ -335,7 +343,8 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
             l += lpage;
             // P over this thread's own row of the scores it has read: the P V that read the P of two pages ago from this
             // buffer was issued before these scores, and the tensor core works in order
-            tc5::st32(S_t + lane_off + (uint32_t)((j & 1) * 64), pb);
+            if constexpr (PAIR) tc5::st16(S_t + lane_off + (uint32_t)((j & 1) * 64 + half * 32), pb);
+            else tc5::st32(S_t + lane_off + (uint32_t)((j & 1) * 64), pb);
             tc5::wait_st();
             tc5::fence_before();
             __syncwarp();
@@ -344,18 +353,19 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
         ok = ok && tma::mbar_wait(u_done, 0, abort_flag, status, 68);
         const size_t at = (size_t)(tok0 + row0 + row) * H + h;
         if (PAIR) {
-            // the odd pages' sums join the even pages' (both warpgroups come here, whatever happened to their waits)
+            // the groups' sums of a row come together (all of them come here, whatever happened to their waits)
             float* sums = reinterpret_cast<float*>(smem);   // (Q is not read any more: its last reader is complete, or nothing is)
-            if (wg == 1) sums[row] = l;
-            asm volatile("bar.sync 1, 256;" ::: "memory");
-            if (wg == 0) l += sums[row];
+            if (wg > 0) sums[(wg - 1) * 128 + row] = l;
+            asm volatile("bar.sync 1, %0;" :: "n"(GROUPS * 128) : "memory");
+            if (wg == 0)
+                for (int k = 0; k < GROUPS - 1; ++k) l += sums[k * 128 + row];
         }
         if (ok) {
             tc5::fence_after();
             if (row < rows && v0 == 0 && wg == 0) { ml[at * 2] = ref; ml[at * 2 + 1] = l; }
-            // (a pair of warpgroups shares the runs of 32 columns out between its two)
+            // (the warpgroups share the runs of 32 columns out)
 #pragma unroll 1
-            for (int c0 = 32 * wg; c0 < nv * DV; c0 += PAIR ? 64 : 32) {
+            for (int c0 = 32 * wg; c0 < nv * DV; c0 += 32 * GROUPS) {
                 const int n = c0 / DV, e0 = c0 % DV;
                 float* dst = u + (at * G + v0 + n) * dv + e0;
                 uint32_t orow[32];
@@ -382,12 +392,12 @@ __global__ void __launch_bounds__(PAIR ? 320 : 192, PromptSizes<D, DV, NV>::TMEM
     }
 }
 
-template <int D, int DV, int NV, bool PAIR>
+template <int D, int DV, int NV, int GROUPS>
 int launch_prompt_form(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, float* u, float* ml, const int* cu_seqlens,
                   const int* ctx_lens, const int* seq_of_token, const int* page_table, int max_pages, int n_seqs, int max_tiles,
                   int H, int G, int d, int dv, float scale, float cap, float coef, float every, int window, int n_pages,
                   int* status, cudaStream_t stream) {
-    auto kern = mixed_head_prompt_kernel<D, DV, NV, PAIR>;
+    auto kern = mixed_head_prompt_kernel<D, DV, NV, GROUPS>;
     constexpr int smem = PromptSizes<D, DV, NV>::SMEM;
     static bool configured = false;                        // per instantiation
     if (!configured) {
@@ -395,18 +405,16 @@ int launch_prompt_form(const CUtensorMap& tq, const CUtensorMap& tk, const CUten
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return gg_launch(kern, dim3(H * ((G + NV - 1) / NV), max_tiles), dim3(PAIR ? 320 : 192), smem, stream, 1, tq, tk, tv, u, ml, cu_seqlens,
+    return gg_launch(kern, dim3(H * ((G + NV - 1) / NV), max_tiles), dim3(GROUPS * 128 + 64), smem, stream, 1, tq, tk, tv, u, ml, cu_seqlens,
                      ctx_lens, seq_of_token, page_table, max_pages, n_seqs, H, G, d, dv, scale, cap, coef, every, window, n_pages,
                      status);
 }
 
 template <int D, int DV, int NV, typename... Args>
 int launch_prompt(bool no_reference, Args... args) {
-    // forms that fill tensor memory have the multiprocessor to themselves: a second softmax warpgroup has room there
-    if constexpr (PromptSizes<D, DV, NV>::TMEM == 512) {
-        if (no_reference) return launch_prompt_form<D, DV, NV, true>(args...);
-    }
-    return launch_prompt_form<D, DV, NV, false>(args...);
+    // forms that fill tensor memory have the multiprocessor to themselves, the others share it between two CTAs
+    if (no_reference) return launch_prompt_form<D, DV, NV, PromptSizes<D, DV, NV>::TMEM == 512 ? 4 : 2>(args...);
+    return launch_prompt_form<D, DV, NV, 1>(args...);
 }
 
 }  // namespace
