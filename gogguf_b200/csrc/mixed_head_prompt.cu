@@ -30,6 +30,10 @@ __device__ __forceinline__ float mhp_ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ void mhp_store8(float* dst, const uint32_t* r) {
+    asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(dst), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]),
+                 "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]) : "memory");
+}
 typedef unsigned long long f2;
 __device__ __forceinline__ f2 pk2(float lo, float hi) {
     f2 v;
@@ -148,10 +152,13 @@ __global__ void __launch_bounds__(GROUPS * 128 + 64, PromptSizes<D, DV, NV>::TME
             tma::mbar_expect_tx(q_full, Z::Q_BYTES);
 #pragma unroll
             for (int hf = 0; hf < Z::QH; ++hf) tma::load_2d(Qs + hf * Z::QBOX, &tmQ, q_full, h * d + hf * 64, tok0 + row0);
+            auto page_of = [&](int j) { return gg_page(pt, kt_first + j, max_pages, PageBounds{n_pages, status}, 53); };
+            int next = ntiles > 0 ? page_of(0) : 0;
             for (int j = 0; j < ntiles; ++j) {
                 const int s = j & 1;
                 const uint32_t ph = (uint32_t)((j >> 1) & 1) ^ 1u;
-                const int page = gg_page(pt, kt_first + j, max_pages, PageBounds{n_pages, status}, 53);
+                const int page = next;
+                if (j + 1 < ntiles) next = page_of(j + 1);     // (on its way while this page's places come free)
                 if (!tma::mbar_wait(&k_empty[s], ph, abort_flag, status, 61)) break;
                 tma::mbar_expect_tx(&k_full[s], Z::K_STAGE);
 #pragma unroll
@@ -170,48 +177,61 @@ __global__ void __launch_bounds__(GROUPS * 128 + 64, PromptSizes<D, DV, NV>::TME
             }
         }
     } else if (warp == SW + 1) {
-        if (lane == 0 && active) {
+        // All lanes walk the loop together, so that addresses and descriptors stay uniform; one elected lane issues.
+        if (active) {
             const uint32_t idesc_qk = tc5::idesc_bf16(128, 64, 0), idesc_pv = tc5::idesc_bf16(128, DV, 1);
-            const uint32_t q_a = tma::smem_u32(Qs), k_a = tma::smem_u32(Ks), v_a = tma::smem_u32(Vs);
-            bool ok = tma::mbar_wait(q_full, 0, abort_flag, status, 63);
+            const uint64_t q_d = tc5::smem_desc(tma::smem_u32(Qs), 16, 1024), k_d = tc5::smem_desc(tma::smem_u32(Ks), 16, 1024);
+            const uint64_t v_d = tc5::smem_desc(tma::smem_u32(Vs), Z::KBOX, 1024);
+            auto await = [&](uint64_t* bar, int j, int code) -> bool {      // (a lane that gives up takes the others with it)
+                return __all_sync(0xffffffffu, tma::mbar_wait(bar, (uint32_t)((j >> 1) & 1), abort_flag, status, code));
+            };
             auto issue_scores = [&](int j) -> bool {            // scores of page j into buffer j & 1
                 const int s = j & 1;
-                if (!tma::mbar_wait(&k_full[s], (uint32_t)((j >> 1) & 1), abort_flag, status, 64)) return false;
+                if (!await(&k_full[s], j, 64)) return false;
                 tc5::fence_after();
+                const uint64_t kd = k_d + (uint64_t)(s * (Z::K_STAGE >> 4));
+                if (tc5::elect_one()) {
 #pragma unroll
-                for (int ks = 0; ks < D / 16; ++ks) {
-                    const uint64_t a = tc5::smem_desc(q_a + (ks >> 2) * Z::QBOX + (ks & 3) * 32, 16, 1024);
-                    const uint64_t bb = tc5::smem_desc(k_a + s * Z::K_STAGE + (ks >> 2) * Z::KBOX + (ks & 3) * 32, 16, 1024);
-                    tc5::mma(S_t + (uint32_t)(s * 64), a, bb, idesc_qk, ks > 0 ? 1u : 0u);
+                    for (int ks = 0; ks < D / 16; ++ks) {
+                        const uint64_t qo = (uint64_t)(((ks >> 2) * Z::QBOX + (ks & 3) * 32) >> 4);
+                        const uint64_t ko = (uint64_t)(((ks >> 2) * Z::KBOX + (ks & 3) * 32) >> 4);
+                        tc5::mma(S_t + (uint32_t)(s * 64), q_d + qo, kd + ko, idesc_qk, ks > 0 ? 1u : 0u);
+                    }
+                    tc5::commit(&s_full[s]);
+                    tc5::commit(&k_empty[s]);
                 }
-                tc5::commit(&s_full[s]);
-                tc5::commit(&k_empty[s]);
+                __syncwarp();
                 return true;
             };
+            bool ok = await(q_full, 0, 63);
             if (ok && ntiles > 0) ok = issue_scores(0);
             for (int j = 0; j < ntiles && ok; ++j) {
                 // the next page's scores: their buffer was last read by the softmax of page j - 1, whose p_ready this
-                // thread has seen, and by the P V of page j - 1, which was issued before them
+                // warp has seen, and by the P V of page j - 1, which was issued before them
                 if (j + 1 < ntiles && !(ok = issue_scores(j + 1))) break;
                 const int s = j & 1;
-                if (!(ok = tma::mbar_wait(&p_ready[s], (uint32_t)((j >> 1) & 1), abort_flag, status, 65))) break;
-                if (!(ok = tma::mbar_wait(&v_full[s], (uint32_t)((j >> 1) & 1), abort_flag, status, 66))) break;
+                if (!(ok = await(&v_full[s], j, 66))) break;
+                if (!(ok = await(&p_ready[s], j, 65))) break;
                 tc5::fence_after();
+                const uint64_t vd = v_d + (uint64_t)(s * (Z::V_STAGE >> 4));
+                const uint32_t pa = S_t + (uint32_t)(s * 64), first = j > 0 ? 1u : 0u;
+                if (tc5::elect_one()) {
 #pragma unroll
-                for (int n = 0; n < NV; ++n) {
-                    if (n >= nv) break;
+                    for (int n = 0; n < NV; ++n) {
+                        if (n >= nv) break;
 #pragma unroll
-                    for (int kk = 0; kk < 4; ++kk) {
-                        const uint64_t bb = tc5::smem_desc(v_a + s * Z::V_STAGE + n * Z::V_HEAD + kk * 2048, Z::KBOX, 1024);
-                        // (16 keys of P are 8 columns; each group's lie over the scores it alone has read)
-                        tc5::mma_a_tmem(U_t + (uint32_t)(n * DV), S_t + (uint32_t)(s * 64 + (PAIR ? (kk >> 1) * 32 + (kk & 1) * 8 : kk * 8)), bb, idesc_pv,
-                                        (j > 0 || kk > 0) ? 1u : 0u);
+                        for (int kk = 0; kk < 4; ++kk)
+                            // (16 keys of P are 8 columns; each group's lie over the scores it alone has read)
+                            tc5::mma_a_tmem(U_t + (uint32_t)(n * DV), pa + (uint32_t)(PAIR ? (kk >> 1) * 32 + (kk & 1) * 8 : kk * 8),
+                                            vd + (uint64_t)((n * Z::V_HEAD + kk * 2048) >> 4), idesc_pv, kk > 0 ? 1u : first);
                     }
+                    tc5::commit(pv_done);
+                    tc5::commit(&v_empty[s]);
                 }
-                tc5::commit(pv_done);
-                tc5::commit(&v_empty[s]);
+                __syncwarp();
             }
-            if (ok) tc5::commit(u_done);
+            if (ok && tc5::elect_one()) tc5::commit(u_done);
+            __syncwarp();
         }
     } else if (active) {
         const int row = threadIdx.x & 127;                 // query row of the tile = tensor-memory lane
@@ -373,8 +393,8 @@ __global__ void __launch_bounds__(GROUPS * 128 + 64, PromptSizes<D, DV, NV>::TME
                 tc5::wait_ld();
                 if (row < rows) {
 #pragma unroll
-                    for (int c = 0; c < 32; c += 4)
-                        if (e0 + c < dv) *reinterpret_cast<uint4*>(dst + c) = make_uint4(orow[c], orow[c + 1], orow[c + 2], orow[c + 3]);
+                    for (int c = 0; c < 32; c += 8)            // (dv is a multiple of 8: whole sectors of 32 bytes)
+                        if (e0 + c < dv) mhp_store8(dst + c, orow + c);
                 }
             }
         }
@@ -437,7 +457,7 @@ GG_API gg_mixed_head_prompt(const void* row, long long ld, const void* k_pool, c
     if (!gg_mixed_head_prompt_takes(H, G, d, dv, page_size) || max_tiles > 65535 || n_pages <= 0 || status == nullptr || u == nullptr ||
         ml == nullptr || (ld % 8) || ld < (long long)H * d || cap < 0.f || (coef != 0.f && !(every > 0.f)) ||
         (value_heads != 1 && value_heads != 2 && !(value_heads == 4 && dv <= 64)) ||
-        (((uintptr_t)row | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)u) & 15))
+        (((uintptr_t)row | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) || (((uintptr_t)u) & 31))
         return GG_ERR_ARG;
     CUtensorMap tq, tk, tv;
     int rc;
