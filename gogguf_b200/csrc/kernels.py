@@ -588,8 +588,10 @@ def mixed_head_decode_takes(heads: int, kv_heads: int, d: int, dv: int, page_siz
 
 
 def mixed_head_decode_splits(n_tokens: int, kv_heads: int, max_ctx: int) -> int:
-    """Into how many shares the pages of a (token, kv head) are cut: towards three CTAs a multiprocessor."""
-    return int(max(1, min(32, 444 // max(n_tokens * kv_heads, 1), -(-max_ctx // 64))))
+    """Into how many shares the pages of a (token, kv head) are cut: three CTAs a multiprocessor, and two
+    shares up to five."""
+    ctas = max(n_tokens * kv_heads, 1)
+    return int(max(1, min(32, max(444 // ctas, min(2, 740 // ctas)), -(-max_ctx // 64))))
 
 
 def mixed_head_attention_decode(row: torch.Tensor, g_off: int, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,

@@ -182,8 +182,9 @@ __global__ void __launch_bounds__(128) mixed_head_scores_kernel(
     }
 }
 
-// HP: query heads of a kv head, rounded up to 4, 8 or 16.
-template <int DV, int HP>
+// HP: query heads of a kv head, rounded up to 4, 8 or 16.  STAGED: the scores come through the ring with the values (models
+// of few heads; the ring's stages are then longer by 64 bytes a head).
+template <int DV, int HP, bool STAGED>
 __global__ void __launch_bounds__(128) mixed_head_values_kernel(
     const float* scores, long long ctx_pad, const float* ml, const bf16* v_pool, float* part, const float* __restrict__ talk,
     const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ page_table, int max_pages,
@@ -197,6 +198,7 @@ __global__ void __launch_bounds__(128) mixed_head_values_kernel(
     bf16* Ws = rings + 4 * MD_STAGES * MdRing<DV>::STAGE + warp * 2 * 16 * WL;          // [2 terms][16][WL]
     float* tk = reinterpret_cast<float*>(rings + 4 * MD_STAGES * MdRing<DV>::STAGE + 4 * 2 * 16 * WL);     // [H][HP]
     float* fm = tk + H * HP;                                        // [H][2]: maximum, 1 / sum
+    float* Ss = fm + 2 * ((H + 1) & ~1) + warp * MD_STAGES * H * 16;            // STAGED: [stage][H][16]
     const int t = blockIdx.x, g = blockIdx.y, hpg = H / G;
     const int b = seq_of_token[t];
     if (b < 0) return;
@@ -215,6 +217,11 @@ __global__ void __launch_bounds__(128) mixed_head_values_kernel(
         if (i < n) {
             const int page = gg_page(pt, j_lo + i, max_pages, pb, 53);
             ring.load(i % MD_STAGES, v_pool + (((size_t)page * G + g) * 64 + warp * 16) * dv);
+            if (STAGED) {
+                const float* src = scores + (size_t)t * H * ctx_pad + (size_t)(j_lo + i) * 64 + warp * 16;
+                for (int x = lane; x < H * 4; x += 32)
+                    md_cp16(Ss + (i % MD_STAGES) * H * 16 + x * 4, src + (size_t)(x >> 2) * ctx_pad + (x & 3) * 4);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -238,14 +245,19 @@ __global__ void __launch_bounds__(128) mixed_head_values_kernel(
     const float* sp = scores + (size_t)t * H * ctx_pad + warp * 16 + kk;
     for (int i = 0; i < n; ++i) {
         fetch(i + MD_STAGES - 1);
+        if (STAGED) {
+            asm volatile("cp.async.wait_group %0;" :: "n"(MD_STAGES - 1) : "memory");
+            __syncwarp();
+        }
         // this lane's key: every second head's weight there, its share of the mixed weights of all rows
         float w[HP];
 #pragma unroll
         for (int r = 0; r < HP; ++r) w[r] = 0.f;
-        const float* sk = sp + (size_t)(j_lo + i) * 64;
+        const float* sk = STAGED ? Ss + (i % MD_STAGES) * H * 16 + kk : sp + (size_t)(j_lo + i) * 64;
+        const long long sstep = STAGED ? 16 : ctx_pad;
 #pragma unroll 8
         for (int gh = half; gh < H; gh += 2) {
-            const float p = md_ex2(sk[(size_t)gh * ctx_pad] - fm[2 * gh]) * fm[2 * gh + 1];
+            const float p = md_ex2(sk[gh * sstep] - fm[2 * gh]) * fm[2 * gh + 1];
             const float4* tr = reinterpret_cast<const float4*>(tk + gh * HP);
 #pragma unroll
             for (int q = 0; q < HP / 4; ++q) {
@@ -260,7 +272,7 @@ __global__ void __launch_bounds__(128) mixed_head_values_kernel(
             const bf16 hi = __float2bfloat16_rn(w[r]);
             Ws[half * 16 * WL + r * WL + kk] = half ? __float2bfloat16_rn(w[r] - __bfloat162float(hi)) : hi;
         }
-        asm volatile("cp.async.wait_group %0;" :: "n"(MD_STAGES - 1) : "memory");
+        if (!STAGED) asm volatile("cp.async.wait_group %0;" :: "n"(MD_STAGES - 1) : "memory");
         __syncwarp();
         uint32_t ah[4], al[4];
         md_ldsm4(ah, Ws + (lane & 15) * WL + (lane >> 4) * 8);
@@ -349,21 +361,22 @@ static int md_scores(int ntok, int H, int G, int nsplit, cudaStream_t stream, co
                      ml, positions, seq_of_token, page_table, max_pages, H, G, d, scale, cap, coef, every, window, nsplit, pb);
 }
 
-template <int DV, int HP>
+template <int DV, int HP, bool STAGED>
 static int md_values(int ntok, int H, int G, int nsplit, cudaStream_t stream, const float* scores, long long ctx_pad, const float* ml,
                      const bf16* v_pool, float* part, const float* talk, const int* positions, const int* seq_of_token,
                      const int* page_table, int max_pages, int dv, float one, int window, const PageBounds pb) {
     size_t smem = (size_t)(4 * MD_STAGES * MdRing<DV>::STAGE + 4 * 2 * 16 * 24) * sizeof(bf16);
     static_assert((size_t)4 * MD_STAGES * MdRing<DV>::STAGE * sizeof(bf16) >= (size_t)4 * HP * DV * sizeof(float),
                   "the rings must hold the warps' sums");
-    smem += (size_t)H * (HP + 2) * sizeof(float);
+    smem += ((size_t)H * HP + 2 * ((H + 1) & ~1)) * sizeof(float);
+    if (STAGED) smem += (size_t)4 * MD_STAGES * H * 16 * sizeof(float);
     static size_t configured = 0;
     if (smem > configured) {
-        cudaError_t e = cudaFuncSetAttribute(mixed_head_values_kernel<DV, HP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(mixed_head_values_kernel<DV, HP, STAGED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = smem;
     }
-    return gg_launch(mixed_head_values_kernel<DV, HP>, dim3(ntok, G, nsplit), dim3(128), smem, stream, 1, scores, ctx_pad, ml, v_pool,
+    return gg_launch(mixed_head_values_kernel<DV, HP, STAGED>, dim3(ntok, G, nsplit), dim3(128), smem, stream, 1, scores, ctx_pad, ml, v_pool,
                      part, talk, positions, seq_of_token, page_table, max_pages, H, G, dv, one, window, nsplit, pb);
 }
 
@@ -389,12 +402,14 @@ GG_API gg_mixed_head_decode(const void* row, long long ld, int g_off, const void
 #undef MD_S
     if (rc != 0) return rc;
     const int hpg = H / G;
-#define MD_V(V_, P_) md_values<V_, P_>(ntok, H, G, nsplit, stream, (const float*)scores, ctx_pad, (const float*)ml, vp, part, talk, \
+#define MD_V(V_, P_) (H <= 32 ? MD_VS(V_, P_, true) : MD_VS(V_, P_, false))
+#define MD_VS(V_, P_, S_) md_values<V_, P_, S_>(ntok, H, G, nsplit, stream, (const float*)scores, ctx_pad, (const float*)ml, vp, part, talk, \
                                        positions, seq_of_token, page_table, max_pages, dv, one, window, pb)
 #define MD_VH(V_) (hpg <= 4 ? MD_V(V_, 4) : (hpg <= 8 ? MD_V(V_, 8) : MD_V(V_, 16)))
     rc = dv <= 32 ? MD_VH(32) : (dv <= 64 ? MD_VH(64) : MD_VH(128));
 #undef MD_VH
 #undef MD_V
+#undef MD_VS
     if (rc != 0) return rc;
     const int chunks = (H * dv + 511) / 512;
     return gg_launch(mixed_head_merge_kernel, dim3(ntok, chunks > 64 ? 64 : chunks), dim3(128), 0, stream, 1, (const float*)part, r, ld,
