@@ -5,7 +5,7 @@
 //   p_h(i, j) = exp(s_h(i, j)) / (one + sum over the seen j of exp(s_h(i, j)))          one: 0 or 1
 //   o_h(i)    = gate_h(i) sum_j ( sum_g T[h, g] p_g(i, j) ) v_g(h),j
 //
-// Query head h reads kv head g(h) = h / (H / G).  tau(i) = 1 + coef ln(floor((pos_i + 1) / every) + 1) is the query
+// Query head h reads kv head g(h) = h / (H / G).  tau(i) = 1 + coef log(1 + floor((pos_i + 1) / every)) is the query
 // temperature (coef 0: none).  gate_h(i) = sigmoid of a logit per token and head (null: no gate).  The mix is linear
 // in the weights, so it may also be applied to the heads' results on every kv head's values:
 //
@@ -19,7 +19,7 @@
 
 // ----------------------------------------------------------------------------- keys and values into the cache
 // k goes into the pool as it is.  v: each head's run of dv is divided by its root mean square (unit != 0), then mixed
-// with the step's first such layer's values, v <- (1 - lambda) v + lambda first, where `first` is given and `keep` is
+// with the step's first such layer's values, v <- v + lambda (first - v), where `first` is given and `keep` is
 // null; with `keep` the layer is the first one and leaves its values there ([T][G][dv] float32).
 template <typename T>
 __global__ void __launch_bounds__(128) head_kv_prep_kernel(const T* row, long long ld, int k_off, int v_off, T* k_pool,

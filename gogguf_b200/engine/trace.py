@@ -42,9 +42,11 @@ class TraceRunner:
     def __init__(self, model: Model, max_tokens: int, out_dir: str, graphs: bool = True, layers: bool = False):
         self.model = model
         # `max_tokens` counts tokens, a sequence holds whole pages: a quarter more pages than the count alone asks
-        # for, and 64, leave room for the live requests' partly filled last pages (many short requests have little else)
+        # for, and 64, leave room for the live requests' partly filled last pages (many short requests have little
+        # else); a count that fits one page is taken as it stands
         pages = -(-max_tokens // PAGE_SIZE)
-        self.cache = model.new_cache((pages + pages // 4 + 64) * PAGE_SIZE)
+        spare = pages // 4 + 64 if pages > 1 else 0
+        self.cache = model.new_cache((pages + spare) * PAGE_SIZE)
         if graphs and model.rt.device.type == "cuda":
             from .graphs import GraphStepper
             self.stepper: Stepper = GraphStepper(model, self.cache)
@@ -116,7 +118,7 @@ def main(argv: Optional[list] = None) -> int:
     ap.add_argument("--dtype", required=True, choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder for <step>.f32 files")
     ap.add_argument("--max-tokens", type=int, required=True,
-                    help="most tokens live requests hold at any time (the cache holds a quarter more pages of 64, and 64)")
+                    help="most tokens live requests hold at any time (beyond one page of 64 the cache holds a quarter more pages, and 64)")
     ap.add_argument("--device", default="cuda:0")
     ap.add_argument("--graphs", dest="graphs", action="store_true", default=True,
                     help="replay plain decode steps as captured CUDA graphs, as generation does (default)")

@@ -2,10 +2,10 @@
 temperature instead of a rotation.
 
     q = W_q h + b_q [heads x head_dim],  k = W_k h + b_k [kv_heads x head_dim],  v = W_v h + b_v [kv_heads x value_dim]
-    q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)                     (query_temperature)
+    q at position p is multiplied by 1 + coef log(1 + floor((p + 1) / every))                   (query_temperature)
     v: each head's run divided by its root mean square over value_dim                            (unit_values)
-    v <- (1 - lambda) v + lambda v_first, v_first being the values that the step's source layer made for the same
-        token, lambda a stored number                                                            (value_mix)
+    v <- v + mu (v0 - v), v0 being the values that the step's source layer made for the same token, mu a stored
+        number                                                                                   (value_mix)
     s = cap tanh(scale q . k / cap),   p_h(i, j) = exp(s_j) / (one + sum_j exp(s_j))             (softcap, extra_one)
     o_h = sigmoid(W_g h)_h * sum_j ( sum_g T[h, g] p_g(i, j) ) v_j                               (talking, head_gate)
     y = W_o concat_h o + b_o
@@ -19,7 +19,8 @@ values are the ones later layers mix in, "mix"), extra_one, talking (False: T is
 head_gate, window (absent: none), names.
 
 Temperature, scores, softmax, mixing and gate are float32 in both compute paths.  In the bfloat16 path head sizes of up
-to 128 run on the tensor cores (prompts on tcgen05, short stretches and decode steps on mma.sync); GOGGUF_B200_MIXED_HEAD_MMA=0 keeps the plain kernel, their twin.
+to 128 run on the tensor cores (prompts on tcgen05, short stretches and decode steps on mma.sync);
+GOGGUF_B200_MIXED_HEAD_MMA=0 keeps the plain kernel, their twin.
 """
 from __future__ import annotations
 

@@ -40,7 +40,7 @@ def _gen(seed):
 
 
 # ----------------------------------------------------------------------------------------------- mechanisms alone
-@pytest.mark.parametrize("N,K", [(448, 256), (1000, 512), (2056, 1024), (20, 80), (137, 64)])
+@pytest.mark.parametrize("N,K", [(456, 264), (1000, 512), (2056, 1024), (20, 80), (137, 64)])
 def test_bias_inside_the_products(N, K):
     """Every form of the product: decode (with and without a K split), prompts of several lengths, adding into float32
     rows with and without row statistics, a folded norm, the plain kernel."""
@@ -121,7 +121,7 @@ def test_keys_and_values_into_the_cache(dt, G, d, dv, unit):
             assert rel_err(keep[:T - 1], own[:T - 1].reshape(T - 1, -1)) < 1e-5 and float(keep[T - 1].min()) == 9.0
 
 
-def _mixed_reference(q, k, v, gate, talk, pos, lens, scale, cap, coef, every, one):
+def _mixed_reference(q, k, v, gate, talk, pos, lens, scale, cap, coef, every, one, window=0):
     """q [T, H, d] of the step's tokens, k [b][n, G, d] and v [b][n, G, dv] everything each sequence has cached."""
     out = []
     t = 0
@@ -133,6 +133,8 @@ def _mixed_reference(q, k, v, gate, talk, pos, lens, scale, cap, coef, every, on
             p = int(pos[t])
             tau = plain.query_temperature(p + 1, coef, every)[p] if coef else 1.0
             s = plain.bounded(torch.einsum("hd,jhd->hj", q[t] * tau, k[b][:p + 1][:, own]) * scale, cap)
+            if window:
+                s[:, :max(0, p - window + 1)] = -math.inf
             a = plain.weights_with_one(s) if one else torch.softmax(s, dim=-1)
             a = torch.einsum("hg,gj->hj", talk, a)
             o = torch.einsum("hj,jhe->he", a, v[b][:p + 1][:, own])
@@ -180,7 +182,7 @@ def test_prompt_form_with_scores_of_every_size(cap, factor):
 
 
 @pytest.mark.parametrize("H,G,d,dv,cap,temp,one,gated", [
-    (4, 2, 64, 64, 20.0, (0.3, 16.0), True, True), (6, 2, 12, 20, 5.0, (0.5, 7.0), True, True),
+    (8, 4, 64, 64, 18.0, (0.25, 16.0), True, True), (6, 2, 12, 20, 5.0, (0.5, 7.0), True, True),
     (8, 1, 32, 128, 0.0, None, True, True), (3, 3, 128, 40, 10.0, (1.0, 1.0), True, False),
     (5, 1, 40, 32, 30.0, (-0.1, 3.0), False, True), (12, 4, 64, 96, 15.0, None, True, True),
     (32, 8, 128, 128, 25.0, (0.1, 64.0), True, True), (1, 1, 16, 16, 3.0, None, True, True), (24, 1, 8, 8, 0.0, (0.2, 9.0), True, True)])
@@ -203,7 +205,8 @@ def test_attention_with_mixed_heads_alone(H, G, d, dv, cap, temp, one, gated):
     done = [0, 0, 0]
     g_off = H * d + 8 if gated else -1
     width = H * d + 8 + (H + 7) // 8 * 8
-    kw = dict(cap=cap, coef=coef, every=every, one=one)
+    window = {12: 70, 3: 100}.get(H, 0)
+    kw = dict(cap=cap, coef=coef, every=every, one=one, window=window)
     for lens in ((130, 1, 67), (65, 180, 2), (1, 1, 1), (2, 1, 3), (1, 1, 1)):
         cu, sot = _batch(lens)
         T = sum(lens)
@@ -211,7 +214,7 @@ def test_attention_with_mixed_heads_alone(H, G, d, dv, cap, temp, one, gated):
         row = torch.randn(T, width, generator=g).to(torch.bfloat16)
         want = _mixed_reference(row[:, :H * d].double().reshape(T, H, d), ks, vs,
                                 row[:, g_off:g_off + H].double() if gated else None, talk.double(), pos, lens, scale, cap, coef,
-                                every, one).reshape(T, H * dv)
+                                every, one, window).reshape(T, H * dv)
         for dt in (torch.float32, torch.bfloat16):
             o = torch.empty(T, H * dv, dtype=dt, device=DEV)
             K.mixed_head_attention_plain(row.to(dt).to(DEV), g_off, kf.to(dt).to(DEV), vf.to(dt).to(DEV), o, talk.to(DEV), _i32(pos),
@@ -385,6 +388,58 @@ def test_one_mechanism_in_a_layer_of_its_own(tmp_path_factory, name, dtype):
         out = run_cut(st, cache, tokens if cuts else tokens[:70], cuts)
         ref = want if cuts else want[:70]
         assert close(out, ref, dtype, own32=own32[:ref.shape[0]], gauge=got[:ref.shape[0]]), (rel_err(out, ref), name, cuts)
+
+
+def test_attention_with_its_options_left_out(tmp_path_factory):
+    """Another design's use of the mixer: no biases, no mixing of heads, no gate, no one in the denominator, values as they
+    are.  The same tensors with the identity, zeros and closed options through the plain functions."""
+    from gogguf_b200.config.spec import BlockSpec, PartSpec
+    from gogguf_b200.engine import Model, StepEntry, Stepper
+    import dataclasses
+    folder = make_folder(tmp_path_factory.getbasetemp(), "S", "float32")
+    cfg, w = read_folder(folder)
+    from gogguf_b200.config import config_from_dict
+    spec = config_from_dict(cfg).to_spec()
+    blocks, drop = [], []
+    for i, b in enumerate(spec.blocks):
+        ps = b.parts["mixer"]
+        if ps.kind == "mixed_head_attention":
+            off = dict(bias=False, talking=False, head_gate=False, extra_one=False, unit_values=False, value_mix=None)
+            b = BlockSpec(b.arrangement, {**b.parts, "mixer": PartSpec(kind=ps.kind, prefix=ps.prefix, params={**ps.params, **off})})
+            drop += [ps.prefix + n for n in ("q.b", "k.b", "v.b", "o.b", "talk", "g", "vmix")]
+        blocks.append(b)
+    spec = dataclasses.replace(spec, blocks=tuple(blocks))
+    tensors = {n: t for n, t in w.items() if n not in drop}
+    tokens = random_tokens(cfg["vocab"], 90, seed=2)
+    eps = cfg["norm"]["eps"]
+
+    def bare(m, p, h):
+        n, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        q, k, v = (plain.linear(h, w, p + x) for x in "qkv")
+        qt = m.get("q_temp")
+        tau = plain.query_temperature(n, qt["coef"], qt["every"]) if qt else torch.ones(n, dtype=torch.float64)
+        own = [x // (H // G) for x in range(H)]
+        s = torch.einsum("ihd,jhd->hij", q.reshape(n, H, d) * tau[:, None, None], k.reshape(n, G, d)[:, own]) * m["scale"]
+        a = torch.softmax(plain.bounded(s, m.get("softcap") or 0.0) + plain.unseen(n, h.dtype), dim=-1)
+        return plain.linear(torch.einsum("hij,jhe->ihe", a, v.reshape(n, G, dv)[:, own]).reshape(n, H * dv), w, p + "o")
+
+    E = w["embed"].double()
+    x = E[torch.tensor(tokens)] * cfg["embedding"]["scale"]
+    for i, l in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        h = plain.norm_about_one(x, w[p + "norm1"], eps)
+        y = (bare(l["mixer"], p + "mix.", h) if l["type"] == "attention" else plain.latent_attention(l["mixer"], w, p + "mix.", h, eps))
+        x = x + plain.norm_about_one(y, w[p + "norm1b"], eps)
+        if l["mlp"] is not None:
+            y = plain.feed_forward(w, p + "mlp.", plain.norm_about_one(x, w[p + "norm2"], eps))
+            x = x + plain.norm_about_one(y, w[p + "norm2b"], eps)
+    want = plain.norm_about_one(x, w["final.norm"], eps) @ E.t() * cfg["logit_scale"]
+    for dtype in ("float32", "bfloat16"):
+        m = Model(spec, tensors, dtype=dtype)
+        cache = m.new_cache(max_tokens=512)
+        for cuts in ([90], [64, 2]):
+            got = run_cut(Stepper(m, cache), cache, tokens, cuts)
+            assert rel_err(got, want) < (1e-4 if dtype == "float32" else 1e-1), (dtype, cuts, rel_err(got, want))
 
 
 # ----------------------------------------------------------------------------------------------- whole models
