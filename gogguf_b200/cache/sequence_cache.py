@@ -2,12 +2,13 @@
 
 What each scheduled layer needs is asked of its mixer as a *request*:
 
-* `KVRequest(num_kv_heads, head_dim, window, value_dim)` - keys and values of every position
-  (window None) or of the last `window` positions.  Layers with equal requests form a *group* with
+* `KVRequest(num_kv_heads, head_dim, window, value_dim, chunk)` - keys and values of every position
+  (window None) or of the last `window` positions, or (chunk) of the positions' own chunk, the runs of `chunk`
+  positions counted from the sequence's start.  Layers with equal requests form a *group* with
   storage of its own: pools ``k [layer_in_group][page][kv_head][page_size][head_dim]``, ``v`` alike
   with `value_dim` (the head size of the keys unless given) and, per slot, the list of pages that
-  hold its positions.  A windowed group gives pages back as soon as every position in them has left
-  the window.
+  hold its positions.  A windowed or chunked group gives pages back as soon as no position to come
+  reads any position in them.
 * `LatentRequest(width, window)` - one vector per position (latent attention caches its compressed
   key/value vector and the shared rotated key part instead of per-head keys and values); paged and
   windowed like the above, pool ``[layer_in_group][page][page_size][width]``.
@@ -58,6 +59,7 @@ class KVRequest:
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None      # head size of the values where it differs from the keys'
+    chunk: Optional[int] = None          # a position reads only its own chunk of this many positions
 
 
 @dataclass(frozen=True)
@@ -148,16 +150,18 @@ class CacheStore:
 class PagedStore(CacheStore):
     """Page bookkeeping for per-token storage: a free list of pages and, per slot, the pages that hold
     its positions.  A subclass allocates its tensors (indexed ``[layer_in_store][page]...``) and
-    implements `view`; an optional `window` gives pages back once every position in them has left it."""
+    implements `view`; an optional `window` (or `chunk`) gives pages back once no position to come reads them."""
 
     paged = True
 
-    def __init__(self, request, entries: List[int], n_pages: int, page_size: int, window: Optional[int] = None):
+    def __init__(self, request, entries: List[int], n_pages: int, page_size: int, window: Optional[int] = None,
+                 chunk: Optional[int] = None):
         self.request = request
         self.entries = list(entries)          # schedule entries that own a layer of this store
         self.page_size = page_size
         self.n_pages = n_pages
         self.window = window
+        self.chunk = chunk
         self.pages = FreeList(n_pages, "page")
         self.seq_pages: Dict[int, List[int]] = {}   # slot -> page id per page index (-1 once given back)
         self.index = -1                        # position among the cache's paged stores (set by the cache):
@@ -174,6 +178,15 @@ class PagedStore(CacheStore):
             if not is_open(s):
                 raise CacheError(f"pages are listed for slot {s}, which is not open")
 
+    def first_needed(self, length: int) -> int:
+        """The first position that a token at position `length` reads."""
+        first = 0
+        if self.window is not None:
+            first = max(first, length - self.window + 1)
+        if self.chunk is not None:
+            first = max(first, length // self.chunk * self.chunk)
+        return first
+
     def pages_needed(self, slot: int, new_len: int) -> int:
         have = len(self.seq_pages.get(slot, ()))
         want = (new_len + self.page_size - 1) // self.page_size
@@ -185,11 +198,10 @@ class PagedStore(CacheStore):
             self.seq_pages.setdefault(slot, []).extend(self.pages.take_many(n))
 
     def trim(self, slot: int, length: int) -> None:
-        """Windowed group: give back pages all of whose positions are below length - window + 1."""
-        w = self.window
-        if w is None:
+        """Windowed or chunked group: give back pages all of whose positions lie before what the next token reads."""
+        if self.window is None and self.chunk is None:
             return
-        first_needed = length - w + 1
+        first_needed = self.first_needed(length)
         pl = self.seq_pages.get(slot, [])
         for idx, pg in enumerate(pl):
             if (idx + 1) * self.page_size > first_needed:
@@ -200,11 +212,10 @@ class PagedStore(CacheStore):
 
     def can_shorten(self, slot: int, length: int) -> bool:
         """Are the positions that a token at position `length` reads still held?"""
-        w = self.window
-        if w is None:
+        if self.window is None and self.chunk is None:
             return True
         pl = self.seq_pages.get(slot, [])
-        first_needed = max(0, length - w + 1)
+        first_needed = self.first_needed(length)
         last = (length + self.page_size - 1) // self.page_size
         return all(pg >= 0 for pg in pl[first_needed // self.page_size:last])
 
@@ -241,7 +252,7 @@ class KVGroup(PagedStore):
 
     def __init__(self, request: KVRequest, entries: List[int], n_pages: int, page_size: int,
                  dtype: torch.dtype, device, max_slots: int = 0):
-        super().__init__(request, entries, n_pages, page_size, window=request.window)
+        super().__init__(request, entries, n_pages, page_size, window=request.window, chunk=request.chunk)
         lead = (len(entries), n_pages, request.num_kv_heads, page_size)
         # zero-filled once: a page that is handed out again holds old finite numbers, never NaN patterns
         self.k = torch.zeros(lead + (request.head_dim,), dtype=dtype, device=device)

@@ -8,6 +8,7 @@ from .sokirax import SokiraxConfig
 from .felolorn import FelolornConfig
 from .dinuzen import DinuzenConfig
 from .kulesun import KulesunConfig
+from .niresun import NiresunConfig
 
 __all__ = ["ConfigError", "config_from_dict", "load_config", "register_architecture", "registered_architectures",
-           "BlockSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule", "Qwen3Config", "GigopelConfig", "SokiraxConfig", "FelolornConfig", "DinuzenConfig", "KulesunConfig"]
+           "BlockSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "default_schedule", "Qwen3Config", "GigopelConfig", "SokiraxConfig", "FelolornConfig", "DinuzenConfig", "KulesunConfig", "NiresunConfig"]

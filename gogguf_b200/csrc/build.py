@@ -59,6 +59,8 @@ MODULES: Dict[str, str] = {
     "retention": "retention.cu",
     "recurrence": "recurrence.cu",
     "diag_recurrence": "diag_recurrence.cu",
+    "selective_scan": "selective_scan.cu",
+    "matrix_memory": "matrix_memory.cu",
     "diff_attention": "diff_attention.cu",
     "mixed_head_attention": "mixed_head_attention.cu",
     "mixed_head_prompt": "mixed_head_prompt.cu",

@@ -8,6 +8,8 @@
 // (angles in float64); the residual stream is float32 in both precisions.
 #include "common.cuh"
 
+#define CONV_MAX_TAPS 16
+
 // ----------------------------------------------------------------------------- embedding
 template <typename TW>
 __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* tokens,
@@ -131,6 +133,139 @@ GG_API gg_rmsnorm(const float* x, const int* rows, const float* w, void* out, in
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     GG_DISPATCH_DTYPE(out_dtype, TO,
         gg_launch(rmsnorm_kernel<TO>, dim3(R), dim3(threads), 0, stream, 1, x, rows, w, (TO*)out, H, eps));
+    return gg_last_error();
+}
+
+// ----------------------------------------------------------------------------- dynamic tanh
+// out[r, :] = tanh(alpha * x[src(r), :]) * w + b with a scalar alpha: a norm without mean or variance.  src(r) = rows ?
+// rows[r] : r; a negative source row gives a zero row.  One block per row; V columns a thread at a time (4: 16-byte
+// accesses).
+template <typename TO, int V> __device__ __forceinline__ void store_row_v(TO* o, const float* v);
+template <> __device__ __forceinline__ void store_row_v<float, 1>(float* o, const float* v) { o[0] = v[0]; }
+template <> __device__ __forceinline__ void store_row_v<bf16, 1>(bf16* o, const float* v) { o[0] = __float2bfloat16_rn(v[0]); }
+template <> __device__ __forceinline__ void store_row_v<float, 4>(float* o, const float* v) {
+    *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <> __device__ __forceinline__ void store_row_v<bf16, 4>(bf16* o, const float* v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(o) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+template <int V> __device__ __forceinline__ void load_row_v(const float* p, float* v) {
+    if (V == 4) { const float4 a = *reinterpret_cast<const float4*>(p); v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; }
+    else v[0] = p[0];
+}
+
+template <typename TO, int V>
+__global__ void __launch_bounds__(256) dynamic_tanh_kernel(const float* x, const int* __restrict__ rows, float alpha,
+                                                           const float* __restrict__ w, const float* __restrict__ b,
+                                                           TO* __restrict__ out, int H) {
+    pdl_launch();
+    pdl_wait();
+    const int r = blockIdx.x, src = rows ? rows[r] : r;
+    for (int i = V * (blockIdx.y * blockDim.x + threadIdx.x); i < H; i += V * gridDim.y * blockDim.x) {
+        float v[V], ww[V], bb[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = 0.f;
+        if (src >= 0) {
+            load_row_v<V>(x + (size_t)src * H + i, v);
+            load_row_v<V>(w + i, ww);
+            load_row_v<V>(b + i, bb);
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[k] = fmaf(tanhf(alpha * v[k]), ww[k], bb[k]);
+        }
+        store_row_v<TO, V>(out + (size_t)r * H + i, v);
+    }
+}
+
+GG_API gg_dynamic_tanh(const float* x, const int* rows, float alpha, const float* w, const float* b, void* out, int out_dtype,
+                       int R, int H, cudaStream_t stream) {
+    if (R <= 0) return 0;
+    if (H <= 0 || w == nullptr || b == nullptr) return GG_ERR_ARG;
+    const bool vec = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+    const int per = vec ? 1024 : 256;
+    const dim3 grid(R, min((H + per - 1) / per, 65535));
+    GG_DISPATCH_DTYPE(out_dtype, TO,
+        if (vec) gg_launch(dynamic_tanh_kernel<TO, 4>, grid, dim3(256), 0, stream, 1, x, rows, alpha, w, b, (TO*)out, H);
+        else gg_launch(dynamic_tanh_kernel<TO, 1>, grid, dim3(256), 0, stream, 1, x, rows, alpha, w, b, (TO*)out, H));
+    return gg_last_error();
+}
+
+// ----------------------------------------------------------------------------- a sum of normed parts, added
+// x[r, :] += sum_k y_k[r, :] / sqrt(mean(y_k[r, :]^2) + eps_k) * w_k for up to NORMED_MAX parts (y [parts][rows][H],
+// w [parts][H] with any factor of a part's already in it), all float32; y is left zeroed.  With hout the updated row's
+// dynamic tanh (alpha, nw, nb) is left there in the compute dtype too, so the norm that comes next needs no kernel of
+// its own.  One block per row.
+#define NORMED_MAX 4
+struct NormedEps { float v[NORMED_MAX]; };
+
+template <typename TO, int V>
+__global__ void __launch_bounds__(256) normed_sum_kernel(float* x, float* y, const float* __restrict__ w, int parts, int H,
+                                                         long long part_stride, const NormedEps eps, TO* __restrict__ hout,
+                                                         float alpha, const float* __restrict__ nw, const float* __restrict__ nb) {
+    pdl_launch();
+    pdl_wait();
+    __shared__ float red[33];
+    const size_t r = blockIdx.x;
+    float f[NORMED_MAX];
+    for (int k = 0; k < parts; ++k) {
+        const float* yr = y + k * part_stride + r * H;
+        float ss = 0.f;
+        for (int i = V * threadIdx.x; i < H; i += V * blockDim.x) {
+            float v[V];
+            load_row_v<V>(yr + i, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+        }
+        ss = block_sum(ss, red);
+        const float g = 1.0f / sqrtf(ss / (float)H + eps.v[k]);
+#pragma unroll
+        for (int j = 0; j < NORMED_MAX; ++j)
+            if (j == k) f[j] = g;
+    }
+    float zero[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) zero[e] = 0.f;
+    for (int i = V * threadIdx.x; i < H; i += V * blockDim.x) {
+        float a[V];
+        load_row_v<V>(x + r * H + i, a);
+#pragma unroll
+        for (int k = 0; k < NORMED_MAX; ++k) {
+            if (k < parts) {
+                float v[V], ww[V];
+                float* yr = y + k * part_stride + r * H + i;
+                load_row_v<V>(yr, v);
+                load_row_v<V>(w + (size_t)k * H + i, ww);
+#pragma unroll
+                for (int e = 0; e < V; ++e) a[e] = fmaf(v[e] * f[k], ww[e], a[e]);
+                store_row_v<float, V>(yr, zero);
+            }
+        }
+        store_row_v<float, V>(x + r * H + i, a);
+        if (hout != nullptr) {
+            float ww[V], bb[V];
+            load_row_v<V>(nw + i, ww);
+            load_row_v<V>(nb + i, bb);
+#pragma unroll
+            for (int e = 0; e < V; ++e) a[e] = fmaf(tanhf(alpha * a[e]), ww[e], bb[e]);
+            store_row_v<TO, V>(hout + r * H + i, a);
+        }
+    }
+}
+
+// hout (rows of H numbers in `out_dtype`) may be null, and nw and nb with it.
+GG_API gg_normed_sum(float* x, float* y, const float* w, int parts, int rows, int H, long long part_stride, float eps0,
+                     float eps1, float eps2, float eps3, void* hout, int out_dtype, float alpha, const float* nw, const float* nb,
+                     cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (H <= 0 || parts < 1 || parts > NORMED_MAX || (hout != nullptr && (nw == nullptr || nb == nullptr))) return GG_ERR_ARG;
+    const NormedEps eps = {{eps0, eps1, eps2, eps3}};
+    const bool vec = H % 4 == 0 && part_stride % 4 == 0 &&
+                     (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)hout | (uintptr_t)nw | (uintptr_t)nb) & 15) == 0;
+    GG_DISPATCH_DTYPE(out_dtype, TO,
+        if (vec) gg_launch(normed_sum_kernel<TO, 4>, dim3(rows), dim3(256), 0, stream, 1, x, y, w, parts, H, part_stride, eps, (TO*)hout,
+                           alpha, nw, nb);
+        else gg_launch(normed_sum_kernel<TO, 1>, dim3(rows), dim3(256), 0, stream, 1, x, y, w, parts, H, part_stride, eps, (TO*)hout,
+                       alpha, nw, nb));
     return gg_last_error();
 }
 
@@ -393,21 +528,50 @@ GG_API gg_qk_norm_rope_cache(const void* qkv, int dtype, void* q_out, const floa
 }
 
 // ----------------------------------------------------------------------------- q/k/v preparation, general form
-// One block per token of the fused projection output qkv[T, nq*d + nkv*d + nkv*dv] (q heads, k heads, v heads):
-//   norm_mode 0: no q/k norm; 1: every q and k head normed over its d elements with one weight of size d;
+// One block per token of the fused projection output qkv[T, nq*d + nkv*d + nkv*dv] (q heads, k heads, v heads; rows ld
+// apart):
+//   first, with taps > 0, a causal convolution over time of every column (cw [taps][columns] float32, the last tap meets
+//   the token itself; rows from before the step come from cstate [slot][taps - 1][columns]; see column_conv_kernel);
+//   norm_mode 0: no q/k norm; 1: every q and k head normed over its d elements with one weight of size d (null: none);
 //   2: q normed over all its nq*d elements at once with a weight of that size, k over its nkv*d alike;
+//   q times 1 + coef ln(1 + floor((p + 1) / every)) at position p (coef 0: not);
 //   then the rotation of the pairs (i, i + rot/2) of the first `rot` elements of every q and k head;
-//   q to q_out[T, nq, d], k into the paged key pool [page][kv_head][page_size][d], v (untouched) into the paged
-//   value pool [page][kv_head][page_size][dv].  The key and value head sizes may differ.  All arithmetic float32.
+//   q to q_out[T, nq, d], k into the paged key pool [page][kv_head][page_size][d], v into the paged value pool
+//   [page][kv_head][page_size][dv].  The key and value head sizes may differ.  All arithmetic float32.
+struct QkvConv {
+    const float* w;              // [taps][columns]
+    float* state;                // [slots][taps - 1][columns]
+    const int* cu_seqlens;
+    const int* slots;
+    int taps;                    // 0: no convolution
+    int one_each;                // no sequence brings more than one row: the state moves on here
+};
+
+template <typename T>
+__device__ __forceinline__ float qkv_column(const T* qkv, long long ld, int t, int start, float* st, int cols, int c,
+                                            const QkvConv& cv) {
+    const float cur = to_f<T>(qkv[(size_t)t * ld + c]);
+    if (cv.taps == 0) return cur;
+    const int R = cv.taps - 1;
+    float acc = cv.w[(size_t)R * cols + c] * cur, carry = cur;
+    for (int j = R - 1; j >= 0; --j) {
+        const int s = t - R + j;
+        const float v = s >= start ? to_f<T>(qkv[(size_t)s * ld + c]) : st[(size_t)(R + (s - start)) * cols + c];
+        acc = fmaf(cv.w[(size_t)j * cols + c], v, acc);
+        if (cv.one_each) { st[(size_t)j * cols + c] = carry; carry = v; }
+    }
+    return acc;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) qkv_prep_kernel(
-    const T* qkv, T* __restrict__ q_out,
+    const T* qkv, long long ld, T* __restrict__ q_out,
     const float* __restrict__ qw, const float* __restrict__ kw, float eps, int norm_mode,
     const float* cosv, const float* sinv,
     const int* __restrict__ positions, const int* __restrict__ seq_of_token,
     const int* __restrict__ page_table, int max_pages, int page_size,
     T* __restrict__ k_pool, T* __restrict__ v_pool,
-    int nq, int nkv, int d, int dv, int rot, const PageBounds pb) {
+    int nq, int nkv, int d, int dv, int rot, const QkvConv cv, float coef, double every, const PageBounds pb) {
     pdl_launch();
     pdl_wait();
     extern __shared__ float sm[];
@@ -416,10 +580,18 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(
     float* buf = sm;                 // [nqk] q and k as float
     float* hs = sm + nqk;            // [nq + nkv] one factor per head
     float* red = hs + nq + nkv;      // [33]
+    __shared__ float q_factor;
     const int b = seq_of_token[t];
-    const T* src = qkv + (size_t)t * row;
-    const bool write_kv = k_pool != nullptr && b >= 0;
-    for (int i = threadIdx.x; i < nqk; i += blockDim.x) buf[i] = to_f<T>(src[i]);
+    if (b < 0) {                     // padding row: nothing reads its q, the caches are not touched
+        for (int i = threadIdx.x; i < nq * d; i += blockDim.x) q_out[(size_t)t * nq * d + i] = from_f<T>(0.f);
+        return;
+    }
+    const int pos = positions[t];
+    const int start = cv.taps ? cv.cu_seqlens[b] : 0;
+    float* st = cv.taps > 1 ? cv.state + (size_t)cv.slots[b] * (cv.taps - 1) * row : nullptr;
+    if (threadIdx.x == 0) q_factor = coef != 0.f ? 1.f + coef * (float)log(floor(((double)pos + 1.0) / every) + 1.0) : 1.f;
+    const bool write_kv = k_pool != nullptr;
+    for (int i = threadIdx.x; i < nqk; i += blockDim.x) buf[i] = qkv_column<T>(qkv, ld, t, start, st, row, i, cv);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     if (norm_mode == 1) {
@@ -441,7 +613,6 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(
     __syncthreads();
     int page = -1, slot_in_page = 0;
     if (write_kv) {
-        const int pos = positions[t];
         page = gg_page_w(page_table + (size_t)b * max_pages, pos / page_size, max_pages, pb, 46);
         slot_in_page = pos % page_size;
     }
@@ -455,8 +626,8 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(
         const float* w = is_q ? qw : kw;
         // weight index: per head (mode 1) or over the whole projection (mode 2)
         const int wbase = norm_mode == 2 ? (is_q ? h * d : (h - nq) * d) : 0;
-        const float f = norm_mode ? hs[h] : 1.f;
-        auto val = [&](int j) { return buf[h * d + j] * f * (norm_mode ? w[wbase + j] : 1.f); };
+        const float f = (norm_mode ? hs[h] : 1.f) * (is_q ? q_factor : 1.f);
+        auto val = [&](int j) { return buf[h * d + j] * f * (w != nullptr ? w[wbase + j] : 1.f); };
         float o;
         if (i < half) o = val(i) * c[i] - val(i + half) * s[i];
         else if (i < rot) o = val(i - half) * s[i - half] + val(i) * c[i - half];
@@ -464,29 +635,50 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(
         if (is_q) q_out[(size_t)t * nq * d + idx] = from_f<T>(o);
         else k_pool[(((size_t)page * nkv + (h - nq)) * page_size + slot_in_page) * d + i] = from_f<T>(o);
     }
-    if (page >= 0) {
+    // (the convolution's state moves on for the values' columns too, whether or not the page is a good one)
+    if (page >= 0 || cv.taps) {
         for (int idx = threadIdx.x; idx < nkv * dv; idx += blockDim.x) {
             const int h = idx / dv, i = idx - h * dv;
-            v_pool[(((size_t)page * nkv + h) * page_size + slot_in_page) * dv + i] = src[nqk + idx];
+            const float v = qkv_column<T>(qkv, ld, t, start, st, row, nqk + idx, cv);
+            if (page >= 0) v_pool[(((size_t)page * nkv + h) * page_size + slot_in_page) * dv + i] = from_f<T>(v);
         }
     }
 }
 
-GG_API gg_qkv_prep(const void* qkv, int dtype, void* q_out, const float* qw, const float* kw, float eps, int norm_mode,
-                   const float* cosv, const float* sinv, const int* positions, const int* seq_of_token,
+template <typename T>
+__global__ void column_conv_state_kernel(const T* h, long long ldh, const float* __restrict__ in_bias, float* state,
+                                         const int* __restrict__ cu_seqlens, const int* __restrict__ slots,
+                                         const int* __restrict__ seq_of_token, int C, int taps);
+
+// conv_w null: no convolution.  max_new: the most tokens one sequence brings, where the caller knows it (1: the
+// convolution's state moves on in the same launch).  rot 0: cosv and sinv are not read.
+GG_API gg_qkv_prep(const void* qkv, int dtype, long long ld, void* q_out, const float* qw, const float* kw, float eps,
+                   int norm_mode, const float* cosv, const float* sinv, const int* positions, const int* seq_of_token,
                    const int* page_table, int max_pages, int page_size, int n_pages, void* k_pool, void* v_pool,
-                   int ntok, int nq, int nkv, int d, int dv, int rot, int* status, cudaStream_t stream) {
+                   int ntok, int nq, int nkv, int d, int dv, int rot, const float* conv_w, float* conv_state, int taps,
+                   const int* cu_seqlens, const int* slots, int n_seqs, int max_new, float coef, float every, int* status,
+                   cudaStream_t stream) {
     if (ntok <= 0) return 0;
-    if (d <= 0 || dv <= 0 || rot < 0 || rot > d || (rot & 1) || nq <= 0 || nkv <= 0 || page_size <= 0 ||
-        norm_mode < 0 || norm_mode > 2 || (norm_mode && (qw == nullptr || kw == nullptr))) return GG_ERR_ARG;
+    const int row = (nq + nkv) * d + nkv * dv;
+    if (d <= 0 || dv <= 0 || rot < 0 || rot > d || (rot & 1) || nq <= 0 || nkv <= 0 || page_size <= 0 || ld < row ||
+        norm_mode < 0 || norm_mode > 2 || (norm_mode == 2 && (qw == nullptr || kw == nullptr)) || !(every > 0.f) ||
+        (rot && (cosv == nullptr || sinv == nullptr)))
+        return GG_ERR_ARG;
+    if (conv_w != nullptr && (taps < 1 || taps > CONV_MAX_TAPS || (taps > 1 && conv_state == nullptr) || cu_seqlens == nullptr ||
+                              slots == nullptr || n_seqs <= 0))
+        return GG_ERR_ARG;
     const size_t smem = ((size_t)(nq + nkv) * d + nq + nkv + 33) * sizeof(float);
     if (smem > 200 * 1024) return GG_ERR_ARG;
+    const QkvConv cv = {conv_w, conv_state, cu_seqlens, slots, conv_w != nullptr ? taps : 0, max_new == 1 ? 1 : 0};
     GG_DISPATCH_DTYPE(dtype, T,
-        if (smem > 48 * 1024)
+        if (smem > 47 * 1024)
             cudaFuncSetAttribute(qkv_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         gg_launch(qkv_prep_kernel<T>, dim3(ntok), dim3(256), smem, stream, 1,
-            (const T*)qkv, (T*)q_out, qw, kw, eps, norm_mode, cosv, sinv, positions, seq_of_token, page_table, max_pages,
-            page_size, (T*)k_pool, (T*)v_pool, nq, nkv, d, dv, rot, PageBounds{n_pages, status}));
+            (const T*)qkv, ld, (T*)q_out, qw, kw, eps, norm_mode, cosv, sinv, positions, seq_of_token, page_table, max_pages,
+            page_size, (T*)k_pool, (T*)v_pool, nq, nkv, d, dv, rot, cv, coef, (double)every, PageBounds{n_pages, status});
+        if (cv.taps > 1 && !cv.one_each)
+            gg_launch(column_conv_state_kernel<T>, dim3(n_seqs, (row + 255) / 256), dim3(256), 0, stream, 1, (const T*)qkv, ld,
+                      (const float*)nullptr, conv_state, cu_seqlens, slots, seq_of_token, row, taps));
     return gg_last_error();
 }
 
@@ -623,9 +815,14 @@ GG_API gg_rmsnorm_add(float* x, float* y, const float* w, int rows, int H, float
     return gg_last_error();
 }
 
-// ----------------------------------------------------------------------------- SwiGLU
-// out[t, i] = silu(gu[t, i]) * gu[t, I + i], silu(z) = z / (1 + exp(-z)) (pkg/ops/ops.go:316-318).
-template <typename T>
+// ----------------------------------------------------------------------------- gated units
+// out[t, i] = act(gu[t, i]) * gu[t, I + i]; act 0: silu(z) = z / (1 + exp(-z)) (pkg/ops/ops.go:316-318); act 1: the tanh
+// form of gelu, 0.5 z (1 + tanh(u)) = z / (1 + exp(-2 u)) with u = sqrt(2 / pi) (z + 0.044715 z^3).
+template <int ACT> __device__ __forceinline__ float glu_act(float z) {
+    return z / (1.0f + expf(ACT == 1 ? -1.5957691216057308f * (z + 0.044715f * z * z * z) : -z));
+}
+
+template <typename T, int ACT>
 __global__ void swiglu_kernel(const T* gu, T* __restrict__ out, long long n, int I) {
     pdl_launch();
     pdl_wait();
@@ -635,10 +832,11 @@ __global__ void swiglu_kernel(const T* gu, T* __restrict__ out, long long n, int
     const int i = (int)(idx - t * I);
     const float g = to_f<T>(gu[t * 2 * I + i]);
     const float u = to_f<T>(gu[t * 2 * I + I + i]);
-    out[idx] = from_f<T>(g / (1.0f + expf(-g)) * u);
+    out[idx] = from_f<T>(glu_act<ACT>(g) * u);
 }
 
 // Eight elements per thread with 16-byte accesses (rows of I elements, I a multiple of 8).
+template <int ACT>
 __global__ void swiglu_vec8_kernel(const bf16* gu, bf16* __restrict__ out, long long nvec, int I8) {
     pdl_launch();
     pdl_wait();
@@ -655,26 +853,29 @@ __global__ void swiglu_vec8_kernel(const bf16* gu, bf16* __restrict__ out, long 
     for (int k = 0; k < 4; ++k) {
         const __nv_bfloat162 g2 = *reinterpret_cast<const __nv_bfloat162*>(&gw[k]);
         const __nv_bfloat162 u2 = *reinterpret_cast<const __nv_bfloat162*>(&uw[k]);
-        const float g0 = __low2float(g2), g1 = __high2float(g2);
-        const float r0 = g0 / (1.0f + expf(-g0)) * __low2float(u2);
-        const float r1 = g1 / (1.0f + expf(-g1)) * __high2float(u2);
+        const float r0 = glu_act<ACT>(__low2float(g2)) * __low2float(u2);
+        const float r1 = glu_act<ACT>(__high2float(g2)) * __high2float(u2);
         const __nv_bfloat162 r = __floats2bfloat162_rn(r0, r1);
         ow[k] = *reinterpret_cast<const uint32_t*>(&r);
     }
     *reinterpret_cast<uint4*>(out + idx * 8) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
 }
 
-GG_API gg_swiglu(const void* gu, int dtype, void* out, int ntok, int I, cudaStream_t stream) {
+GG_API gg_swiglu(const void* gu, int dtype, void* out, int ntok, int I, int act, cudaStream_t stream) {
     if (ntok <= 0) return 0;
-    if (I <= 0) return GG_ERR_ARG;
+    if (I <= 0 || act < 0 || act > 1) return GG_ERR_ARG;
     const long long n = (long long)ntok * I;
     if (dtype == GG_BF16 && I % 8 == 0 && ((((uintptr_t)gu) | ((uintptr_t)out)) & 15) == 0) {
         const long long nvec = n / 8;
-        gg_launch(swiglu_vec8_kernel, dim3((unsigned)((nvec + 255) / 256)), dim3(256), 0, stream, 1, (const bf16*)gu, (bf16*)out, nvec, I / 8);
+        const dim3 grid((unsigned)((nvec + 255) / 256));
+        if (act) gg_launch(swiglu_vec8_kernel<1>, grid, dim3(256), 0, stream, 1, (const bf16*)gu, (bf16*)out, nvec, I / 8);
+        else gg_launch(swiglu_vec8_kernel<0>, grid, dim3(256), 0, stream, 1, (const bf16*)gu, (bf16*)out, nvec, I / 8);
         return gg_last_error();
     }
+    const dim3 grid((unsigned)((n + 255) / 256));
     GG_DISPATCH_DTYPE(dtype, T,
-        gg_launch(swiglu_kernel<T>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, 1, (const T*)gu, (T*)out, n, I));
+        if (act) gg_launch(swiglu_kernel<T, 1>, grid, dim3(256), 0, stream, 1, (const T*)gu, (T*)out, n, I);
+        else gg_launch(swiglu_kernel<T, 0>, grid, dim3(256), 0, stream, 1, (const T*)gu, (T*)out, n, I));
     return gg_last_error();
 }
 
@@ -815,7 +1016,6 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const T* h, T* out, con
 // The state after the step: the last taps - 1 input rows of every sequence (rows of the step where it brought
 // that many, else the old state moved up).  Blocks (sequence, 256 channels); a thread reads all it needs of a channel
 // before it writes.  Padding sequences (seq_of_token < 0 at their first row) are left alone.
-#define CONV_MAX_TAPS 16
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_state_kernel(const T* h, float* state, const int* __restrict__ cu_seqlens,
                                                                const int* __restrict__ slots,
@@ -1327,8 +1527,8 @@ GG_API gg_row_gate(void* act, int F, const void* h, int W, int dtype, const floa
 // in_bias may be null.  Blocks (token, 256 channels).  one_each != 0: no sequence brings more than one row, so the
 // thread of a channel is the only one that reads its state and moves it on itself; otherwise
 // column_conv_state_kernel does that once every block has read the old state.
-template <typename T>
-__global__ void __launch_bounds__(256) column_conv_kernel(const T* h, long long ldh, float* out, long long ldo,
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256) column_conv_kernel(const T* h, long long ldh, TO* out, long long ldo,
                                                           const float* __restrict__ w, const float* __restrict__ bias,
                                                           const float* __restrict__ in_bias, float* state,
                                                           const int* __restrict__ cu_seqlens, const int* __restrict__ slots,
@@ -1338,9 +1538,9 @@ __global__ void __launch_bounds__(256) column_conv_kernel(const T* h, long long 
     pdl_wait();
     const int t = blockIdx.x;
     const int b = seq_of_token[t];
-    float* o = out + (size_t)t * ldo;
+    TO* o = out + (size_t)t * ldo;
     if (b < 0) {
-        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) o[c] = 0.f;
+        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) o[c] = from_f<TO>(0.f);
         return;
     }
     const int start = cu_seqlens[b];
@@ -1357,7 +1557,7 @@ __global__ void __launch_bounds__(256) column_conv_kernel(const T* h, long long 
             acc = fmaf(w[(size_t)j * C + c], v, acc);
             if (one_each) { st[(size_t)j * C + c] = carry; carry = v; }
         }
-        o[c] = act == 1 ? acc / (1.0f + expf(-acc)) : acc;
+        o[c] = from_f<TO>(act == 1 ? acc / (1.0f + expf(-acc)) : acc);
     }
 }
 
@@ -1392,8 +1592,8 @@ __global__ void __launch_bounds__(256) column_conv_state_kernel(const T* h, long
 // The same for up to eight taps, a thread walking TT consecutive rows of one channel with the window of earlier values
 // in registers, so that a row of h is read once instead of once per tap; the window is filled again (from the
 // step's rows or the sequence's state) where a new sequence starts among the rows.  Blocks (TT rows, 256 channels).
-template <typename T, int TAPS, int TT>
-__global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long long ldh, float* out, long long ldo,
+template <typename T, typename TO, int TAPS, int TT>
+__global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long long ldh, TO* out, long long ldo,
                                                                const float* __restrict__ w, const float* __restrict__ bias,
                                                                const float* __restrict__ in_bias, float* state,
                                                                const int* __restrict__ cu_seqlens,
@@ -1417,7 +1617,7 @@ __global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long 
         const int t = t0 + tt;
         if (t >= ntok) break;
         const int b = seq_of_token[t];
-        if (b < 0) { out[(size_t)t * ldo + c] = 0.f; prev_b = -2; continue; }
+        if (b < 0) { out[(size_t)t * ldo + c] = from_f<TO>(0.f); prev_b = -2; continue; }
         float* st = state + (size_t)slots[b] * R * C + c;
         if (b != prev_b) {
             const int start = cu_seqlens[b];
@@ -1432,7 +1632,7 @@ __global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long 
         float acc = fmaf(wr[R], cur, ob);
 #pragma unroll
         for (int j = 0; j < R; ++j) acc = fmaf(wr[j], win[j], acc);
-        out[(size_t)t * ldo + c] = act == 1 ? acc / (1.0f + expf(-acc)) : acc;
+        out[(size_t)t * ldo + c] = from_f<TO>(act == 1 ? acc / (1.0f + expf(-acc)) : acc);
 #pragma unroll
         for (int j = 0; j + 1 < R; ++j) win[j] = win[j + 1];
         if (R > 0) win[R - 1] = cur;
@@ -1443,49 +1643,57 @@ __global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long 
     }
 }
 
-template <typename T, int TAPS>
-static int column_conv_tile_launch(const T* h, long long ldh, float* out, long long ldo, const float* w, const float* bias,
+template <typename T, typename TO, int TAPS>
+static int column_conv_tile_launch(const T* h, long long ldh, TO* out, long long ldo, const float* w, const float* bias,
                                    const float* in_bias, float* state, const int* cu_seqlens, const int* slots,
                                    const int* seq_of_token, int ntok, int C, int act, int one_each, cudaStream_t stream) {
     const unsigned cb = (unsigned)((C + 255) / 256);
     if (ntok < 1024 || one_each)       // few rows, or a row a sequence: a row a thread, so that the step fills more of the GPU
-        return gg_launch(column_conv_tile_kernel<T, TAPS, 1>, dim3((unsigned)ntok, cb), dim3(256), 0, stream, 1, h, ldh, out, ldo,
+        return gg_launch(column_conv_tile_kernel<T, TO, TAPS, 1>, dim3((unsigned)ntok, cb), dim3(256), 0, stream, 1, h, ldh, out, ldo,
                          w, bias, in_bias, state, cu_seqlens, slots, seq_of_token, C, ntok, act, one_each);
-    return gg_launch(column_conv_tile_kernel<T, TAPS, 8>, dim3((unsigned)((ntok + 7) / 8), cb), dim3(256), 0, stream, 1, h, ldh,
+    return gg_launch(column_conv_tile_kernel<T, TO, TAPS, 8>, dim3((unsigned)((ntok + 7) / 8), cb), dim3(256), 0, stream, 1, h, ldh,
                      out, ldo, w, bias, in_bias, state, cu_seqlens, slots, seq_of_token, C, ntok, act, one_each);
 }
 
-template <typename T>
-static int column_conv_tile(int taps, const T* h, long long ldh, float* out, long long ldo, const float* w, const float* bias,
+template <typename T, typename TO>
+static int column_conv_tile(int taps, const T* h, long long ldh, TO* out, long long ldo, const float* w, const float* bias,
                             const float* in_bias, float* state, const int* cu_seqlens, const int* slots,
                             const int* seq_of_token, int ntok, int C, int act, int one_each, cudaStream_t stream) {
-#define CC_CASE(N) case N: return column_conv_tile_launch<T, N>(h, ldh, out, ldo, w, bias, in_bias, state, cu_seqlens, slots, \
+#define CC_CASE(N) case N: return column_conv_tile_launch<T, TO, N>(h, ldh, out, ldo, w, bias, in_bias, state, cu_seqlens, slots, \
                                                                 seq_of_token, ntok, C, act, one_each, stream);
     switch (taps) { CC_CASE(1) CC_CASE(2) CC_CASE(3) CC_CASE(4) CC_CASE(5) CC_CASE(6) CC_CASE(7) CC_CASE(8) }
 #undef CC_CASE
     return GG_ERR_ARG;
 }
 
-// w [taps][C] float32 (a tap's weights side by side); state [slots][taps - 1][C] float32 (null only for one tap).
-GG_API gg_column_conv(const void* h, long long ldh, int dtype, float* out, long long ldo, const float* w, const float* bias,
-                      const float* in_bias, float* state, const int* cu_seqlens, const int* slots, const int* seq_of_token,
-                      int ntok, int n_seqs, int C, int taps, int act, int max_new, cudaStream_t stream) {
+// w [taps][C] float32 (a tap's weights side by side); state [slots][taps - 1][C] float32 (null only for one tap).  h in
+// `dtype`; out in `out_dtype`: float32, or `dtype` where that is bfloat16.
+GG_API gg_column_conv(const void* h, long long ldh, int dtype, void* out, int out_dtype, long long ldo, const float* w,
+                      const float* bias, const float* in_bias, float* state, const int* cu_seqlens, const int* slots,
+                      const int* seq_of_token, int ntok, int n_seqs, int C, int taps, int act, int max_new, cudaStream_t stream) {
     if (ntok <= 0 || n_seqs <= 0) return 0;
     if (C <= 0 || taps < 1 || taps > CONV_MAX_TAPS || (taps > 1 && state == nullptr) || act < 0 || act > 1 || ldh < C || ldo < C)
         return GG_ERR_ARG;
+    if (out_dtype != GG_F32 && !(out_dtype == GG_BF16 && dtype == GG_BF16)) return GG_ERR_DTYPE;
     const int cb = min((C + 255) / 256, 65535);
     const int one_each = max_new == 1;
-    GG_DISPATCH_DTYPE(dtype, T,
-        if (taps <= 8 && cb <= 65535) {
-            column_conv_tile<T>(taps, (const T*)h, ldh, out, ldo, w, bias, in_bias, state, cu_seqlens, slots, seq_of_token, ntok,
-                                C, act, one_each, stream);
-        } else {
-            gg_launch(column_conv_kernel<T>, dim3(ntok, cb), dim3(256), 0, stream, 1, (const T*)h, ldh, out, ldo, w, bias, in_bias,
-                      state, cu_seqlens, slots, seq_of_token, C, taps, act, one_each);
-        }
-        if (taps > 1 && !one_each)
-            gg_launch(column_conv_state_kernel<T>, dim3(n_seqs, cb), dim3(256), 0, stream, 1, (const T*)h, ldh, in_bias, state,
-                      cu_seqlens, slots, seq_of_token, C, taps));
+#define GG_CC(T_, TO_)                                                                                                    \
+    do {                                                                                                                  \
+        if (taps <= 8)                                                                                                    \
+            column_conv_tile<T_, TO_>(taps, (const T_*)h, ldh, (TO_*)out, ldo, w, bias, in_bias, state, cu_seqlens, slots, \
+                                      seq_of_token, ntok, C, act, one_each, stream);                                      \
+        else                                                                                                              \
+            gg_launch(column_conv_kernel<T_, TO_>, dim3(ntok, cb), dim3(256), 0, stream, 1, (const T_*)h, ldh, (TO_*)out, ldo, w, \
+                      bias, in_bias, state, cu_seqlens, slots, seq_of_token, C, taps, act, one_each);                     \
+        if (taps > 1 && !one_each)                                                                                        \
+            gg_launch(column_conv_state_kernel<T_>, dim3(n_seqs, cb), dim3(256), 0, stream, 1, (const T_*)h, ldh, in_bias, state, \
+                      cu_seqlens, slots, seq_of_token, C, taps);                                                          \
+    } while (0)
+    if (dtype == GG_F32) GG_CC(float, float);
+    else if (dtype != GG_BF16) return GG_ERR_DTYPE;
+    else if (out_dtype == GG_F32) GG_CC(bf16, float);
+    else GG_CC(bf16, bf16);
+#undef GG_CC
     return gg_last_error();
 }
 

@@ -70,14 +70,15 @@ def attn_prefill_tc(q, k_pool, v_pool, out, cu_seqlens, ctx_lens, seq_of_token, 
         status_word(q.device).data_ptr(), torch.cuda.current_stream().cuda_stream)
 
 
-def try_make(nq: int, nkv: int, d: int, scale: float, window: int) -> Optional[Callable]:
+def try_make(nq: int, nkv: int, d: int, scale: float, window: int, dv: Optional[int] = None,
+             chunk: int = 0) -> Optional[Callable]:
     """f(q, k_pool, v_pool, out, ctx, table, page_size, sink=None, out_scale=1.0) for bfloat16, or None when the
     sizes are outside what the tensor-core kernels take (head size 64 or 128, at most 16 query heads per kv
     head); then the plain kernel serves."""
-    if d not in (64, 128) or nq % nkv or nq // nkv > 16:
+    if d not in (64, 128) or nq % nkv or nq // nkv > 16 or chunk or dv not in (None, d):
         return None
 
-    def run(q, k_pool, v_pool, out, ctx, table, page_size, sink=None, out_scale=1.0):
+    def run(q, k_pool, v_pool, out, ctx, table, page_size, sink=None, out_scale=1.0, gate=None):
         T = ctx.n_tokens
         if page_size != 64 or q.dtype != torch.bfloat16:
             K.attention_plain(q, k_pool, v_pool, out, ctx.positions, ctx.seq_of_token, table, page_size,

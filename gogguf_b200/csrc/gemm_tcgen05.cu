@@ -75,7 +75,11 @@ __device__ __forceinline__ void tc_fence_after() { tc5::fence_after(); }
 __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t* r) { tc5::ld16(taddr, r); }
 __device__ __forceinline__ void tmem_ld_wait() { tc5::wait_ld(); }
 
-__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + __expf(-g)) * u; }
+// act(g) * u of a gated unit: act 0 silu, 1 the tanh form of gelu, 0.5 z (1 + tanh y) = z / (1 + exp(-2 y))
+__device__ __forceinline__ float glu_mul(float g, float u, int act) {
+    const float e = act == 1 ? -1.5957691216057308f * (g + 0.044715f * g * g * g) : -g;
+    return g / (1.0f + __expf(e)) * u;
+}
 
 // RMSNorm folded into the products around it.  The norm's weight is multiplied into the next matrix
 // when the model is built, the activations are the bfloat16 copy of the raw residual, and what is left
@@ -85,6 +89,8 @@ __device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f +
 //   out_ssq  (float32-add output only) after out += product, the partial sums of squares of the updated
 //            rows, one per 128 output columns (ceil(N / 128) per token), and out_xhat, their bfloat16
 //            copy [M, N] (row stride N): what the next product and its factor need.  Null: nothing.
+//   t_w, t_b, t_alpha  (with out_xhat) the norm that comes next is a dynamic tanh, which needs no sum over the row:
+//            out_xhat gets tanh(t_alpha v) t_w + t_b of the updated rows v, finished.  out_ssq may then be null.
 // Sums are float32 and their order is fixed, so results do not depend on timing.
 struct NormIO {
     const float* in_ssq;
@@ -94,7 +100,16 @@ struct NormIO {
     float* out_ssq;
     bf16* out_xhat;
     const float* bias;       // [N] float32 or null: added to every row after the factor (all modes but SwiGLU and q/k/v)
+    const float* t_w;        // [N] float32 or null
+    const float* t_b;
+    float t_alpha;
+    int glu_act;             // the gated unit's activation (SwiGLU mode): 0 silu, 1 gelu in its tanh form
 };
+
+// What goes to out_xhat for an updated residual value v of column c.
+__device__ __forceinline__ float emit_value(const NormIO& nio, float v, int c) {
+    return nio.t_w != nullptr ? fmaf(tanhf(nio.t_alpha * v), __ldg(nio.t_w + c), __ldg(nio.t_b + c)) : v;
+}
 
 // Bias values of `n` consecutive columns from c0 on (columns at or beyond N get 0), added to v.
 template <int n>
@@ -242,7 +257,7 @@ __device__ __forceinline__ void store_row_chunk16(const uint32_t* r, int gi, int
         return;
     }
     float* op = (float*)out + o;
-    const bool stats = nio.out_ssq != nullptr && out_mode == OUT_F32_ACC;
+    const bool stats = nio.out_xhat != nullptr && out_mode == OUT_F32_ACC;
     bf16* xp = stats ? nio.out_xhat + (size_t)gi * N + gj0 : nullptr;
     if (whole && ((((uintptr_t)op) & 15) == 0) && (!stats || (((uintptr_t)xp) & 15) == 0)) {
         uint32_t pk[8];
@@ -258,7 +273,9 @@ __device__ __forceinline__ void store_row_chunk16(const uint32_t* r, int gi, int
             *dst = v;
             if (stats) {
                 ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
-                __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+                const int c = gj0 + 4 * j;
+                __nv_bfloat162 a = __floats2bfloat162_rn(emit_value(nio, v.x, c), emit_value(nio, v.y, c + 1)),
+                               b = __floats2bfloat162_rn(emit_value(nio, v.z, c + 2), emit_value(nio, v.w, c + 3));
                 pk[2 * j] = *reinterpret_cast<uint32_t*>(&a);
                 pk[2 * j + 1] = *reinterpret_cast<uint32_t*>(&b);
             }
@@ -274,11 +291,11 @@ __device__ __forceinline__ void store_row_chunk16(const uint32_t* r, int gi, int
                 float v = __uint_as_float(r[j]);
                 if (out_mode == OUT_F32_ACC) v += op[j];
                 op[j] = v;
-                if (stats) { ss = fmaf(v, v, ss); xp[j] = __float2bfloat16_rn(v); }
+                if (stats) { ss = fmaf(v, v, ss); xp[j] = __float2bfloat16_rn(emit_value(nio, v, gj0 + j)); }
             }
     }
     if (stats && (((gj0 & 127) == 112) || gj0 + 16 >= N)) {
-        nio.out_ssq[(size_t)gi * ((N + 127) / 128) + (gj0 >> 7)] = ss;
+        if (nio.out_ssq != nullptr) nio.out_ssq[(size_t)gi * ((N + 127) / 128) + (gj0 >> 7)] = ss;
         ss = 0.f;
     }
 }
@@ -311,8 +328,8 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
 #pragma unroll
                     for (int j = 0; j < 8; ++j) {
                         __nv_bfloat162 h2 = __floats2bfloat162_rn(
-                            silu_mul(__uint_as_float(g[2 * j]) * sc, __uint_as_float(u[2 * j]) * sc),
-                            silu_mul(__uint_as_float(g[2 * j + 1]) * sc, __uint_as_float(u[2 * j + 1]) * sc));
+                            glu_mul(__uint_as_float(g[2 * j]) * sc, __uint_as_float(u[2 * j]) * sc, nio.glu_act),
+                            glu_mul(__uint_as_float(g[2 * j + 1]) * sc, __uint_as_float(u[2 * j + 1]) * sc, nio.glu_act));
                         pk[j] = *reinterpret_cast<uint32_t*>(&h2);
                     }
                     reinterpret_cast<uint4*>(op)[0] = make_uint4(pk[0], pk[1], pk[2], pk[3]);
@@ -320,7 +337,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
                 } else {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        if (ocol + j < nout) op[j] = __float2bfloat16_rn(silu_mul(__uint_as_float(g[j]) * sc, __uint_as_float(u[j]) * sc));
+                        if (ocol + j < nout) op[j] = __float2bfloat16_rn(glu_mul(__uint_as_float(g[j]) * sc, __uint_as_float(u[j]) * sc, nio.glu_act));
                 }
             }
         }
@@ -332,7 +349,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
         // Adding into the residual reads what is there: one thread's 16 columns at a time, every group would
         // wait a whole trip to L2 for its 64 bytes (about 20 us per tile, in the open after a product's last
         // tile).  So the old values of 64 columns are asked for at once, before the accumulator is read.
-        const bool stats = nio.out_ssq != nullptr;
+        const bool stats = nio.out_xhat != nullptr;
         const bool scaled = nio.in_ssq != nullptr;
         const bool live = gi < M;
         float* orow = (float*)out + (size_t)(live ? gi : 0) * ldo + tn * BN;
@@ -370,7 +387,9 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
                     reinterpret_cast<float4*>(orow + c0 + 16 * q)[j] = v;
                     if (stats) {
                         ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
-                        __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+                        const int c = tn * BN + c0 + 16 * q + 4 * j;
+                        __nv_bfloat162 a = __floats2bfloat162_rn(emit_value(nio, v.x, c), emit_value(nio, v.y, c + 1)),
+                                       b = __floats2bfloat162_rn(emit_value(nio, v.z, c + 2), emit_value(nio, v.w, c + 3));
                         pk[2 * j] = *reinterpret_cast<uint32_t*>(&a);
                         pk[2 * j + 1] = *reinterpret_cast<uint32_t*>(&b);
                     }
@@ -381,7 +400,7 @@ __device__ __forceinline__ void epilogue_row_256(uint32_t taddr, int gi, int tn,
                 }
             }
             if (stats && (c0 & 64)) {            // a part of 128 columns is complete
-                nio.out_ssq[(size_t)gi * ((N + 127) / 128) + ((tn * BN + c0) >> 7)] = ss;
+                if (nio.out_ssq != nullptr) nio.out_ssq[(size_t)gi * ((N + 127) / 128) + ((tn * BN + c0) >> 7)] = ss;
                 ss = 0.f;
             }
         }
@@ -524,7 +543,7 @@ __device__ __forceinline__ bool residual_prefetch(int gj, int tile_a, int lane, 
     const int gi0 = tile_a * BM + 4 * lane;
     if (gi0 + 4 > N) return false;
     const float* op = (const float*)out + (size_t)gj * ldo + gi0;
-    const bool stats = nio.out_ssq != nullptr;
+    const bool stats = nio.out_xhat != nullptr;
     if ((((uintptr_t)op) & 15) != 0 || (stats && (((uintptr_t)(nio.out_xhat + (size_t)gj * N + gi0)) & 7) != 0)) return false;
     old = *reinterpret_cast<const float4*>(op);
     return true;
@@ -539,8 +558,8 @@ __device__ __forceinline__ void finish_token_block(float4 acc, int gj, int tile_
         const int feat = tile_a * 64 + 4 * lane;
         if (lane < 16 && feat < N / 2) {                 // N / 2 is a multiple of 64 here
             bf16* op = (bf16*)out + (size_t)gj * ldo + feat;
-            __nv_bfloat162 a = __floats2bfloat162_rn(silu_mul(acc.x, ux), silu_mul(acc.y, uy));
-            __nv_bfloat162 b = __floats2bfloat162_rn(silu_mul(acc.z, uz), silu_mul(acc.w, uw));
+            __nv_bfloat162 a = __floats2bfloat162_rn(glu_mul(acc.x, ux, nio.glu_act), glu_mul(acc.y, uy, nio.glu_act));
+            __nv_bfloat162 b = __floats2bfloat162_rn(glu_mul(acc.z, uz, nio.glu_act), glu_mul(acc.w, uw, nio.glu_act));
             if ((((uintptr_t)op) & 7) == 0) {
                 *reinterpret_cast<uint2*>(op) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
             } else {
@@ -550,7 +569,7 @@ __device__ __forceinline__ void finish_token_block(float4 acc, int gj, int tile_
         return;
     }
     const int gi0 = tile_a * BM + 4 * lane;              // first of this lane's four features
-    const bool stats = nio.out_ssq != nullptr && out_mode == OUT_F32_ACC;
+    const bool stats = nio.out_xhat != nullptr && out_mode == OUT_F32_ACC;
     float ss = 0.f;
     if (gi0 < N) {
         const bool whole = gi0 + 4 <= N;
@@ -579,7 +598,8 @@ __device__ __forceinline__ void finish_token_block(float4 acc, int gj, int tile_
                 *reinterpret_cast<float4*>(op) = w4;
                 if (stats) {
                     ss = fmaf(w4.x, w4.x, ss); ss = fmaf(w4.y, w4.y, ss); ss = fmaf(w4.z, w4.z, ss); ss = fmaf(w4.w, w4.w, ss);
-                    __nv_bfloat162 a = __floats2bfloat162_rn(w4.x, w4.y), b = __floats2bfloat162_rn(w4.z, w4.w);
+                    __nv_bfloat162 a = __floats2bfloat162_rn(emit_value(nio, w4.x, gi0), emit_value(nio, w4.y, gi0 + 1)),
+                                   b = __floats2bfloat162_rn(emit_value(nio, w4.z, gi0 + 2), emit_value(nio, w4.w, gi0 + 3));
                     *reinterpret_cast<uint2*>(xp) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
                 }
             } else {
@@ -589,12 +609,12 @@ __device__ __forceinline__ void finish_token_block(float4 acc, int gj, int tile_
                         float val = f[t];
                         if (out_mode == OUT_F32_ACC) val += op[t];
                         op[t] = val;
-                        if (stats) { ss = fmaf(val, val, ss); xp[t] = __float2bfloat16_rn(val); }
+                        if (stats) { ss = fmaf(val, val, ss); xp[t] = __float2bfloat16_rn(emit_value(nio, val, gi0 + t)); }
                     }
             }
         }
     }
-    if (stats) {
+    if (stats && nio.out_ssq != nullptr) {
         ss = warp_sum(ss);                               // one 128-feature part per tile
         if (lane == 0) nio.out_ssq[(size_t)gj * ((N + 127) / 128) + tile_a] = ss;
     }
@@ -652,7 +672,7 @@ __global__ void __launch_bounds__(NUM_THREADS, MINB) gemm_tc_kernel(
     // activation, and (decode form) whenever a norm is folded into this product or a bias goes with it
     // (only the decode form splits K or fuses the activation; the launcher sees to that)
     const bool staged = SWAP && (cluster_reduce || out_mode == OUT_SWIGLU || out_mode == OUT_QKV ||
-                                 (partial == nullptr && (nio.in_ssq != nullptr || nio.out_ssq != nullptr || nio.bias != nullptr)));
+                                 (partial == nullptr && (nio.in_ssq != nullptr || nio.out_xhat != nullptr || nio.bias != nullptr)));
     uint32_t* tmem_slot = (uint32_t*)(recv_bar + 1);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
     // decode form with a folded norm: the factor of every token of the tile, computed by the epilogue warps while
@@ -1686,7 +1706,7 @@ GG_API gg_gemm_tc(const void* x, const void* w, void* out, int out_mode, int M, 
                   long long ldo, float* scratch, long long scratch_elems, int use_cluster, int* status,
                   cudaStream_t stream) {
     if (out_mode == OUT_QKV) return GG_ERR_ARG;
-    const NormIO none = {nullptr, 0, 0.f, 0.f, nullptr, nullptr, nullptr};
+    const NormIO none = {};
     const QkvIO noq = {};
     return gemm_tc_impl(x, w, out, out_mode, M, N, K, ldx, ldo, scratch, scratch_elems, use_cluster, status, none, noq, stream);
 }
@@ -1700,15 +1720,21 @@ GG_API gg_gemm_tc(const void* x, const void* w, void* out, int out_mode, int M, 
 //   out_ssq != null (out_mode 2 only): after out += product the kernel also writes out_xhat[M, N]
 //     (bfloat16 copy of the updated rows, row stride N) and out_ssq[M, ceil(N / 128)], their partial sums
 //     of squares over blocks of 128 columns: the inputs of the next folded product.
+//   t_w, t_b != null (out_mode 2 with out_xhat; out_ssq may be null): out_xhat[M, N] gets tanh(t_alpha v) t_w + t_b of the
+//     updated rows v instead, the finished rows of a dynamic tanh that comes next.
+//   glu_act (out_mode 3): the gate's activation, 0 silu, 1 gelu in its tanh form.
 //   bias != null (not with out_mode 3): [N] float32, added to every row after the factor, before the output mode.
 GG_API gg_gemm_tc_norm(const void* x, const void* w, void* out, int out_mode, int M, int N, int K, long long ldx,
                        long long ldo, const float* in_ssq, int in_parts, float eps, float* out_ssq, void* out_xhat,
-                       const float* bias, float* scratch, long long scratch_elems, int* status, cudaStream_t stream) {
+                       const float* bias, const float* t_w, const float* t_b, float t_alpha, int glu_act, float* scratch,
+                       long long scratch_elems, int* status, cudaStream_t stream) {
     if (in_ssq != nullptr && (in_parts != (K + 127) / 128 || !(eps > 0.f))) return GG_ERR_ARG;
     if (bias != nullptr && out_mode == OUT_SWIGLU) return GG_ERR_ARG;
     if (out_ssq != nullptr && (out_mode != OUT_F32_ACC || out_xhat == nullptr)) return GG_ERR_ARG;
+    if (out_xhat != nullptr && (out_mode != OUT_F32_ACC || (out_ssq == nullptr && t_w == nullptr))) return GG_ERR_ARG;
+    if ((t_w == nullptr) != (t_b == nullptr) || (t_w != nullptr && out_xhat == nullptr) || glu_act < 0 || glu_act > 1) return GG_ERR_ARG;
     if (out_mode == OUT_QKV) return GG_ERR_ARG;
-    const NormIO nio = {in_ssq, in_parts, 1.0f / (float)K, eps, out_ssq, (bf16*)out_xhat, bias};
+    const NormIO nio = {in_ssq, in_parts, 1.0f / (float)K, eps, out_ssq, (bf16*)out_xhat, bias, t_w, t_b, t_alpha, glu_act};
     const QkvIO noq = {};
     return gemm_tc_impl(x, w, out, out_mode, M, N, K, ldx, ldo, scratch, scratch_elems, 1, status, nio, noq, stream);
 }
@@ -1733,7 +1759,7 @@ GG_API gg_gemm_tc_qkv_rope(const void* x, const void* w, int M, int K, long long
                            int max_pages, int page_size, int n_pages, void* k_pool, void* v_pool, int nq, int nkv,
                            float* scratch, long long scratch_elems, int* status, cudaStream_t stream) {
     if (in_ssq != nullptr && (in_parts != (K + 127) / 128 || !(in_eps > 0.f))) return GG_ERR_ARG;
-    const NormIO nio = {in_ssq, in_parts, K > 0 ? 1.0f / (float)K : 0.f, in_eps, nullptr, nullptr, nullptr};
+    const NormIO nio = {in_ssq, in_parts, K > 0 ? 1.0f / (float)K : 0.f, in_eps, nullptr, nullptr, nullptr, nullptr, nullptr, 0.f, 0};
     const QkvIO qio = {(bf16*)q_out, qw, kw, eps, cosv, sinv, positions, seq_of_token, page_table, max_pages, page_size,
                        (bf16*)k_pool, (bf16*)v_pool, nq, nkv, n_pages, status};
     const int N = (nq + 2 * nkv) * 128;

@@ -86,6 +86,47 @@ def row_stats(x: torch.Tensor, xhat: torch.Tensor, ssq: torch.Tensor) -> None:
     kernel("elementwise", "gg_row_stats")(_p(x), _p(xhat), _p(ssq), T, H, _stream())
 
 
+def dynamic_tanh(x: torch.Tensor, alpha: float, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor,
+                 rows: Optional[torch.Tensor] = None) -> None:
+    """out[r] = tanh(alpha * (x[rows[r]] or x[r])) * weight + bias; x, weight, bias float32, out float32/bfloat16."""
+    _need(x, torch.float32, "x")
+    _need(weight, torch.float32, "weight")
+    _need(bias, torch.float32, "bias")
+    H = x.shape[-1]
+    R = rows.numel() if rows is not None else x.numel() // H
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    if weight.numel() != H or bias.numel() != H or out.shape[-1] != H or out.numel() < R * H or not out.is_contiguous():
+        raise KernelError("dynamic_tanh: shapes disagree")
+    kernel("elementwise", "gg_dynamic_tanh")(_p(x), _p(rows), float(alpha), _p(weight), _p(bias), _p(out), dtype_code(out.dtype), R,
+                                              H, _stream())
+
+
+NORMED_MAX = 4                # parts that `normed_sum` takes (csrc/elementwise.cu)
+
+
+def normed_sum(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps, out: Optional[torch.Tensor] = None,
+               norm=None) -> None:
+    """x[r] += sum_k y[k, r] / sqrt(mean(y[k, r]^2) + eps[k]) * weight[k], all float32 (y [parts, rows, H], left zeroed).
+    norm (alpha, weight, bias): the updated rows' dynamic tanh goes to `out` as well."""
+    _need(x, torch.float32, "x")
+    _need(y, torch.float32, "y")
+    _need(weight, torch.float32, "weights")
+    H = x.shape[-1]
+    parts = y.shape[0]
+    if y.dim() != 3 or parts != len(eps) or parts > NORMED_MAX or weight.numel() != parts * H or y.numel() != parts * x.numel():
+        raise KernelError("normed_sum: y is [parts, rows, H] with a weight row and an eps per part")
+    alpha, nw, nb = norm if norm is not None else (0.0, None, None)
+    if (out is None) != (norm is None):
+        raise KernelError("normed_sum: a norm and the rows for it come together")
+    if out is not None and (out.numel() != x.numel() or not out.is_contiguous()):
+        raise KernelError("normed_sum: out has the shape of x")
+    e = list(eps) + [1.0] * (NORMED_MAX - parts)
+    kernel("elementwise", "gg_normed_sum")(_p(x), _p(y), _p(weight), parts, x.numel() // H, H, x.numel(), *(float(v) for v in e),
+                                            _p(out), dtype_code(out.dtype) if out is not None else F32, float(alpha), _p(nw), _p(nb),
+                                            _stream())
+
+
 def rope_tables(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor,
                 mag: float = 1.0) -> None:
     """cos, sin [T, half] (float32) = mag * cos / sin of positions[t] * inv_freq[i], angles in float64."""
@@ -113,29 +154,46 @@ def qk_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optiona
 
 
 def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor],
-             eps: float, norm_mode: int, cos: torch.Tensor, sin: torch.Tensor, positions: torch.Tensor,
+             eps: float, norm_mode: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor,
              seq_of_token: torch.Tensor, page_table: torch.Tensor, page_size: int, k_pool: Optional[torch.Tensor],
-             v_pool: Optional[torch.Tensor], n_tokens: int, nq: int, nkv: int, d: int, dv: int, rot: int) -> None:
-    """The general q/k/v preparation: qkv [T, nq*d + nkv*d + nkv*dv]; norm_mode 0 none, 1 per head (weights of
-    size d), 2 over the whole q and the whole k projection (weights of size nq*d and nkv*d); rotation of the first
-    `rot` elements of each q and k head; q to q_out, k and v into the paged pools (head sizes d and dv)."""
+             v_pool: Optional[torch.Tensor], n_tokens: int, nq: int, nkv: int, d: int, dv: int, rot: int,
+             conv: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None,
+             cu_seqlens: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None, n_seqs: int = 0, max_new: int = 0,
+             coef: float = 0.0, every: float = 1.0) -> None:
+    """The general q/k/v preparation: qkv [T, nq*d + nkv*d + nkv*dv] (a column range of a wider row may be given);
+    conv [taps, columns] (float32): a causal convolution over time of every column first, from and into conv_state [slots,
+    taps - 1, columns]; norm_mode 0 none, 1 per head (weights of size d, or None: no weight), 2 over the whole q and the
+    whole k projection (weights of size nq*d and nkv*d); q times 1 + coef ln(1 + floor((p + 1) / every)); rotation of the
+    first `rot` elements of every q and k head; q to q_out, k and v into the paged pools (head sizes d and dv)."""
+    cols = (nq + nkv) * d + nkv * dv
     if q_out.dtype != qkv.dtype or (k_pool is not None and (k_pool.dtype != qkv.dtype or v_pool.dtype != qkv.dtype)):
         raise KernelError("qkv_prep: qkv, q_out and the cache must share one dtype")
-    if not qkv.is_contiguous() or qkv.shape[-1] != (nq + nkv) * d + nkv * dv:
-        raise KernelError("qkv_prep: qkv must be contiguous [T, nq*d + nkv*d + nkv*dv]")
-    if norm_mode:
+    if qkv.stride(-1) != 1 or qkv.shape[-1] != cols:
+        raise KernelError("qkv_prep: qkv is [T, nq*d + nkv*d + nkv*dv] with unit column stride")
+    if norm_mode and (norm_mode == 2 or q_weight is not None):
         want = (d, d) if norm_mode == 1 else (nq * d, nkv * d)
         _need(q_weight, torch.float32, "q norm weight")
         _need(k_weight, torch.float32, "k norm weight")
         if (q_weight.numel(), k_weight.numel()) != want:
             raise KernelError(f"qkv_prep: norm weights of {q_weight.numel()} and {k_weight.numel()} elements, "
                               f"{want[0]} and {want[1]} expected")
+    taps = 0
+    if conv is not None:
+        _need(conv, torch.float32, "taps")
+        taps = conv.shape[0]
+        if conv.shape[-1] != cols:
+            raise KernelError("qkv_prep: the taps are [taps, columns]")
+        if taps > 1:
+            _need(conv_state, torch.float32, "conv state")
+            if tuple(conv_state.shape[1:]) != (taps - 1, cols):
+                raise KernelError("qkv_prep: the convolution's state is [slots, taps - 1, columns]")
     from .tcgen05_gemm import status_word
     kernel("elementwise", "gg_qkv_prep")(
-        _p(qkv), dtype_code(qkv.dtype), _p(q_out), _p(q_weight), _p(k_weight), float(eps), int(norm_mode), _p(cos),
+        _p(qkv), dtype_code(qkv.dtype), qkv.stride(0), _p(q_out), _p(q_weight), _p(k_weight), float(eps), int(norm_mode), _p(cos),
         _p(sin), _p(positions), _p(seq_of_token), _p(page_table), page_table.shape[-1], page_size,
         k_pool.shape[0] if k_pool is not None else 0, _p(k_pool), _p(v_pool),
-        n_tokens, nq, nkv, d, dv, rot, _p(status_word(qkv.device)), _stream())
+        n_tokens, nq, nkv, d, dv, rot, _p(conv), _p(conv_state), int(taps), _p(cu_seqlens), _p(slots), int(n_seqs), int(max_new),
+        float(coef), float(every), _p(status_word(qkv.device)), _stream())
 
 
 def rmsnorm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
@@ -263,13 +321,13 @@ def column_conv(h: torch.Tensor, out: torch.Tensor, weight: torch.Tensor, bias: 
                 slots: torch.Tensor, seq_of_token: torch.Tensor, n_tokens: int, n_seqs: int, act: int = 0,
                 max_new: int = 0) -> None:
     """out[t] = act(bias + sum_j weight[j] * v[t - taps + 1 + j]) per channel inside each sequence, v = h + in_bias;
-    h [T, C] may be a column range of a wider buffer (compute dtype), out [T, C] is float32 (likewise), weight is
-    [taps, C] float32; rows before the step come from state [slots, taps - 1, C] (float32), which is then moved on.
+    h [T, C] may be a column range of a wider buffer (compute dtype), out [T, C] is float32 or the dtype of h (likewise),
+    weight is [taps, C] float32; rows before the step come from state [slots, taps - 1, C] (float32), which is then moved on.
     act 0 none, 1 silu."""
     taps, C = weight.shape
     _need(weight, torch.float32, "taps")
-    if out.dtype != torch.float32 or h.stride(-1) != 1 or out.stride(-1) != 1 or h.shape[-1] != C or out.shape[-1] != C:
-        raise KernelError("column_conv: h [T, C] and out [T, C] (float32) have unit column stride")
+    if out.dtype not in (torch.float32, h.dtype) or h.stride(-1) != 1 or out.stride(-1) != 1 or h.shape[-1] != C or out.shape[-1] != C:
+        raise KernelError("column_conv: h [T, C] and out [T, C] (float32, or the dtype of h) have unit column stride")
     for t in (bias, in_bias):
         if t is not None:
             _need(t, torch.float32, "bias")
@@ -279,7 +337,7 @@ def column_conv(h: torch.Tensor, out: torch.Tensor, weight: torch.Tensor, bias: 
         _need(state, torch.float32, "state")
         if tuple(state.shape[1:]) != (taps - 1, C):
             raise KernelError("column_conv: the state is [slots, taps - 1, C]")
-    kernel("elementwise", "gg_column_conv")(_p(h), h.stride(0), dtype_code(h.dtype), _p(out), out.stride(0), _p(weight),
+    kernel("elementwise", "gg_column_conv")(_p(h), h.stride(0), dtype_code(h.dtype), _p(out), dtype_code(out.dtype), out.stride(0), _p(weight),
                                              _p(bias), _p(in_bias), _p(state), _p(cu_seqlens), _p(slots), _p(seq_of_token),
                                              int(n_tokens), int(n_seqs), C, taps, int(act), int(max_new), _stream())
 
@@ -300,10 +358,14 @@ def softcap(z: torch.Tensor, cap: float, n: Optional[int] = None, scale: float =
     kernel("elementwise", "gg_softcap")(_p(z), float(cap), float(scale), int(z.numel() if n is None else n), _stream())
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, n_tokens: int, inter: int) -> None:
+GLU_ACTS = {"silu": 0, "gelu_tanh": 1}      # activations of the gated units
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, n_tokens: int, inter: int, act: int = 0) -> None:
+    """out = act(gate) * up; act: a number of GLU_ACTS."""
     if gate_up.dtype != out.dtype:
         raise KernelError("swiglu: input and output must share one dtype")
-    kernel("elementwise", "gg_swiglu")(_p(gate_up), dtype_code(gate_up.dtype), _p(out), n_tokens, inter, _stream())
+    kernel("elementwise", "gg_swiglu")(_p(gate_up), dtype_code(gate_up.dtype), _p(out), n_tokens, inter, int(act), _stream())
 
 
 def residual_add(x: torch.Tensor, delta: torch.Tensor) -> None:
@@ -360,9 +422,12 @@ def gemm_plain(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: 
 def attention_plain(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                     positions: torch.Tensor, seq_of_token: torch.Tensor, page_table: torch.Tensor,
                     page_size: int, n_tokens: int, nq: int, nkv: int, d: int, scale: float, window: int,
-                    dv: Optional[int] = None, sink: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+                    dv: Optional[int] = None, sink: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+                    chunk: int = 0, gate: Optional[torch.Tensor] = None) -> None:
     """Attention over the paged cache on the CUDA cores; `dv` is the values' head size (default d), `sink` one
-    float32 per query head that joins the softmax's denominator, `out_scale` a factor on the result."""
+    float32 per query head that joins the softmax's denominator, `out_scale` a factor on the result; chunk > 0: a
+    position sees its own chunk of that many positions only; gate (rows of nq * dv logits): the result is multiplied by
+    their sigmoid."""
     if not (q.dtype == k_pool.dtype == v_pool.dtype == out.dtype):
         raise KernelError("attention: q, cache and out must share one dtype")
     dv = d if dv is None else int(dv)
@@ -370,11 +435,14 @@ def attention_plain(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         raise KernelError("attention: the pools' head sizes disagree with d and dv")
     if sink is not None:
         _need(sink, torch.float32, "sink")
+    if gate is not None and (gate.dtype != out.dtype or gate.stride(-1) != 1 or gate.shape[-1] != nq * dv):
+        raise KernelError("attention: the gate has rows of nq * dv logits in the output's dtype")
     from .tcgen05_gemm import status_word
     kernel("attention_plain", "gg_attention_plain")(
         _p(q), _p(k_pool), _p(v_pool), _p(out), dtype_code(q.dtype), _p(positions), _p(seq_of_token),
         _p(page_table), page_table.shape[-1], page_size, k_pool.shape[0], n_tokens, nq, nkv, d, dv, float(scale),
-        int(window), _p(sink), float(out_scale), _p(status_word(q.device)), _stream())
+        int(window), int(chunk), _p(sink), float(out_scale), _p(gate), gate.stride(0) if gate is not None else 0,
+        _p(status_word(q.device)), _stream())
 
 
 def diff_qk_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch.Tensor, k_weight: Optional[torch.Tensor],
@@ -882,6 +950,73 @@ def stepsize_finish(raw: torch.Tensor, xc: torch.Tensor, xd: torch.Tensor, z_off
     kernel("recurrence", "gg_stepsize_finish")(
         _p(raw), _p(xc), xc.stride(0), _p(xd), dtype_code(xd.dtype), dtype_code(out.dtype), xd.stride(0), int(z_off), _p(skip), _p(weight), _p(out),
         _p(seq_of_token), int(n_tokens), int(heads), int(dv), int(norm_groups), float(eps), _stream())
+
+
+# ------------------------------------------------------------------------------- selective scan
+SELECTIVE_MAX_STATE = 256
+
+
+def selective_scan_scratch(n_tokens: int, n_seqs: int, inner: int, N: int, chunk: int) -> int:
+    """Floats of scratch the chunked form of `selective_scan` needs: a state and a sum of steps per chunk and channel."""
+    return (n_tokens // chunk + n_seqs) * inner * (N + 1)
+
+
+def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, xdt: torch.Tensor,
+                   out: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
+                   seq_of_token: torch.Tensor, a: torch.Tensor, skip: torch.Tensor, n_tokens: int, n_seqs: int, chunk: int = 0,
+                   scratch: Optional[torch.Tensor] = None) -> None:
+    """dt = softplus(xdt); S[c, n] <- exp(dt a[c, n]) S[c, n] + dt x_c B_n; out_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c)
+    per channel, from and into state [slots, inner, N] (float32).  x, z [T, inner] and B, C (columns b_off and c_off of bc)
+    in the dtype of out, xdt [T, inner] float32 (all may be column ranges of wider rows); a [inner, N], skip [inner]
+    float32.  chunk > 0: in chunks of that many rows (prompts with few channels)."""
+    inner, N = a.shape
+    for t, n in ((xdt, "xdt"), (state, "state"), (a, "a"), (skip, "skip")):
+        if t.dtype != torch.float32:
+            raise KernelError(f"selective_scan: {n} is float32")
+    if not (x.dtype == z.dtype == bc.dtype == out.dtype) or not out.is_contiguous() or not a.is_contiguous():
+        raise KernelError("selective_scan: x, z, bc and out share one dtype")
+    for t in (x, z, bc, xdt):
+        if t.stride(-1) != 1:
+            raise KernelError("selective_scan: rows have unit column stride")
+    if tuple(state.shape[1:]) != (inner, N) or skip.numel() != inner or any(t.shape[-1] != inner for t in (x, z, xdt, out)) \
+            or bc.shape[-1] < max(b_off, c_off) + N:
+        raise KernelError("selective_scan: shapes disagree")
+    if chunk:
+        _need(scratch, torch.float32, "scratch")
+        if scratch.numel() < selective_scan_scratch(n_tokens, n_seqs, inner, N, chunk):
+            raise KernelError("selective_scan: the scratch is too small")
+    kernel("selective_scan", "gg_selective_scan")(
+        _p(x), x.stride(0), _p(z), z.stride(0), _p(bc), bc.stride(0), int(b_off), int(c_off), _p(xdt), xdt.stride(0), _p(out),
+        dtype_code(out.dtype), _p(state), _p(cu_seqlens), _p(slots), _p(seq_of_token), _p(a), _p(skip), int(n_tokens), int(n_seqs),
+        inner, N, int(chunk), _p(scratch), _stream())
+
+
+# ------------------------------------------------------------------------------- matrix memory
+def _memory_check(x, off, zi, zf, out, states, w, heads, d, dv):
+    S, n, m = states
+    for t in (S, n, m, w):
+        _need(t, torch.float32, "states and weight")
+    if tuple(S.shape[1:]) != (heads, d, dv) or tuple(n.shape[1:]) != (heads, d) or tuple(m.shape[1:]) != (heads,):
+        raise KernelError("memory: the states are [slots, heads, d, dv], [slots, heads, d] and [slots, heads]")
+    if zi.dtype != torch.float32 or zf.dtype != torch.float32 or zi.stride(0) != zf.stride(0) or zi.stride(-1) != 1 \
+            or zf.stride(-1) != 1 or zi.shape[-1] != heads or zf.shape[-1] != heads:
+        raise KernelError("memory: the gates' rows are float32 [T, heads] of one stride")
+    if x.stride(-1) != 1 or not out.is_contiguous() or out.shape[-1] != heads * dv or w.numel() != heads * dv:
+        raise KernelError("memory: shapes disagree")
+
+
+def memory_scan(x: torch.Tensor, off, zi: torch.Tensor, zf: torch.Tensor, out: torch.Tensor, states, cu_seqlens: torch.Tensor,
+                slots: torch.Tensor, seq_of_token: torch.Tensor, weight: torch.Tensor, n_tokens: int, n_seqs: int, heads: int,
+                d: int, dv: int, q_scale: float, cap: float, eps: float) -> None:
+    """A matrix memory with exponential gates, token by token, with each head's norm, the weight [heads * dv] and the output
+    gate (csrc/matrix_memory.cu).  x holds q, k, v and the gate's logits at the columns off = (q, k, v, g); zi, zf the input
+    and forget gates' pre-activations; states = (S, n, m) are read and written at the slots."""
+    _memory_check(x, off, zi, zf, out, states, weight, heads, d, dv)
+    S, n, m = states
+    kernel("matrix_memory", "gg_memory_scan")(
+        _p(x), dtype_code(x.dtype), x.stride(0), *(int(o) for o in off), _p(zi), _p(zf), zi.stride(0), _p(out), dtype_code(out.dtype),
+        _p(S), _p(n), _p(m), _p(cu_seqlens), _p(slots), _p(seq_of_token), _p(weight), int(n_tokens), int(n_seqs), int(heads), int(d),
+        int(dv), float(q_scale), float(cap), float(eps), _stream())
 
 
 # ------------------------------------------------------------------------------- vector-state recurrences

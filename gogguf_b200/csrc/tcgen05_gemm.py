@@ -108,7 +108,7 @@ def gemm_tc_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
                  m: Optional[int] = None, swiglu: bool = False, in_ssq: Optional[torch.Tensor] = None,
                  eps: float = 0.0, out_ssq: Optional[torch.Tensor] = None,
                  out_xhat: Optional[torch.Tensor] = None, scratch: Optional[torch.Tensor] = None,
-                 bias: Optional[torch.Tensor] = None) -> None:
+                 bias: Optional[torch.Tensor] = None, out_norm=None, glu_act: int = 0) -> None:
     """`gemm_tc` with an RMSNorm folded in on either side (K splits inside clusters).  bias (float32 [N], not with
     swiglu): added to every row after the norm's factor.
 
@@ -148,6 +148,13 @@ def gemm_tc_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
                 or out_xhat.dtype != torch.bfloat16 or not out_xhat.is_contiguous() or out_xhat.shape[-1] != N \
                 or out_ssq.numel() < M * ((N + 127) // 128) or out_xhat.numel() < M * N:
             raise KernelError("gemm_tc_norm: out_ssq is float32 [M, ceil(N / 128)], out_xhat bfloat16 [M, N]")
+    if out_norm is not None:
+        # (alpha, weight, bias): out_xhat gets the updated rows' dynamic tanh, finished, instead of their copy
+        if not accumulate or out_xhat is None or any(t.dtype != torch.float32 or t.numel() != N or not t.is_contiguous()
+                                                     for t in out_norm[1:]):
+            raise KernelError("gemm_tc_norm: a norm that comes next has float32 vectors [N] and goes with out_xhat")
+        if out_xhat.dtype != torch.bfloat16 or not out_xhat.is_contiguous() or out_xhat.shape[-1] != N or out_xhat.numel() < M * N:
+            raise KernelError("gemm_tc_norm: out_xhat is bfloat16 [M, N]")
     if bias is not None and (swiglu or bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != N):
         raise KernelError("gemm_tc_norm: a bias is float32 [N] and does not go with the fused SwiGLU")
     st = status_word(x.device)
@@ -155,7 +162,9 @@ def gemm_tc_norm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
         x.data_ptr(), w.data_ptr(), out.data_ptr(), mode, M, N, K, x.stride(0), out.stride(0),
         in_ssq.data_ptr() if in_ssq is not None else 0, in_parts, float(eps),
         out_ssq.data_ptr() if out_ssq is not None else 0, out_xhat.data_ptr() if out_xhat is not None else 0,
-        bias.data_ptr() if bias is not None else 0, scratch.data_ptr() if scratch is not None else 0, scratch.numel() if scratch is not None else 0,
+        bias.data_ptr() if bias is not None else 0, out_norm[1].data_ptr() if out_norm is not None else 0,
+        out_norm[2].data_ptr() if out_norm is not None else 0, float(out_norm[0]) if out_norm is not None else 0.0, int(glu_act),
+        scratch.data_ptr() if scratch is not None else 0, scratch.numel() if scratch is not None else 0,
         st.data_ptr(), torch.cuda.current_stream().cuda_stream)
 
 
@@ -198,8 +207,8 @@ def gemm_tc_qkv_rope(x: torch.Tensor, w: torch.Tensor, m: int, q_out: torch.Tens
         st.data_ptr(), torch.cuda.current_stream().cuda_stream)
 
 
-def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable]:
-    """A callable f(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None) for this
+def make_linear(weight: torch.Tensor, swiglu: bool = False, glu_act: int = 0) -> Optional[Callable]:
+    """A callable f(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None, out_norm=None) for this
     weight, or None if its sizes are not taken (K must be a multiple of 8 so that rows start on 16-byte
     boundaries for TMA).  swiglu=True: the weight is interleaved gate/up (see `interleave_gate_up`) and
     out is [M, N / 2].  The keyword arguments are those of `gemm_tc_norm`; a call that has to fall back
@@ -212,8 +221,8 @@ def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable
 
     split_room: Dict[int, int] = {}      # tokens -> floats of scratch with which the prefill form splits K
 
-    def run(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None):
-        folded = in_ssq is not None or out_ssq is not None
+    def run(x, out, accumulate, m, ws, in_ssq=None, eps=0.0, out_ssq=None, out_xhat=None, bias=None, out_norm=None):
+        folded = in_ssq is not None or out_xhat is not None
         if x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
             if swiglu or folded:
                 raise KernelError("fused product: activations must be 16-byte aligned rows")
@@ -228,8 +237,8 @@ def make_linear(weight: torch.Tensor, swiglu: bool = False) -> Optional[Callable
                 need = split_room[M] = pair_scratch_elems(M, N, K)
             if need:
                 scratch = ws.get("gemm_partial_tiles", (need,), torch.float32)
-        if folded or bias is not None:
-            gemm_tc_norm(x, weight, out, accumulate, m, swiglu, in_ssq, eps, out_ssq, out_xhat, scratch, bias)
+        if folded or bias is not None or (swiglu and glu_act):
+            gemm_tc_norm(x, weight, out, accumulate, m, swiglu, in_ssq, eps, out_ssq, out_xhat, scratch, bias, out_norm, glu_act)
         else:
             gemm_tc(x, weight, out, accumulate, m, scratch, cluster=True, swiglu=swiglu)
 

@@ -259,6 +259,9 @@ class Stepper:
                     prep(ctx)
         for i, e in enumerate(m.spec.schedule):
             block = m.blocks[e.block]
+            # the norm the next block starts with, for products that can apply it to the rows they leave
+            follows = m.blocks[m.spec.schedule[i + 1].block] if i + 1 < len(m.spec.schedule) else None
+            ctx.shared["next_norm"] = getattr(follows, "entry_norm", None) if getattr(follows, "normed_ahead", False) else None
             block.forward(x, ctx, self.cache.view(i), e.cache_of is None)
             stats = ctx.shared.get("row_stats")
             if stats is not None and not getattr(block, "keeps_row_stats", False):

@@ -109,6 +109,19 @@ class RowStats:
         return self
 
 
+class NormedRows:
+    """The rows that the next part reads where the norm before it works element by element (no sum over a row): a
+    product that adds into the residual stream can apply such a norm to the values it has just updated, so `rows` is
+    finished when the part starts and no norm kernel runs.  `norm` is the norm whose turn comes next (None: nobody
+    knows) and offers `emit` = (alpha, weight, bias); `fresh` says whether `rows` holds that norm of the residual rows as
+    they are now (see RowStats for who clears and sets it)."""
+
+    def __init__(self, rows: torch.Tensor):
+        self.rows = rows
+        self.norm = None
+        self.fresh = False
+
+
 class Linear:
     """y = x W^T (+ bias) for a weight W[N, K]; float32 accumulation, optional add into a float32 output.  The bias
     [N] is kept in float32 and added to the float32 sums inside the product.
@@ -117,20 +130,21 @@ class Linear:
     core kernel otherwise (and always in the 32-bit path and for a matrix stored in 32-bit).
 
     `fold_input_norm` turns the projection into one that reads `RowStats` instead of normalised rows;
-    `emit=stats` asks an accumulating product to write the statistics of the rows it updates.
+    `emit=stats` asks an accumulating product to write the statistics of the rows it updates, or (`NormedRows`) those
+    rows behind the norm that comes next.  swiglu: the fused gated unit, `glu_act` its activation (K.GLU_ACTS).
     """
 
     def __init__(self, weight: torch.Tensor, rt: Runtime, swiglu: bool = False,
-                 bias: Optional[torch.Tensor] = None):
+                 bias: Optional[torch.Tensor] = None, glu_act: int = 0):
         self.rt = rt
         self.weight = rt.matrix(weight)
         self.out_features, self.in_features = self.weight.shape
-        self.swiglu = swiglu
+        self.swiglu, self.glu_act = swiglu, glu_act
         self.folded_eps: Optional[float] = None
         self._fast = None
         if rt.fast and rt.dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16:
             from ..csrc import tcgen05_gemm
-            self._fast = tcgen05_gemm.make_linear(self.weight, swiglu=swiglu)
+            self._fast = tcgen05_gemm.make_linear(self.weight, swiglu=swiglu, glu_act=glu_act)
         self.bias = rt.vector(bias) if bias is not None else None
         if self.bias is not None and (swiglu or self.bias.numel() != self.out_features):
             raise ValueError("Linear: a bias has one number per output and does not go with the fused SwiGLU form")
@@ -148,7 +162,7 @@ class Linear:
         from ..csrc import tcgen05_gemm
         w = (self.weight.float() * norm_weight.to(self.weight.device).float()[None, :]).to(torch.bfloat16).contiguous()
         self.weight = w
-        self._fast = tcgen05_gemm.make_linear(w, swiglu=self.swiglu)
+        self._fast = tcgen05_gemm.make_linear(w, swiglu=self.swiglu, glu_act=self.glu_act)
         self.folded_eps = float(eps)
 
     @property
@@ -172,7 +186,7 @@ class Linear:
         tcgen05_gemm.gemm_tc_qkv_rope(x, self.weight, m, **outputs)
 
     def __call__(self, x, out: torch.Tensor, accumulate: bool = False, m: Optional[int] = None,
-                 ws: Optional[Workspace] = None, emit: Optional[RowStats] = None) -> None:
+                 ws: Optional[Workspace] = None, emit=None) -> None:
         kw = {}
         if self.folded_eps is not None:
             if not isinstance(x, RowStats):
@@ -181,7 +195,13 @@ class Linear:
             x = x.xhat
         elif isinstance(x, RowStats):
             raise TypeError("Linear: RowStats given to a projection without a folded norm")
-        if (emit is not None and accumulate and self._fast is not None and x.dtype == torch.bfloat16
+        if isinstance(emit, NormedRows):
+            if (emit.norm is not None and accumulate and self._fast is not None and x.dtype == torch.bfloat16
+                    and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and out.is_contiguous()
+                    and out.shape[-1] == emit.rows.shape[-1] and x.data_ptr() != emit.rows.data_ptr()):
+                kw.update(out_xhat=emit.rows, out_norm=emit.norm.emit)
+                emit.fresh = True
+        elif (emit is not None and accumulate and self._fast is not None and x.dtype == torch.bfloat16
                 and x.data_ptr() != emit.xhat.data_ptr() and out.shape[-1] == emit.xhat.shape[-1]
                 and out.is_contiguous()):
             kw.update(out_ssq=emit.ssq, out_xhat=emit.xhat)

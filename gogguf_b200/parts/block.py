@@ -7,33 +7,65 @@ import torch
 
 from ..config.spec import BlockSpec
 from ..csrc import kernels as K
-from .base import RowStats, Runtime, StepContext
+from .base import NormedRows, RowStats, Runtime, StepContext
 from .registry import register_arrangement
 
 
 @register_arrangement("pre_norm")
 class PreNormBlock:
     """x += mixer(norm1(x)); x += feed_forward(norm2(x)) (pkg/model/qwen3/model.go:198-288).
-    The residual stream x is float32; the parts add their outputs into it."""
+    The residual stream x is float32; the parts add their outputs into it.  The feed-forward (with its norm) may be
+    absent.  Where the norms work element by element (they offer `emit`), a part's last product leaves the rows behind
+    the norm that comes next (`NormedRows`): this block's second norm, or the next block's first, which the stepper
+    names in ctx.shared["next_norm"]."""
 
     # role -> family: what a block of this arrangement is made of (the builder builds exactly these)
     roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm"}
+    optional_roles = ("feed_forward", "feed_forward_norm")
     keeps_row_stats = True      # clears RowStats.fresh itself before each write to the residual
 
     def __init__(self, spec: BlockSpec, parts: Dict[str, object], rt: Runtime):
         self.parts = dict(parts)
-        mixer, feed_forward = parts["mixer"], parts["feed_forward"]
-        mixer_norm, feed_forward_norm = parts["mixer_norm"], parts["feed_forward_norm"]
+        mixer, feed_forward = parts["mixer"], parts.get("feed_forward")
+        mixer_norm, feed_forward_norm = parts["mixer_norm"], parts.get("feed_forward_norm")
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("pre_norm: a feed-forward and feed_forward_norm come together")
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
         self.rt = rt
         # A part may take its pre-norm into its first projection (`absorb_norm(norm) -> bool`); it then
         # gets the residual's RowStats as `h` instead of normalised rows, and the norm kernel does not run.
         self.mixer_folded = _offer_norm(mixer, mixer_norm, rt)
-        self.feed_forward_folded = _offer_norm(feed_forward, feed_forward_norm, rt)
+        self.feed_forward_folded = feed_forward is not None and _offer_norm(feed_forward, feed_forward_norm, rt)
+        self.entry_norm = mixer_norm               # what a block before this one may apply for it
+        # element-wise norms, applied by the products before them (bfloat16 rows of the tensor-core products)
+        self.normed_ahead = (rt.fast and rt.fold_norms and rt.dtype == torch.bfloat16 and hasattr(mixer_norm, "emit")
+                             and (feed_forward is None or hasattr(feed_forward_norm, "emit")))
+
+    def _forward_ahead(self, x: torch.Tensor, ctx: StepContext, cache, writes_cache: bool) -> None:
+        ahead = ctx.shared.get("row_stats")
+        if not isinstance(ahead, NormedRows):
+            ahead = ctx.shared["row_stats"] = NormedRows(ctx.ws.get("block_normed", tuple(x.shape), self.rt.dtype))
+        next_norm = ctx.shared.get("next_norm")
+        next_norm = next_norm if hasattr(next_norm, "emit") else None
+        steps = [(self.mixer_norm, lambda h: self.mixer.forward(h, x, ctx, cache, writes_cache))]
+        if self.feed_forward is not None:
+            steps.append((self.feed_forward_norm, lambda h: self.feed_forward.forward(h, x, ctx)))
+        for i, (norm, run) in enumerate(steps):
+            if not (ahead.fresh and ahead.norm is norm):
+                norm.forward(x, ahead.rows)
+            ahead.fresh = False            # the part is about to change the residual rows
+            ahead.norm = steps[i + 1][0] if i + 1 < len(steps) else next_norm
+            run(ahead.rows)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache, writes_cache: bool) -> None:
+        if self.normed_ahead:
+            self._forward_ahead(x, ctx, cache, writes_cache)
+            return
         stats = ctx.shared.get("row_stats")
+        if isinstance(stats, NormedRows):          # (a block of the other make ran before)
+            ctx.shared.pop("row_stats")
+            stats = None
         if stats is None and (self.mixer_folded or self.feed_forward_folded):
             T, H = x.shape
             stats = ctx.shared["row_stats"] = RowStats(
@@ -41,8 +73,9 @@ class PreNormBlock:
                 ctx.ws.get("residual_ssq", (T, (H + 127) // 128), torch.float32))
         h = self._input(self.mixer_folded, self.mixer_norm, x, ctx, stats)
         self.mixer.forward(h, x, ctx, cache, writes_cache)
-        h = self._input(self.feed_forward_folded, self.feed_forward_norm, x, ctx, stats)
-        self.feed_forward.forward(h, x, ctx)
+        if self.feed_forward is not None:
+            h = self._input(self.feed_forward_folded, self.feed_forward_norm, x, ctx, stats)
+            self.feed_forward.forward(h, x, ctx)
 
     def _input(self, folded: bool, norm, x: torch.Tensor, ctx: StepContext, stats):
         if folded:

@@ -209,7 +209,11 @@ class RoutedExperts:
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
         if self.shared is not None:
+            # (its last product is not this part's last add into the stream: it must not be offered the stream's rows)
+            ahead = ctx.shared.pop("row_stats", None)
             self.shared.forward(h, residual, ctx)
+            if ahead is not None:
+                ctx.shared["row_stats"] = ahead
         self._routed(h, residual, ctx)
 
     def _routed(self, h: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:

@@ -4,7 +4,8 @@
 ``names`` of the spec renames the stored matrices (keys gate, up, down, row_gate).  ``row_gate`` (optional, True):
 a stored vector g of the input's width (names key row_gate, stored [1, hidden] or [hidden]) makes one gate per
 token, and the unit's output is multiplied by sigmoid(g . h); the factor goes onto the activation rows in float32,
-before the down projection (which is linear).
+before the down projection (which is linear).  ``activation`` (default "silu", or "gelu_tanh": the tanh form of gelu)
+is the gate's.
 
 `gelu_mlp`: down( gelu(up h) ), no bias; ``approximate`` "none" (default: the exact erf form) or "tanh"."""
 from __future__ import annotations
@@ -41,6 +42,10 @@ class SwiGLU:
     def __init__(self, spec: PartSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
         self.hidden = int(spec["hidden_size"])
         self.inter = int(spec["intermediate_size"])
+        act = spec.get("activation", "silu")
+        if act not in K.GLU_ACTS:
+            raise ValueError(f"swiglu: activation={act!r} is not known ({', '.join(sorted(K.GLU_ACTS))})")
+        self.act = K.GLU_ACTS[act]
         n = self._names(spec)
         g, u = rt.matrix(weights[n["gate"]]), rt.matrix(weights[n["up"]])
         if g.dtype != u.dtype:
@@ -52,7 +57,7 @@ class SwiGLU:
             # gate and up rows interleaved in blocks of 64: the product's epilogue applies silu(gate) * up
             # and writes the activation directly, so the [T, 2 I] intermediate never exists
             from ..csrc import tcgen05_gemm
-            self.fused = Linear(tcgen05_gemm.interleave_gate_up(g, u), rt, swiglu=True)
+            self.fused = Linear(tcgen05_gemm.interleave_gate_up(g, u), rt, swiglu=True, glu_act=self.act)
         if self.fused is None:
             # gate rows first, then up rows: one product for both, then the activation kernel
             self.gate_up = Linear(torch.cat([g, u], dim=0), rt)
@@ -75,7 +80,7 @@ class SwiGLU:
         else:
             gu = ctx.ws.get("ffn_gate_up", (T, 2 * self.inter), self.rt.dtype)
             self.gate_up(h, gu, ws=ctx.ws)
-            K.swiglu(gu, act, T, self.inter)
+            K.swiglu(gu, act, T, self.inter, self.act)
         if self.row_gate is not None:
             K.row_gate(act, h, self.row_gate, ctx.seq_of_token, T)
         self.down(act, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))

@@ -11,15 +11,23 @@
     S_t = exp(-exp(A_log_h) dt) S_(t-1) + dt B_t x_t^T,   y_t = S_t^T C_t + D_h x_t      head h reads group h / (heads / groups)
     out = W_o ( groupnorm(y * silu(z); norm_groups runs) * w )                           the gate comes before the norm
 
+`mamba1` (a selective scan: a diagonal state per channel, its decay, input and read-out made from the token; state: a
+matrix [inner, state]):
+    W_in h = [x: inner | z: inner],  x <- silu(conv(x));   W_x x = [r: dt_rank | B: state | C: state]
+    dt = softplus(W_dt r + b_dt),  A = -exp(A_log) [inner, state]
+    S_t[c, n] = exp(dt_c A[c, n]) S_(t-1)[c, n] + dt_c x_c B_n,   y_c = sum_n S_t[c, n] C_n + D_c x_c
+    out = W_o (y * silu(z))
+
 conv(v)_t = bias + sum_j c[:, j] v_(t - taps + 1 + j) inside a sequence (the last tap meets the token itself, zeros
 before the start).  What a layer keeps per sequence is the convolution's last taps - 1 inputs and S (two
 `StateRequest`s: the part's cache request is the pair), so prompts may come in portions and decoding goes on from
-them.  The projections of h run as one product on the compute dtype's rows and matrices and leave their float32
-sums unrounded; the convolution's sums, the gates, decays, step sizes, the state, the outputs' norm and gate are
+them.  The projections of h run as one product on the compute dtype's rows and matrices and (`rglru`, `mamba2`) leave
+their float32 sums unrounded; in `mamba1` x, z, r, B and C are rounded to the compute dtype and the step sizes'
+pre-activations are not; the convolution's sums, the gates, decays, step sizes, the state, the outputs' norm and gate are
 float32 in both compute paths.
 
 Spec parameters: hidden_size, taps, names; `rglru`: width, blocks, decay_scale (8 unless given); `mamba2`:
-num_heads, value_dim, state_dim, groups, norm_groups, eps.
+num_heads, value_dim, state_dim, groups, norm_groups, eps; `mamba1`: inner, state_dim, dt_rank.
 """
 from __future__ import annotations
 
@@ -198,3 +206,92 @@ class Mamba2Mixer:
         y = ctx.ws.get("mamba2_out", (T, inner), self.rt.dtype)
         K.stepsize_finish(raw, xc, p, 0, self.skip, self.norm_weight, y, ctx.seq_of_token, T, H, P, self.norm_groups, self.eps)
         self.o(y, residual, accumulate=True, ws=ctx.ws)
+
+
+@register_mixer("mamba1")
+class Mamba1Mixer:
+    @classmethod
+    def _names(cls, spec: PartSpec) -> Dict[str, str]:
+        n = dict(in_proj="in", conv="conv", conv_bias="conv.b", x_proj="x", dt="dt", dt_bias="dt.b", a_log="A_log", skip="D", o="o")
+        n.update(spec.get("names") or {})
+        return n
+
+    @classmethod
+    def _sizes(cls, spec: PartSpec):
+        return tuple(int(spec[k]) for k in ("hidden_size", "inner", "state_dim", "dt_rank", "taps"))
+
+    @classmethod
+    def tensors(cls, spec: PartSpec) -> Dict[str, TensorDecl]:
+        W, C, N, R, taps = cls._sizes(spec)
+        n = cls._names(spec)
+        return {n["in_proj"]: TensorDecl(shape=(2 * C, W)), n["conv"]: TensorDecl(shape=(C, taps), init="small_normal"),
+                n["conv_bias"]: TensorDecl(shape=(C,), init="zeros_normal"), n["x_proj"]: TensorDecl(shape=(R + 2 * N, C)),
+                n["dt"]: TensorDecl(shape=(C, R)), n["dt_bias"]: TensorDecl(shape=(C,), init="small_normal"),
+                n["a_log"]: TensorDecl(shape=(C, N), init="small_normal"), n["skip"]: TensorDecl(shape=(C,), init="ones_normal"),
+                n["o"]: TensorDecl(shape=(W, C))}
+
+    @classmethod
+    def cache_request(cls, spec: PartSpec):
+        _, C, N, _, taps = cls._sizes(spec)
+        tail = StateRequest(shape=(taps - 1, C), dtype=torch.float32) if taps > 1 else None
+        return (tail, StateRequest(shape=(C, N), dtype=torch.float32))
+
+    def __init__(self, spec: PartSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
+        self.rt = rt
+        self.hidden, self.C, self.N, self.R, self.taps = self._sizes(spec)
+        if self.taps < 1:
+            raise ValueError("mamba1: taps must be at least 1")
+        if self.N > K.SELECTIVE_MAX_STATE:
+            raise ValueError(f"mamba1: states of {self.N} are not supported (at most {K.SELECTIVE_MAX_STATE})")
+        n = self._names(spec)
+        self.proj = Linear(weights[n["in_proj"]], rt)               # rows: x, z
+        self.conv = rt.vector(weights[n["conv"]]).t().contiguous()  # [taps, channels]
+        self.conv_bias = rt.vector(weights[n["conv_bias"]])
+        # the rows [r | B | C] are filled up to 16 bytes, and so are the columns that read r: what lies behind r in the row
+        # (B's first numbers) meets zeros
+        xp, dt = rt.matrix(weights[n["x_proj"]]), rt.matrix(weights[n["dt"]])
+        self.kdt = -(-self.R // 8) * 8
+        rows = max(-(-xp.shape[0] // 8) * 8, self.kdt)
+        if rows != xp.shape[0]:
+            xp = torch.cat([xp, xp.new_zeros((rows - xp.shape[0], self.C))], dim=0)
+        if self.kdt != self.R:
+            dt = torch.cat([dt, dt.new_zeros((self.C, self.kdt - self.R))], dim=1)
+        self.x_proj = Linear(xp, rt)
+        self.dt = Linear(dt, rt, bias=weights[n["dt_bias"]])
+        self.a = (-torch.exp(rt.vector(weights[n["a_log"]]))).contiguous()
+        self.skip = rt.vector(weights[n["skip"]])
+        self.o = Linear(weights[n["o"]], rt)
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx: StepContext, cache, writes_cache: bool = True) -> None:
+        if not writes_cache:
+            raise ValueError("mamba1: a layer's state cannot be read by another layer")
+        tail, st = _states(cache, "mamba1")
+        T, C, N, dtype = ctx.n_tokens, self.C, self.N, self.rt.dtype
+        p = ctx.ws.get("mamba1_proj", (T, 2 * C), dtype)
+        self.proj(h, p, ws=ctx.ws)
+        x = ctx.ws.get("mamba1_conv", (T, C), dtype)
+        K.column_conv(p[:, :C], x, self.conv, self.conv_bias, None, tail.state if tail is not None else None, ctx.cu_seqlens,
+                      ctx.slots, ctx.seq_of_token, T, ctx.n_seqs, act=1, max_new=int(ctx.max_new))
+        low = ctx.ws.get("mamba1_low", (T, self.x_proj.out_features), dtype)
+        self.x_proj(x, low, ws=ctx.ws)
+        step = ctx.ws.get("mamba1_dt", (T, C), torch.float32)
+        self.dt(low[:, :self.kdt], step, ws=ctx.ws)
+        y = ctx.ws.get("mamba1_out", (T, C), dtype)
+        chunk, scratch = selective_chunk(int(ctx.max_new), ctx.n_seqs, C, N), None
+        if chunk:
+            scratch = ctx.ws.get("mamba1_chunk_states", (K.selective_scan_scratch(T, ctx.n_seqs, C, N, chunk),), torch.float32)
+        K.selective_scan(x, p[:, C:], low, self.R, self.R + N, step, y, st.state, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
+                         self.a, self.skip, T, ctx.n_seqs, chunk=chunk, scratch=scratch)
+        self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
+
+
+def selective_chunk(max_new: int, n_seqs: int, channels: int, states: int) -> int:
+    """Rows per chunk of a selective scan (0: every sequence walked whole).  The chunked form computes every row's decays
+    twice, so it pays only where the channels alone leave most of the GPU idle and the prompts are long."""
+    lanes = 1
+    while 4 * lanes < states and lanes < 32:
+        lanes *= 2
+    warps = n_seqs * channels * lanes // 32
+    if max_new < CHUNKED_FROM or warps * 3 >= 148 * 4:
+        return 0
+    return 64

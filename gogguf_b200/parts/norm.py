@@ -41,6 +41,33 @@ class RMSNorm:
         K.rmsnorm(x, self.weight, self.eps, out, rows)
 
 
+@register_norm("dynamic_tanh")
+class DynamicTanh:
+    """out = tanh(alpha x) * weight + bias with a stored scalar alpha: no mean, no variance, no sum over the row.  The
+    stored tensors are ``tensor`` (default "weight") and, with ".alpha" and ".b" added to that name, the scalar and the
+    bias.  A product that adds into the residual stream can apply it to what it has just updated (`emit`, see
+    parts.base.NormedRows)."""
+
+    foldable = False
+
+    @classmethod
+    def tensors(cls, spec: PartSpec) -> Dict[str, TensorDecl]:
+        name = spec.get("tensor", "weight")
+        return {name: TensorDecl(shape=(spec["size"],), init="ones_normal"),
+                name + ".alpha": TensorDecl(shape=(), init="half"),
+                name + ".b": TensorDecl(shape=(spec["size"],), init="zeros_normal")}
+
+    def __init__(self, spec: PartSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
+        self.size = int(spec["size"])
+        name = spec.get("tensor", "weight")
+        self.alpha = float(weights[name + ".alpha"].double())
+        self.weight, self.bias = rt.vector(weights[name]), rt.vector(weights[name + ".b"])
+        self.emit = (self.alpha, self.weight, self.bias)
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        K.dynamic_tanh(x, self.alpha, self.weight, self.bias, out, rows)
+
+
 @register_norm("group_rmsnorm")
 class GroupRMSNorm:
     """RMS norm in groups: the row is cut into `groups` equal consecutive runs, each is divided by its own

@@ -74,6 +74,32 @@ class RotaryYarn(RotaryNeoX):
         self.key = ("rope_yarn", self.theta, dims, factor, original, fast, slow, self.magnitude)
 
 
+@register_position("rope_banded")
+class RotaryBanded(RotaryNeoX):
+    """NeoX pairing with frequencies scaled by bands of wavelength, for contexts beyond the trained length: with l = 2 pi /
+    f_i the positions a pair needs for one turn, pairs with l < original / high keep f_i, pairs with l > original / low are
+    slowed to f_i / factor, and between the two s = (original / l - low) / (high - low) mixes them, (1 - s) f_i / factor +
+    s f_i.  Parameters: theta, rotary_dim, factor, low, high, original."""
+
+    def __init__(self, params: Dict[str, Any], rt: Runtime):
+        super().__init__(params, rt)
+        factor, low, high, original = (float(params[k]) for k in ("factor", "low", "high", "original"))
+        if not (factor > 0 and low > 0 and high > 0 and original > 0):
+            raise ValueError("rope_banded: factor, low, high and original must be positive")
+        scaled = []
+        for f in self.inv_freq.tolist():
+            turns = original * f / (2.0 * math.pi)          # original / l
+            if turns > high:
+                scaled.append(f)
+            elif turns < low:
+                scaled.append(f / factor)
+            else:
+                s = (turns - low) / (high - low) if high != low else 1.0
+                scaled.append((1.0 - s) * f / factor + s * f)
+        self.inv_freq = torch.tensor(scaled, dtype=torch.float64, device=self.inv_freq.device)
+        self.key = ("rope_banded", self.theta, self.rotary_dim, factor, low, high, original)
+
+
 @register_position("rope_adjacent")
 class RotaryAdjacent(RotaryNeoX):
     """The same angles with the other pairing: element 2i turns with element 2i + 1 (the interleaved layout),

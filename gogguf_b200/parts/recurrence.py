@@ -200,3 +200,90 @@ class Hgrn2Mixer(_MatrixStateMixer):
 
     def _gate_args(self) -> Dict[str, object]:
         return dict(forget_bias=self.f_bias, forget_lower=self.lower, act_q=self.act_q, act_v=self.act_v)
+
+
+@register_mixer("mlstm")
+class MatrixMemoryMixer:
+    """A matrix memory with exponential gates, a normaliser and a running maximum (the matrix memory of xLSTM):
+
+        q = dim^(-1/2) W_q h, k = W_k h [heads x dim], v = W_v h [heads x vdim]
+        i = cap tanh((W_i h + b_i) / cap),  f = log sigmoid(cap tanh((W_f h + b_f) / cap))        one number per head each
+        m_t = max(f + m_(t-1), i)  (m_0 = 0),   S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T,  n_t alike with k alone
+        o = S_t^T q / (max(|n_t . q|, e^(-m_t)) + 1e-6)
+        y = W_o ( concat_h(o_h / rms(o_h)) * w * sigmoid(W_g h) )                                  w: [heads vdim]
+
+    What a layer keeps per sequence is S, n and m (three float32 `StateRequest`s: the part's cache request is the triple).
+    q, k, v and the output gate's logits come in the compute dtype, the gates' pre-activations in float32; everything from
+    there to the rows for the output product is float32.  Prompts of the 16-bit path run in chunks on the tensor cores
+    (csrc/matrix_memory_chunks.cu), everything else token by token.
+
+    Spec parameters: hidden_size, num_heads, head_dim, value_dim, gate_cap, eps, names."""
+
+    @classmethod
+    def _names(cls, spec: PartSpec) -> Dict[str, str]:
+        n = dict(q="q", k="k", v="v", g="g", i="i", i_bias="i.b", f="f", f_bias="f.b", norm="norm", o="o")
+        n.update(spec.get("names") or {})
+        return n
+
+    @classmethod
+    def tensors(cls, spec: PartSpec) -> Dict[str, TensorDecl]:
+        W, H, d, dv = _MatrixStateMixer._sizes(spec)
+        n = cls._names(spec)
+        return {n["q"]: TensorDecl(shape=(H * d, W)), n["k"]: TensorDecl(shape=(H * d, W)), n["v"]: TensorDecl(shape=(H * dv, W)),
+                n["g"]: TensorDecl(shape=(H * dv, W)), n["i"]: TensorDecl(shape=(H, W)),
+                n["i_bias"]: TensorDecl(shape=(H,), init="small_normal"), n["f"]: TensorDecl(shape=(H, W)),
+                n["f_bias"]: TensorDecl(shape=(H,), init="small_normal"),
+                n["norm"]: TensorDecl(shape=(H * dv,), init="ones_normal"), n["o"]: TensorDecl(shape=(W, H * dv))}
+
+    @classmethod
+    def cache_request(cls, spec: PartSpec):
+        _, H, d, dv = _MatrixStateMixer._sizes(spec)
+        return tuple(StateRequest(shape=s, dtype=torch.float32) for s in ((H, d, dv), (H, d), (H,)))
+
+    def __init__(self, spec: PartSpec, weights: Dict[str, torch.Tensor], rt: Runtime):
+        self.rt = rt
+        self.hidden, self.H, self.d, self.dv = _MatrixStateMixer._sizes(spec)
+        self.cap, self.eps = float(spec["gate_cap"]), float(spec["eps"])
+        if not self.cap > 0:
+            raise ValueError("mlstm: gate_cap must be positive")
+        H, d, dv = self.H, self.d, self.dv
+        n = self._names(spec)
+        mats = [rt.matrix(weights[n[key]]) for key in ("q", "k", "v", "g", "i", "f")]
+        if len({m.dtype for m in mats}) != 1:
+            mats = [m.float() for m in mats]
+        self.off = (0, H * d, 2 * H * d, H * (2 * d + dv))
+        cols = H * 2 * (d + dv)
+        self.gates_at = -(-cols // 8) * 8            # the gates' rows start, like every token's row, on a 16-byte boundary
+        gates = [mats[4], mats[5], mats[4].new_zeros((-(2 * H) % 8, self.hidden))]
+        w = torch.cat(mats[:4] + [mats[0].new_zeros((self.gates_at - cols, self.hidden))] + gates, dim=0)
+        bias = torch.cat([rt.vector(weights[n["i_bias"]]), rt.vector(weights[n["f_bias"]])])
+        whole = torch.cat([bias.new_zeros(self.gates_at), bias, bias.new_zeros(w.shape[0] - self.gates_at - 2 * H)])
+        # few rows: one product for everything, its float32 sums unrounded.  Prompts: q, k, v and the output gate's logits in
+        # the compute dtype, the gates' pre-activations (which go through exponentials) in float32 by a product of their own
+        self.proj = Linear(w, rt, bias=whole)
+        self.proj_rows = Linear(w[:self.gates_at], rt)
+        self.proj_gates = Linear(w[self.gates_at:], rt, bias=whole[self.gates_at:])
+        self.norm_weight = rt.vector(weights[n["norm"]])
+        self.o = Linear(weights[n["o"]], rt)
+        self._chunked = (os.environ.get("GOGGUF_B200_MEMORY_CHUNKED", "1") != "0" and rt.fast and rt.dtype == torch.bfloat16)
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx: StepContext, cache, writes_cache: bool = True) -> None:
+        if not writes_cache:
+            raise ValueError("mlstm: a layer's state cannot be read by another layer")
+        if not isinstance(cache, tuple) or len(cache) != 3:
+            raise ValueError("mlstm: the memory's three states are expected")
+        states = tuple(c.state for c in cache)
+        T, H, d, dv = ctx.n_tokens, self.H, self.d, self.dv
+        if ctx.max_new == 1 or self.rt.dtype == torch.float32:
+            row = ctx.ws.get("mlstm_proj", (T, self.proj.out_features), torch.float32)
+            self.proj(h, row, ws=ctx.ws)
+            gates = row[:, self.gates_at:]
+        else:
+            row = ctx.ws.get("mlstm_proj", (T, self.gates_at), self.rt.dtype)
+            self.proj_rows(h, row, ws=ctx.ws)
+            gates = ctx.ws.get("mlstm_gates", (T, self.proj_gates.out_features), torch.float32)
+            self.proj_gates(h, gates, ws=ctx.ws)
+        y = ctx.ws.get("mlstm_out", (T, H * dv), self.rt.dtype)
+        K.memory_scan(row, self.off, gates[:, :H], gates[:, H:2 * H], y, states, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
+                      self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
+        self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
