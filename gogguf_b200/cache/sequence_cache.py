@@ -21,7 +21,8 @@ What each scheduled layer needs is asked of its mixer as a *request*:
   while the rest of its state is its own.
 * a tuple of requests - a mixer made of several mixers asks for one cache or state per member; each
   member's request is grouped and stored as if a layer of its own had made it, and the layer is
-  handed the tuple of their views.
+  handed the tuple of their views.  A member may be such a tuple itself (a mixer of mixers one of which keeps two
+  things); its place in the layer's tuple then holds the tuple of its views.
 
 A sequence's length lives here once, for all groups; a step first *plans* (checks capacity and
 reserves pages for the tokens it brings, all or nothing), the kernels write keys and values at
@@ -366,11 +367,17 @@ class SequenceCache:
         self.stores: List[CacheStore] = []        # every store, paged or not
         self.groups: List[PagedStore] = []        # the paged ones, in the order of their page tables
         self._views: Dict[int, object] = {}
-        # a store's "entry" is a schedule entry i, or (i, k) for member k of a tuple of requests
+        # a store's "entry" is a schedule entry i, or (i, k, ...) for member k of a tuple of requests
         shared: Dict[Tuple[type, object], list] = {}
         own: List[Tuple[type, object, list]] = []
         member_views: Dict[object, object] = {}
-        tuples: Dict[int, int] = {}
+        nested: Dict[int, object] = {}            # schedule entry -> its (possibly nested) tuple of requests
+
+        def leaves(path, r):
+            if isinstance(r, (tuple, list)):
+                return [leaf for k, m in enumerate(r) for leaf in leaves(path + (k,), m)]
+            return [(path if len(path) > 1 else path[0], r)]
+
         single: Dict[object, object] = {}
         borrowed: Dict[object, SharedView] = {}
         for i, (rq, src) in enumerate(zip(requests, cache_of)):
@@ -380,11 +387,8 @@ class SequenceCache:
                 self._views[i] = None
                 continue
             if isinstance(rq, (tuple, list)):
-                tuples[i] = len(rq)
-                members = [((i, k), r) for k, r in enumerate(rq)]
-            else:
-                members = [(i, rq)]
-            for entry, r in members:
+                nested[i] = rq
+            for entry, r in leaves((i,), rq):
                 if r is None:
                     member_views[entry] = None
                     continue
@@ -430,8 +434,14 @@ class SequenceCache:
         for e, v in member_views.items():
             if not isinstance(e, tuple):
                 self._views[e] = v
-        for i, n in tuples.items():
-            self._views[i] = tuple(member_views[(i, k)] for k in range(n))
+
+        def views(path, r):
+            if isinstance(r, (tuple, list)):
+                return tuple(views(path + (k,), m) for k, m in enumerate(r))
+            return member_views[path]
+
+        for i, rq in nested.items():
+            self._views[i] = views((i,), rq)
         # fixed-size states by schedule entry (kept for callers that look at them directly)
         self.states: Dict[object, torch.Tensor] = {e: st.state for st in self.stores if isinstance(st, StateStore)
                                                    for e in st.entries}
