@@ -301,20 +301,42 @@ __device__ __forceinline__ float attn_sink_sum(float l, float m, const float* __
     return l + fast_exp2(sink[head] * 1.4426950408889634f - m);
 }
 
-template <int D>
+// What the kernels below take beside one head size of 64 or 128: the key and value heads' own sizes d and dv (multiples
+// of 8, at most the templates' DK and DV: what lies beyond them in a tile is zeros), chunks of positions (a position sees
+// its own chunk only, counted from the sequence's start; 0: none), and a gate per output element (the result is
+// multiplied by sigmoid(gate[token, head dv + i]); null: none).  EXACT kernels are those with d = DK and dv = DV.
+struct AttnShape {
+    int d, dv, chunk;
+    const bf16* gate;
+    long long ldg;
+};
+__device__ __forceinline__ float attn_gate(float v, const AttnShape& sh, int tok, int col) {
+    if (sh.gate == nullptr) return v;
+    return v / (1.0f + __expf(-__bfloat162float(sh.gate[(size_t)tok * sh.ldg + col])));
+}
+// the first position that a query at position p reads
+__device__ __forceinline__ int attn_first(int p, int window, int chunk) {
+    int lo = 0;
+    if (window > 0 && p - window + 1 > 0) lo = p - window + 1;
+    if (chunk > 0) lo = max(lo, p / chunk * chunk);
+    return lo;
+}
+
+template <int DK, int DV, bool EXACT>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const bf16* q, const bf16* k_pool, const bf16* v_pool, bf16* __restrict__ out,
     const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens, const int* __restrict__ seq_of_token,
     const int* __restrict__ page_table, int max_pages, int n_seqs, int nq, int nkv, float scale_log2, int window,
-    const float* __restrict__ sink, float out_scale, const PageBounds pb) {
+    const float* __restrict__ sink, float out_scale, const AttnShape sh, const PageBounds pb) {
     pdl_wait();      // no early release of the next kernel: many waves of CTAs that exclude its CTAs from their SMs
-    constexpr int CH = D / 8;        // 16-byte chunks per row
-    constexpr int KS = D / 16;       // k-steps of Q.K^T
-    constexpr int NT = D / 8;        // output n-tiles
+    constexpr int CK = DK / 8, CV = DV / 8;      // 16-byte chunks per row
+    constexpr int KS = DK / 16;      // k-steps of Q.K^T
+    constexpr int NT = DV / 8;       // output n-tiles
+    const int d = EXACT ? DK : sh.d, dv = EXACT ? DV : sh.dv;
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);
-    bf16* Ks = Qs + 64 * D;          // two stages
-    bf16* Vs = Ks + 2 * 64 * D;      // two stages
+    bf16* Ks = Qs + 64 * DK;         // two stages
+    bf16* Vs = Ks + 2 * 64 * DK;     // two stages
 
     // which (sequence, query tile) is this CTA?  tiles are numbered sequence by sequence
     int b = -1, tile = blockIdx.x, n_new = 0, tok0 = 0;
@@ -334,25 +356,29 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const int pos0 = ctx_lens[b] - n_new + row0;             // absolute position of query row 0
     const int* pt = page_table + (size_t)b * max_pages;
 
-    int lo = 0;
-    if (window > 0 && pos0 - window + 1 > 0) lo = pos0 - window + 1;
+    const int lo = attn_first(pos0, window, sh.chunk);
     const int kt_first = lo / PAGE, kt_last = (pos0 + rows - 1) / PAGE;
 
     // ---- stage Q (rows beyond the tile are zero) and the first K/V tile
-    for (int idx = threadIdx.x; idx < 64 * CH; idx += 128) {
-        const int r = idx / CH, c = idx - r * CH;
-        bf16* dst = sw<D>(Qs, r, c);
-        if (r < rows) cp_async16(dst, q + ((size_t)(tok0 + row0 + r) * nq + h) * D + c * 8);
+    for (int idx = threadIdx.x; idx < 64 * CK; idx += 128) {
+        const int r = idx / CK, c = idx - r * CK;
+        bf16* dst = sw<DK>(Qs, r, c);
+        if (r < rows && (EXACT || c * 8 < d)) cp_async16(dst, q + ((size_t)(tok0 + row0 + r) * nq + h) * d + c * 8);
         else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
     }
     auto load_kv = [&](int kt, int stage) {
-        const size_t base = (((size_t)gg_page(pt, kt, max_pages, pb, 43) * nkv + kvh) * PAGE) * D;
-        bf16* kd = Ks + stage * 64 * D;
-        bf16* vd = Vs + stage * 64 * D;
-        for (int idx = threadIdx.x; idx < 64 * CH; idx += 128) {
-            const int r = idx / CH, c = idx - r * CH;
-            cp_async16(sw<D>(kd, r, c), k_pool + base + (size_t)r * D + c * 8);
-            cp_async16(sw<D>(vd, r, c), v_pool + base + (size_t)r * D + c * 8);
+        const size_t base = (((size_t)gg_page(pt, kt, max_pages, pb, 43) * nkv + kvh) * PAGE);
+        bf16* kd = Ks + stage * 64 * DK;
+        bf16* vd = Vs + stage * 64 * DV;
+        for (int idx = threadIdx.x; idx < 64 * CK; idx += 128) {
+            const int r = idx / CK, c = idx - r * CK;
+            if (EXACT || c * 8 < d) cp_async16(sw<DK>(kd, r, c), k_pool + (base + r) * d + c * 8);
+            else *reinterpret_cast<uint4*>(sw<DK>(kd, r, c)) = make_uint4(0, 0, 0, 0);
+        }
+        for (int idx = threadIdx.x; idx < 64 * CV; idx += 128) {
+            const int r = idx / CV, c = idx - r * CV;
+            if (EXACT || c * 8 < dv) cp_async16(sw<DV>(vd, r, c), v_pool + (base + r) * dv + c * 8);
+            else *reinterpret_cast<uint4*>(sw<DV>(vd, r, c)) = make_uint4(0, 0, 0, 0);
         }
     };
     load_kv(kt_first, 0);
@@ -373,10 +399,10 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
         __syncthreads();
         if (kt == kt_first) {
 #pragma unroll
-            for (int ks = 0; ks < KS; ++ks) ldsm_x4(qa[ks], sw<D>(Qs, qrow + (lane & 15), ks * 2 + (lane >> 4)));
+            for (int ks = 0; ks < KS; ++ks) ldsm_x4(qa[ks], sw<DK>(Qs, qrow + (lane & 15), ks * 2 + (lane >> 4)));
         }
-        const bf16* kd = Ks + stage * 64 * D;
-        const bf16* vd = Vs + stage * 64 * D;
+        const bf16* kd = Ks + stage * 64 * DK;
+        const bf16* vd = Vs + stage * 64 * DV;
         // rows of this warp that can see any key of this tile?  (whole-warp decision, keeps barriers aligned)
         const int key0 = kt * PAGE;
         float s[8][4];
@@ -387,12 +413,13 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
 #pragma unroll
             for (int np = 0; np < 4; ++np) {       // pairs of n-tiles (16 keys)
                 uint32_t kb[4];
-                ldsm_x4(kb, sw<D>(const_cast<bf16*>(kd), np * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
+                ldsm_x4(kb, sw<DK>(const_cast<bf16*>(kd), np * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
                 mma16816(s[2 * np], qa[ks], kb[0], kb[1]);
                 mma16816(s[2 * np + 1], qa[ks], kb[2], kb[3]);
             }
         }
         // ---- mask + online softmax
+        const int first[2] = {attn_first(pos0 + qrow + g, window, sh.chunk), attn_first(pos0 + qrow + g + 8, window, sh.chunk)};
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt)
@@ -401,8 +428,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
                 const int r = qrow + g + 8 * (e >> 1);
                 const int p = pos0 + r;
                 const int kidx = key0 + nt * 8 + 2 * t + (e & 1);
-                bool ok = kidx <= p;
-                if (window > 0) ok = ok && (kidx > p - window);
+                const bool ok = kidx <= p && kidx >= first[e >> 1];
                 const float v = ok ? s[nt][e] * scale_log2 : -INFINITY;
                 s[nt][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -439,7 +465,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
 #pragma unroll
             for (int np = 0; np < NT / 2; ++np) {
                 uint32_t vb[4];
-                ldsm_x4_trans(vb, sw<D>(const_cast<bf16*>(vd), kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
+                ldsm_x4_trans(vb, sw<DV>(const_cast<bf16*>(vd), kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
                 mma16816(o[2 * np], pa, vb[0], vb[1]);
                 mma16816(o[2 * np + 1], pa, vb[2], vb[3]);
             }
@@ -459,10 +485,14 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
         if (row >= rows) continue;
         const float lr = attn_sink_sum(l[r], m[r], sink, h);
         const float inv = lr > 0.f ? out_scale / lr : 0.f;
-        bf16* dst = out + ((size_t)(tok0 + row0 + row) * nq + h) * D;
+        bf16* dst = out + ((size_t)(tok0 + row0 + row) * nq + h) * dv;
 #pragma unroll
-        for (int i = 0; i < NT; ++i)
-            *reinterpret_cast<uint32_t*>(dst + i * 8 + 2 * t) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
+        for (int i = 0; i < NT; ++i) {
+            const int c = i * 8 + 2 * t, tok = tok0 + row0 + row;
+            if (EXACT || i * 8 < dv)
+                *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(attn_gate(o[i][2 * r] * inv, sh, tok, h * dv + c),
+                                                                  attn_gate(o[i][2 * r + 1] * inv, sh, tok, h * dv + c + 1));
+        }
     }
 }
 
@@ -485,22 +515,23 @@ constexpr int ATT_RECV_ML = 16 * 16 * 2 * 4;
 constexpr int ATT_RECV_BYTES = ATT_RECV_O + ATT_RECV_ML;
 
 
-template <int D, int STAGES>
+template <int DK, int DV, int STAGES, bool EXACT>
 __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
     const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     const bf16* q, bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
     const int* __restrict__ positions, const int* __restrict__ seq_of_token,
     const int* __restrict__ page_table, int max_pages, int nq, int nkv, float scale_log2, int window, int nsplit,
     int cluster_reduce, int early_release, const float* __restrict__ sink, float out_scale, int n_pages,
-    int* __restrict__ status) {
+    int* __restrict__ status, const AttnShape sh) {
     // A grid that is resident as a whole lets the next kernel's CTAs in at once: they share the SMs' free
     // shared memory and start fetching weights.  A grid of several waves releases only after its pages (the
     // rule on dependent launches in common.cuh): until then its own waiting CTAs should get the SMs.
     if (early_release) pdl_launch();
-    constexpr int HALVES = D / 64;
+    constexpr int HK = DK / 64, HV = DV / 64;
     constexpr int BOX_BYTES = 64 * 64 * 2;                 // 8 KB
-    constexpr int STAGE_BYTES = 2 * HALVES * BOX_BYTES;    // K halves then V halves
-    constexpr int KS = D / 16, NT = D / 8;
+    constexpr int STAGE_BYTES = (HK + HV) * BOX_BYTES;     // K halves then V halves
+    constexpr int KS = DK / 16, NT = DV / 8;
+    const int d = EXACT ? DK : sh.d, dv = EXACT ? DV : sh.dv;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint64_t* full = (uint64_t*)(smem + STAGES * STAGE_BYTES);
@@ -532,7 +563,7 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
 
     int lo = 0, p_begin = 0, p_end = 0;
     if (b >= 0) {
-        if (window > 0 && pos - window + 1 > 0) lo = pos - window + 1;
+        lo = attn_first(pos, window, sh.chunk);
         const int first = lo / PAGE, last = pos / PAGE;
         const int pps = (last - first + 1 + nsplit - 1) / nsplit;
         p_begin = first + split * pps;
@@ -559,10 +590,9 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
                 const int row = (gg_page(pt, p_begin + i, max_pages, PageBounds{n_pages, status}, 44) * nkv + kvh) * PAGE;
                 uint8_t* dst = smem + s * STAGE_BYTES;
 #pragma unroll
-                for (int hf = 0; hf < HALVES; ++hf) {
-                    tma::load_2d(dst + hf * BOX_BYTES, &tmK, &full[s], hf * 64, row);
-                    tma::load_2d(dst + (HALVES + hf) * BOX_BYTES, &tmV, &full[s], hf * 64, row);
-                }
+                for (int hf = 0; hf < HK; ++hf) tma::load_2d(dst + hf * BOX_BYTES, &tmK, &full[s], hf * 64, row);
+#pragma unroll
+                for (int hf = 0; hf < HV; ++hf) tma::load_2d(dst + (HK + hf) * BOX_BYTES, &tmV, &full[s], hf * 64, row);
             }
         }
     } else if (npg > 0) {
@@ -570,14 +600,15 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
         uint32_t qa[KS][4];
         pdl_wait();
         {
-            const bf16* q0 = q + ((size_t)tok * nq + (size_t)kvh * G) * D;
+            const bf16* q0 = q + ((size_t)tok * nq + (size_t)kvh * G) * d;
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
                 const int c = ks * 16 + 2 * t;
-                qa[ks][0] = g < G ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)g * D + c) : 0u;
-                qa[ks][1] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)(g + 8) * D + c) : 0u;
-                qa[ks][2] = g < G ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)g * D + c + 8) : 0u;
-                qa[ks][3] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)(g + 8) * D + c + 8) : 0u;
+                const bool in0 = EXACT || c < d, in1 = EXACT || c + 8 < d;
+                qa[ks][0] = g < G && in0 ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)g * d + c) : 0u;
+                qa[ks][1] = g + 8 < G && in0 ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)(g + 8) * d + c) : 0u;
+                qa[ks][2] = g < G && in1 ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)g * d + c + 8) : 0u;
+                qa[ks][3] = g + 8 < G && in1 ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)(g + 8) * d + c + 8) : 0u;
             }
         }
         const int krow = warp * 16;     // this warp's 16 keys of every page
@@ -628,7 +659,7 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
                 }
 #pragma unroll
                 for (int np = 0; np < NT / 2; ++np) {
-                    const bf16* box = reinterpret_cast<const bf16*>(st + (HALVES + (np >> 2)) * BOX_BYTES);
+                    const bf16* box = reinterpret_cast<const bf16*>(st + (HK + (np >> 2)) * BOX_BYTES);
                     uint32_t vb[4];
                     ldsm_x4_trans(vb, sw<64>(const_cast<bf16*>(box), krow + (lane & 7) + (((lane >> 3) & 1) << 3), (np & 3) * 2 + (lane >> 4)));
                     mma16816(o[2 * np], pa, vb[0], vb[1]);
@@ -647,10 +678,10 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
         while (clock64() - t0 < 2000000LL) { }       // let copies in flight land before the CTA goes away
         __syncthreads();
     }
-    float* sm_o = reinterpret_cast<float*>(smem);                 // [4][16][D]
-    float* sm_ml = sm_o + 4 * 16 * D;                             // [4][16][2]
-    float* res_o = sm_ml + 4 * 16 * 2;                            // [16][D]  this CTA's merged output (cluster form)
-    float* res_ml = res_o + 16 * D;                               // [16][2]
+    float* sm_o = reinterpret_cast<float*>(smem);                 // [4][16][DV]
+    float* sm_ml = sm_o + 4 * 16 * DV;                            // [4][16][2]
+    float* res_o = sm_ml + 4 * 16 * 2;                            // [16][DV]  this CTA's merged output (cluster form)
+    float* res_ml = res_o + 16 * DV;                              // [16][2]
     if (warp < 4) {
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
@@ -661,19 +692,19 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
         if (g < G) {
 #pragma unroll
             for (int n = 0; n < NT; ++n)
-                *reinterpret_cast<float2*>(&sm_o[(warp * 16 + g) * D + n * 8 + 2 * t]) = make_float2(o[n][0], o[n][1]);
+                *reinterpret_cast<float2*>(&sm_o[(warp * 16 + g) * DV + n * 8 + 2 * t]) = make_float2(o[n][0], o[n][1]);
             if (t == 0) { sm_ml[(warp * 16 + g) * 2] = m[0]; sm_ml[(warp * 16 + g) * 2 + 1] = l[0]; }
         }
         if (g + 8 < G) {
 #pragma unroll
             for (int n = 0; n < NT; ++n)
-                *reinterpret_cast<float2*>(&sm_o[(warp * 16 + g + 8) * D + n * 8 + 2 * t]) = make_float2(o[n][2], o[n][3]);
+                *reinterpret_cast<float2*>(&sm_o[(warp * 16 + g + 8) * DV + n * 8 + 2 * t]) = make_float2(o[n][2], o[n][3]);
             if (t == 0) { sm_ml[(warp * 16 + g + 8) * 2] = m[1]; sm_ml[(warp * 16 + g + 8) * 2 + 1] = l[1]; }
         }
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
-        const int r = idx / D, c = idx - r * D;
+    for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) {
+        const int r = idx / dv, c = idx - r * dv;
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, sm_ml[(w * 16 + r) * 2]);
@@ -683,18 +714,19 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
             for (int w = 0; w < 4; ++w) {
                 const float f = fast_exp2(sm_ml[(w * 16 + r) * 2] - M);
                 L += sm_ml[(w * 16 + r) * 2 + 1] * f;
-                acc += sm_o[(w * 16 + r) * D + c] * f;
+                acc += sm_o[(w * 16 + r) * DV + c] * f;
             }
         }
         const int head = kvh * G + r;
         if (nsplit == 1) {
             const float Ls = attn_sink_sum(L, M, sink, head);
-            out[((size_t)tok * nq + head) * D + c] = __float2bfloat16_rn(Ls > 0.f ? acc * out_scale / Ls : 0.f);
-        } else if (cluster_reduce && G * D <= ATT_PUSH_MAX_OUT) {
+            out[((size_t)tok * nq + head) * dv + c] =
+                __float2bfloat16_rn(attn_gate(Ls > 0.f ? acc * out_scale / Ls : 0.f, sh, tok, head * dv + c));
+        } else if (cluster_reduce && G * dv <= ATT_PUSH_MAX_OUT) {
             // straight into the shared memory of the CTA that merges this output (slices of 32 go round the
             // ranks), and this head's (max, sum) to every CTA: no load has to cross the cluster afterwards
             const int chunk = idx >> 5, owner = chunk % nsplit, round = chunk / nsplit;
-            const int rounds = ((G * D + 31) / 32 + nsplit - 1) / nsplit;
+            const int rounds = ((G * dv + 31) / 32 + nsplit - 1) / nsplit;
             st_dsmem_f32(tma::smem_u32(recv_o + (split * rounds + round) * 32 + (idx & 31)), (uint32_t)owner, acc);
             if (c == 0) {
                 for (int k = 0; k < nsplit; ++k) {
@@ -703,24 +735,24 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
                 }
             }
         } else if (cluster_reduce) {
-            res_o[r * D + c] = acc;
+            res_o[r * dv + c] = acc;
             if (c == 0) { res_ml[r * 2] = M; res_ml[r * 2 + 1] = L; }
         } else {
             const size_t pi = ((size_t)tok * nq + head) * nsplit + split;
-            part_o[pi * D + c] = acc;
+            part_o[pi * dv + c] = acc;
             if (c == 0) { part_ml[pi * 2] = M; part_ml[pi * 2 + 1] = L; }
         }
     }
-    if (cluster_reduce && G * D <= ATT_PUSH_MAX_OUT) {
+    if (cluster_reduce && G * dv <= ATT_PUSH_MAX_OUT) {
         // The splits of one (token, kv head) form a cluster; what the ranks pushed is complete after one barrier,
         // and every CTA merges its slice of the G x D outputs, in rank order, from its own shared memory.
         asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
         asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-        const int rounds = ((G * D + 31) / 32 + nsplit - 1) / nsplit;
+        const int rounds = ((G * dv + 31) / 32 + nsplit - 1) / nsplit;
         for (int round = warp; round < rounds; round += 5) {
             const int idx = (round * nsplit + split) * 32 + lane;
-            if (idx >= G * D) continue;
-            const int r = idx / D;
+            if (idx >= G * dv) continue;
+            const int r = idx / dv;
             float M = -INFINITY;
             for (int k = 0; k < nsplit; ++k) M = fmaxf(M, recv_ml[(k * 16 + r) * 2]);
             float L = 0.f, acc = 0.f;
@@ -732,15 +764,16 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
                 }
             }
             const float Ls = attn_sink_sum(L, M, sink, kvh * G + r);
-            out[((size_t)tok * nq + kvh * G) * D + idx] = __float2bfloat16_rn(Ls > 0.f ? acc * out_scale / Ls : 0.f);
+            out[((size_t)tok * nq + kvh * G) * dv + idx] =
+                __float2bfloat16_rn(attn_gate(Ls > 0.f ? acc * out_scale / Ls : 0.f, sh, tok, kvh * G * dv + idx));
         }
     } else if (cluster_reduce) {
         // (more than 1,024 outputs per kv head do not fit the receive area: the owner pulls instead)
         asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
         asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
         const uint32_t ro = tma::smem_u32(res_o), rm = tma::smem_u32(res_ml);
-        for (int idx = split * blockDim.x + threadIdx.x; idx < G * D; idx += nsplit * blockDim.x) {
-            const int r = idx / D, c = idx - r * D;
+        for (int idx = split * blockDim.x + threadIdx.x; idx < G * dv; idx += nsplit * blockDim.x) {
+            const int r = idx / dv, c = idx - r * dv;
             float ms[MAX_ATT_CLUSTER], ls[MAX_ATT_CLUSTER], as[MAX_ATT_CLUSTER];
             float M = -INFINITY;
 #pragma unroll
@@ -762,17 +795,18 @@ __global__ void __launch_bounds__(160) attn_decode_tma_kernel(
                 }
             }
             const float Ls = attn_sink_sum(L, M, sink, kvh * G + r);
-            out[((size_t)tok * nq + kvh * G + r) * D + c] = __float2bfloat16_rn(Ls > 0.f ? acc * out_scale / Ls : 0.f);
+            out[((size_t)tok * nq + kvh * G + r) * dv + c] =
+                __float2bfloat16_rn(attn_gate(Ls > 0.f ? acc * out_scale / Ls : 0.f, sh, tok, (kvh * G + r) * dv + c));
         }
         asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
         asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
     }
 }
 
-template <int D, int STAGES>
+template <int DK, int DV, int STAGES>
 constexpr int decode_tma_smem() {
-    constexpr int ring = STAGES * 4 * (D / 64) * 64 * 64;     // bytes: STAGES * 2 * HALVES * 8 KB
-    constexpr int merge = (5 * 16 * D + 5 * 16 * 2) * 4;
+    constexpr int ring = STAGES * ((DK + DV) / 64) * 8192;    // bytes: a box of 8 KB per 64 columns of K and of V
+    constexpr int merge = (5 * 16 * DV + 5 * 16 * 2) * 4;
     return (ring > merge ? ring : merge) + 1024 + 256 + ATT_RECV_BYTES;
 }
 
@@ -799,21 +833,21 @@ int attn_max_cluster() {
         int n = 0;
         if (cudaOccupancyMaxActiveClusters(&n, kern, &cfg) != cudaSuccess || n < 8) ok = false;
     };
-    probe(attn_decode_tma_kernel<128, 3>, decode_tma_smem<128, 3>());
-    probe(attn_decode_tma_kernel<64, 4>, decode_tma_smem<64, 4>());
+    probe(attn_decode_tma_kernel<128, 128, 3, true>, decode_tma_smem<128, 128, 3>());
+    probe(attn_decode_tma_kernel<64, 64, 4, true>, decode_tma_smem<64, 64, 4>());
     cudaGetLastError();
     if (ok) v = 16;
     return v;
 }
 
-template <int D, int STAGES>
+template <int DK, int DV, int STAGES, bool EXACT>
 int launch_decode_tma(const CUtensorMap& tk, const CUtensorMap& tv, const void* q, void* out, float* part_o, float* part_ml,
                       const int* positions, const int* seq_of_token, const int* page_table, int max_pages, int ntok,
                       int nq, int nkv, float scale_log2, int window, int splits, bool cluster, const float* sink,
-                      float out_scale, int n_pages, int* status, cudaStream_t stream) {
-    constexpr int smem = decode_tma_smem<D, STAGES>();
+                      float out_scale, int n_pages, int* status, const AttnShape& sh, cudaStream_t stream) {
+    constexpr int smem = decode_tma_smem<DK, DV, STAGES>();
     static bool configured = false;
-    auto kern = attn_decode_tma_kernel<D, STAGES>;
+    auto kern = attn_decode_tma_kernel<DK, DV, STAGES, EXACT>;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
@@ -832,7 +866,7 @@ int launch_decode_tma(const CUtensorMap& tk, const CUtensorMap& tv, const void* 
     const int early = (long long)ntok * nkv * splits <= places ? 1 : 0;
     return gg_launch(kern, grid, dim3(160), smem, stream, cl ? splits : 1, tk, tv, (const bf16*)q, (bf16*)out, part_o,
                      part_ml, positions, seq_of_token, page_table, max_pages, nq, nkv, scale_log2, window, splits, cl,
-                     early, sink, out_scale, n_pages, status);
+                     early, sink, out_scale, n_pages, status, sh);
 }
 
 
@@ -853,17 +887,18 @@ int launch_decode_tma(const CUtensorMap& tk, const CUtensorMap& tv, const void* 
 // its softmax the other's MMAs keep the tensor pipe busy.
 // All exponentials go to the special-function unit: computing a share of them as polynomials on the FMA pipe,
 // and a pass over the scores for their maximum, cost more issue slots than the unit's time they saved.
-template <int D>
+template <int DK, int DV, bool EXACT>
 __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
     bf16* __restrict__ out, const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens,
     const int* __restrict__ seq_of_token, const int* __restrict__ page_table, int max_pages, int n_seqs,
     int nq, int nkv, float scale_log2, int window, const float* __restrict__ sink, float out_scale, int n_pages,
-    int* __restrict__ status) {
-    constexpr int HALVES = D / 64;
+    int* __restrict__ status, const AttnShape sh) {
+    constexpr int HK = DK / 64, HV = DV / 64;
+    const int d = EXACT ? DK : sh.d, dv = EXACT ? DV : sh.dv;
     constexpr int QBOX = 128 * 64 * 2;              // [64 columns x 128 rows] box of Q: 16 KB
     constexpr int KBOX = 64 * 64 * 2;               // [64 columns x 64 rows] box of K or V: 8 KB
-    constexpr int Q_BYTES = HALVES * QBOX, K_STAGE = HALVES * KBOX, V_BYTES = HALVES * KBOX;
+    constexpr int Q_BYTES = HK * QBOX, K_STAGE = HK * KBOX, V_BYTES = HV * KBOX;
     constexpr int TMEM_COLS = 256;
     // The dynamic segment is the only shared memory of this kernel and is asked to start on a 1024-byte
     // boundary (the swizzled tiles need it) instead of being rounded up in the kernel: two CTAs of 96.25 KB share an SM.
@@ -929,8 +964,7 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
     const int row0 = tile * 128;
     const int rows = active ? min(128, n_new - row0) : 0;
     const int pos0 = active ? ctx_lens[b] - n_new + row0 : 0;
-    int lo = 0;
-    if (window > 0 && pos0 - window + 1 > 0) lo = pos0 - window + 1;
+    const int lo = attn_first(pos0, window, sh.chunk);
     const int kt_first = lo / PAGE, kt_last = active ? (pos0 + rows - 1) / PAGE : -1;
     const int ntiles = kt_last - kt_first + 1;
     // tensor memory: two score buffers of 64 columns (the scores of page j + 1 are computed while the softmax
@@ -942,24 +976,25 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
             const int* pt = page_table + (size_t)b * max_pages;
             tma::mbar_expect_tx(q_full, Q_BYTES);
 #pragma unroll
-            for (int hf = 0; hf < HALVES; ++hf) tma::load_2d(Qs + hf * QBOX, &tmQ, q_full, h * D + hf * 64, tok0 + row0);
+            // (columns beyond d are the next head's, or zeros beyond the row: they meet K columns that are zeros)
+            for (int hf = 0; hf < HK; ++hf) tma::load_2d(Qs + hf * QBOX, &tmQ, q_full, h * d + hf * 64, tok0 + row0);
             for (int j = 0; j < ntiles; ++j) {
                 const int s = j & 1;
                 const int row = (gg_page(pt, kt_first + j, max_pages, PageBounds{n_pages, status}, 45) * nkv + kvh) * PAGE;
                 if (!tma::mbar_wait(&k_empty[s], (uint32_t)((j >> 1) & 1) ^ 1u, abort_flag, status, 21)) break;
                 tma::mbar_expect_tx(&k_full[s], K_STAGE);
 #pragma unroll
-                for (int hf = 0; hf < HALVES; ++hf) tma::load_2d(Ks + s * K_STAGE + hf * KBOX, &tmK, &k_full[s], hf * 64, row);
+                for (int hf = 0; hf < HK; ++hf) tma::load_2d(Ks + s * K_STAGE + hf * KBOX, &tmK, &k_full[s], hf * 64, row);
                 const int vs = j % VST;
                 if (!tma::mbar_wait(&v_empty[vs], (uint32_t)((j / VST) & 1) ^ 1u, abort_flag, status, 22)) break;
                 tma::mbar_expect_tx(&v_full[vs], V_BYTES);
 #pragma unroll
-                for (int hf = 0; hf < HALVES; ++hf) tma::load_2d(Vs + vs * V_BYTES + hf * KBOX, &tmV, &v_full[vs], hf * 64, row);
+                for (int hf = 0; hf < HV; ++hf) tma::load_2d(Vs + vs * V_BYTES + hf * KBOX, &tmV, &v_full[vs], hf * 64, row);
             }
         }
     } else if (warp == 5) {
         if (lane == 0 && active) {
-            const uint32_t idesc_qk = tc5::idesc_bf16(128, 64, 0), idesc_pv = tc5::idesc_bf16(128, D, 1);
+            const uint32_t idesc_qk = tc5::idesc_bf16(128, 64, 0), idesc_pv = tc5::idesc_bf16(128, EXACT ? DV : (dv + 15) & ~15, 1);
             const uint32_t q_a = tma::smem_u32(Qs), k_a = tma::smem_u32(Ks), v_a = tma::smem_u32(Vs);
             bool ok = tma::mbar_wait(q_full, 0, abort_flag, status, 23);
             // scores of page j into buffer j & 1
@@ -968,7 +1003,8 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
                 if (!tma::mbar_wait(&k_full[s], (uint32_t)((j >> 1) & 1), abort_flag, status, 24)) return false;
                 tc5::fence_after();
 #pragma unroll
-                for (int ks = 0; ks < D / 16; ++ks) {
+                for (int ks = 0; ks < DK / 16; ++ks) {
+                    if (!EXACT && ks * 16 >= d) break;
                     const uint64_t a = tc5::smem_desc(q_a + (ks >> 2) * QBOX + (ks & 3) * 32, 16, 1024);
                     const uint64_t bb = tc5::smem_desc(k_a + s * K_STAGE + (ks >> 2) * KBOX + (ks & 3) * 32, 16, 1024);
                     tc5::mma(S_t + (uint32_t)(s * 64), a, bb, idesc_qk, ks > 0 ? 1u : 0u);
@@ -1005,7 +1041,7 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
     } else if (active) {
         const int row = threadIdx.x;                       // query row of the tile = tensor-memory lane
         const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
-        const int p = pos0 + row;
+        const int p = pos0 + row, first = attn_first(p, window, sh.chunk), first_last = attn_first(pos0 + 127, window, sh.chunk);
         float m_used = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < ntiles; ++j) {
@@ -1016,15 +1052,13 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
             tc5::ld32(S_t + lane_off + (uint32_t)((j & 1) * 64) + 32, sr + 32);
             tc5::wait_ld();
             const int key0 = (kt_first + j) * PAGE;
-            const bool edge = (key0 + PAGE - 1 > pos0) || (window > 0 && key0 < pos0 + 127 - window + 1);
+            const bool edge = (key0 + PAGE - 1 > pos0) || key0 < first_last;
             // masked keys become minus infinity (the scale is positive)
             if (edge) {
 #pragma unroll
                 for (int c = 0; c < 64; ++c) {
                     const int kidx = key0 + c;
-                    bool vis = kidx <= p;
-                    if (window > 0) vis = vis && (kidx > p - window);
-                    if (!vis) sr[c] = 0xff800000u;
+                    if (kidx > p || kidx < first) sr[c] = 0xff800000u;
                 }
             }
             uint32_t pk[32];
@@ -1083,7 +1117,7 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
                         if (!tma::mbar_wait(pv_done, (uint32_t)((j - 1) & 1), abort_flag, status, 28)) { ok = false; break; }
                         tc5::fence_after();
 #pragma unroll 1
-                        for (int c0 = 0; c0 < D; c0 += 32) {
+                        for (int c0 = 0; c0 < (EXACT ? DV : dv); c0 += 32) {
                             uint32_t orow[32];
                             tc5::ld32(O_t + lane_off + c0, orow);
                             tc5::wait_ld();
@@ -1114,15 +1148,27 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
             tc5::fence_after();
             const float ls = attn_sink_sum(l, m_used, sink, h);
             const float inv = ls > 0.f ? out_scale / ls : 0.f;
-            bf16* dst = out + ((size_t)(tok0 + row0 + row) * nq + h) * D;
+            bf16* dst = out + ((size_t)(tok0 + row0 + row) * nq + h) * dv;
 #pragma unroll 1
-            for (int c0 = 0; c0 < D; c0 += 32) {
+            for (int c0 = 0; c0 < (EXACT ? DV : dv); c0 += 32) {
                 uint32_t orow[32];
                 tc5::ld32(O_t + lane_off + c0, orow);
                 tc5::wait_ld();
                 if (row < rows) {
 #pragma unroll
                     for (int c = 0; c < 32; c += 8) {
+                        if (!EXACT && c0 + c >= dv) break;
+                        if (sh.gate != nullptr) {
+                            const uint4 gv = *reinterpret_cast<const uint4*>(sh.gate + (size_t)(tok0 + row0 + row) * sh.ldg +
+                                                                             h * dv + c0 + c);
+                            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float2 gf = __bfloat1622float2(g2[e]);
+                                orow[c + 2 * e] = __float_as_uint(__uint_as_float(orow[c + 2 * e]) / (1.0f + __expf(-gf.x)));
+                                orow[c + 2 * e + 1] = __float_as_uint(__uint_as_float(orow[c + 2 * e + 1]) / (1.0f + __expf(-gf.y)));
+                            }
+                        }
                         uint32_t pk[4];
 #pragma unroll
                         for (int e = 0; e < 4; ++e)
@@ -1190,34 +1236,53 @@ GG_API gg_attn_decode(const void* q, const void* k_pool, const void* v_pool, voi
     return gg_last_error();
 }
 
+// The sizes the kernels of this file take: d and dv multiples of 8 up to 128, the exact kernels where both are 64 or both
+// 128.  A gate's rows start on 16-byte boundaries.
+static bool attn_shape_ok(int d, int dv, int chunk, const void* gate, long long ldg) {
+    if (d <= 0 || dv <= 0 || d > 128 || dv > 128 || (d & 7) || (dv & 7) || chunk < 0) return false;
+    return gate == nullptr || ((((uintptr_t)gate) & 15) == 0 && (ldg & 7) == 0);
+}
+// call F<DK, DV, EXACT>(...) for the sizes
+#define GG_ATTN_SIZES(F, ...)                                                              \
+    do {                                                                                   \
+        if (d == 128 && dv == 128) return F<128, 128, true>(__VA_ARGS__);                  \
+        if (d == 64 && dv == 64) return F<64, 64, true>(__VA_ARGS__);                      \
+        if (d <= 64 && dv <= 64) return F<64, 64, false>(__VA_ARGS__);                     \
+        if (d <= 64) return F<64, 128, false>(__VA_ARGS__);                                \
+        if (dv <= 64) return F<128, 64, false>(__VA_ARGS__);                               \
+        return F<128, 128, false>(__VA_ARGS__);                                            \
+    } while (0)
+
+template <int DK, int DV, bool EXACT>
+static int launch_attn_prefill(dim3 grid, const void* q, const void* k_pool, const void* v_pool, void* out, const int* cu_seqlens,
+                               const int* ctx_lens, const int* seq_of_token, const int* page_table, int max_pages, int n_seqs,
+                               int nq, int nkv, float scale_log2, int window, const float* sink, float out_scale,
+                               const AttnShape& sh, PageBounds pb, cudaStream_t stream) {
+    constexpr int smem = 64 * (3 * DK + 2 * DV) * 2;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<DK, DV, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    return gg_launch(attn_prefill_kernel<DK, DV, EXACT>, grid, dim3(128), smem, stream, 1, (const bf16*)q, (const bf16*)k_pool,
+                     (const bf16*)v_pool, (bf16*)out, cu_seqlens, ctx_lens, seq_of_token, page_table, max_pages, n_seqs, nq, nkv,
+                     scale_log2, window, sink, out_scale, sh, pb);
+}
+
 // Prefill attention for a ragged batch: sequence i brings tokens cu_seqlens[i]..cu_seqlens[i+1]-1, whose
 // absolute positions end at ctx_lens[i]-1.  max_tiles >= sum over sequences of ceil(new tokens / 64).
 GG_API gg_attn_prefill(const void* q, const void* k_pool, const void* v_pool, void* out, const int* cu_seqlens,
                        const int* ctx_lens, const int* seq_of_token, const int* page_table, int max_pages,
-                       int page_size, int n_pages, int n_seqs, int max_tiles, int nq, int nkv, int d, float scale,
-                       int window, const float* sink, float out_scale, int* status, cudaStream_t stream) {
+                       int page_size, int n_pages, int n_seqs, int max_tiles, int nq, int nkv, int d, int dv, float scale,
+                       int window, int chunk, const float* sink, float out_scale, const void* gate, long long ldg, int* status,
+                       cudaStream_t stream) {
     if (n_seqs <= 0 || max_tiles <= 0) return 0;
-    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || (d != 64 && d != 128) || nq > 65535) return GG_ERR_ARG;
+    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || nq > 65535 || !attn_shape_ok(d, dv, chunk, gate, ldg)) return GG_ERR_ARG;
     const float scale_log2 = scale * 1.4426950408889634f;
-    dim3 grid(max_tiles, nq);
-    const int smem = 5 * 64 * d * 2;
-    cudaError_t e;
-    if (d == 128) {
-        static bool cfg128 = false;
-        if (!cfg128) {
-            e = cudaFuncSetAttribute(attn_prefill_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-            if (e != cudaSuccess) return (int)e;
-            cfg128 = true;
-        }
-        gg_launch(attn_prefill_kernel<128>, dim3(grid), dim3(128), smem, stream, 1, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out,
-                                                              cu_seqlens, ctx_lens, seq_of_token, page_table, max_pages, n_seqs,
-                                                              nq, nkv, scale_log2, window, sink, out_scale, PageBounds{n_pages, status});
-    } else {
-        gg_launch(attn_prefill_kernel<64>, dim3(grid), dim3(128), smem, stream, 1, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out,
-                                                             cu_seqlens, ctx_lens, seq_of_token, page_table, max_pages, n_seqs,
-                                                             nq, nkv, scale_log2, window, sink, out_scale, PageBounds{n_pages, status});
-    }
-    return gg_last_error();
+    const AttnShape sh = {d, dv, chunk, (const bf16*)gate, ldg};
+    GG_ATTN_SIZES(launch_attn_prefill, dim3(max_tiles, nq), q, k_pool, v_pool, out, cu_seqlens, ctx_lens, seq_of_token, page_table,
+                  max_pages, n_seqs, nq, nkv, scale_log2, window, sink, out_scale, sh, PageBounds{n_pages, status}, stream);
 }
 
 // Splits for the TMA form: whole pages per CTA.  use_cluster != 0: the splits of one (token, kv head)
@@ -1249,48 +1314,71 @@ GG_API gg_attn_decode_tma_splits(int ntok, int nkv, int max_ctx, int use_cluster
 // use_cluster; status as in the tensor-core product (codes 11 producer, 12 consumer).
 GG_API gg_attn_decode_tma(const void* q, const void* k_pool, const void* v_pool, void* out, float* part_o, float* part_ml,
                           const int* positions, const int* seq_of_token, const int* page_table, int max_pages,
-                          int page_size, int n_pages, int ntok, int nq, int nkv, int d, float scale, int window,
-                          int splits, int use_cluster, const float* sink, float out_scale, int* status,
+                          int page_size, int n_pages, int ntok, int nq, int nkv, int d, int dv, float scale, int window, int chunk,
+                          int splits, int use_cluster, const float* sink, float out_scale, const void* gate, long long ldg, int* status,
                           cudaStream_t stream) {
     if (ntok <= 0) return 0;
-    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || nq / nkv > 16 || (d != 64 && d != 128) || splits < 1 ||
+    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || nq / nkv > 16 || splits < 1 || !attn_shape_ok(d, dv, chunk, gate, ldg) ||
         nkv > 65535 || splits > 65535 || n_pages <= 0 || status == nullptr)
         return GG_ERR_ARG;
     const bool cluster = use_cluster != 0;
-    if (cluster && splits > attn_max_cluster()) return GG_ERR_ARG;
+    const bool exact = d == dv && (d == 64 || d == 128);
+    if (cluster && splits > (exact ? attn_max_cluster() : 8)) return GG_ERR_ARG;
     if (splits > 1 && !cluster && (part_o == nullptr || part_ml == nullptr)) return GG_ERR_ARG;
-    // the form that merges its splits by a second kernel knows neither a sink nor a factor on the output
-    if (splits > 1 && !cluster && (sink != nullptr || out_scale != 1.0f)) return GG_ERR_ARG;
+    // the form that merges its splits by a second kernel knows neither a sink, a gate nor a factor on the output
+    if (splits > 1 && !cluster && (!exact || gate != nullptr || sink != nullptr || out_scale != 1.0f)) return GG_ERR_ARG;
     if ((((uintptr_t)k_pool) & 15) || (((uintptr_t)v_pool) & 15)) return GG_ERR_ARG;
     CUtensorMap tk, tv;
     const unsigned long long rows = (unsigned long long)n_pages * nkv * PAGE;
     int rc;
     if ((rc = tma::make_map_bf16(&tk, k_pool, rows, d, d, PAGE)) != 0) return rc;
-    if ((rc = tma::make_map_bf16(&tv, v_pool, rows, d, d, PAGE)) != 0) return rc;
+    if ((rc = tma::make_map_bf16(&tv, v_pool, rows, dv, dv, PAGE)) != 0) return rc;
     const float scale_log2 = scale * 1.4426950408889634f;
-    if (d == 128)
-        rc = launch_decode_tma<128, 3>(tk, tv, q, out, part_o, part_ml, positions, seq_of_token, page_table, max_pages, ntok,
-                                       nq, nkv, scale_log2, window, splits, cluster, sink, out_scale, n_pages, status, stream);
-    else
-        rc = launch_decode_tma<64, 4>(tk, tv, q, out, part_o, part_ml, positions, seq_of_token, page_table, max_pages, ntok,
-                                      nq, nkv, scale_log2, window, splits, cluster, sink, out_scale, n_pages, status, stream);
+    const AttnShape sh = {d, dv, chunk, (const bf16*)gate, ldg};
+#define GG_DTMA(DK_, DV_, ST_, EX_)                                                                                         \
+    launch_decode_tma<DK_, DV_, ST_, EX_>(tk, tv, q, out, part_o, part_ml, positions, seq_of_token, page_table, max_pages, ntok, nq, \
+                                          nkv, scale_log2, window, splits, cluster, sink, out_scale, n_pages, status, sh, stream)
+    if (exact) rc = d == 128 ? GG_DTMA(128, 128, 3, true) : GG_DTMA(64, 64, 4, true);
+    else if (d <= 64 && dv <= 64) rc = GG_DTMA(64, 64, 4, false);
+    else if (d <= 64) rc = GG_DTMA(64, 128, 4, false);
+    else if (dv <= 64) rc = GG_DTMA(128, 64, 4, false);
+    else rc = GG_DTMA(128, 128, 3, false);
+#undef GG_DTMA
     if (rc != 0 || splits == 1 || cluster) return rc;
     if (d == 128) gg_launch(attn_combine_kernel<128>, dim3(ntok * nq), dim3(128), 0, stream, 1, part_o, part_ml, (bf16*)out, splits);
     else gg_launch(attn_combine_kernel<64>, dim3(ntok * nq), dim3(64), 0, stream, 1, part_o, part_ml, (bf16*)out, splits);
     return gg_last_error();
 }
 
-// Prefill attention on tcgen05 (see attn_prefill_tc_kernel).  q and out: [n_tokens, nq, d] bf16, d = 64 or 128;
-// pools [page][nkv][64][d]; max_tiles >= sum over sequences of ceil(new tokens / 128); status as in the
+template <int DK, int DV, bool EXACT>
+static int launch_attn_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, dim3 grid, void* out,
+                                  const int* cu_seqlens, const int* ctx_lens, const int* seq_of_token, const int* page_table,
+                                  int max_pages, int n_seqs, int nq, int nkv, float scale_log2, int window, const float* sink,
+                                  float out_scale, int n_pages, int* status, const AttnShape& sh, cudaStream_t stream) {
+    // Q, K x 2, V x 2 (boxes of 64 columns: 16 KB of Q, 8 KB of K or V), barriers
+    constexpr int smem = (DK / 64) * (16384 + 2 * 8192) + (DV / 64) * 2 * 8192 + 256;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<DK, DV, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    return gg_launch(attn_prefill_tc_kernel<DK, DV, EXACT>, grid, dim3(192), smem, stream, 1, tq, tk, tv, (bf16*)out, cu_seqlens,
+                     ctx_lens, seq_of_token, page_table, max_pages, n_seqs, nq, nkv, scale_log2, window, sink, out_scale, n_pages,
+                     status, sh);
+}
+
+// Prefill attention on tcgen05 (see attn_prefill_tc_kernel).  q [n_tokens, nq, d], out [n_tokens, nq, dv] bf16; pools
+// [page][nkv][64][d] and [..][dv]; max_tiles >= sum over sequences of ceil(new tokens / 128); status as in the
 // tensor-core product (codes 21-28 name the wait that ran out).
 GG_API gg_attn_prefill_tc(const void* q, const void* k_pool, const void* v_pool, void* out, const int* cu_seqlens,
                           const int* ctx_lens, const int* seq_of_token, const int* page_table, int max_pages,
-                          int page_size, int n_pages, int n_tokens, int n_seqs, int max_tiles, int nq, int nkv, int d,
-                          float scale, int window, const float* sink, float out_scale, int* status,
-                          cudaStream_t stream) {
+                          int page_size, int n_pages, int n_tokens, int n_seqs, int max_tiles, int nq, int nkv, int d, int dv,
+                          float scale, int window, int chunk, const float* sink, float out_scale, const void* gate, long long ldg,
+                          int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || max_tiles <= 0 || n_tokens <= 0) return 0;
-    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || (d != 64 && d != 128) || nq > 65535 || max_tiles > 65535 ||
-        n_pages <= 0 || status == nullptr)
+    if (page_size != PAGE || nq <= 0 || nkv <= 0 || nq % nkv || nq > 65535 || max_tiles > 65535 ||
+        n_pages <= 0 || status == nullptr || !attn_shape_ok(d, dv, chunk, gate, ldg))
         return GG_ERR_ARG;
     if ((((uintptr_t)q) & 15) || (((uintptr_t)k_pool) & 15) || (((uintptr_t)v_pool) & 15) || (((uintptr_t)out) & 15)) return GG_ERR_ARG;
     CUtensorMap tq, tk, tv;
@@ -1298,31 +1386,11 @@ GG_API gg_attn_prefill_tc(const void* q, const void* k_pool, const void* v_pool,
     if ((rc = tma::make_map_bf16(&tq, q, (unsigned long long)n_tokens, nq * d, (long long)nq * d, 128)) != 0) return rc;
     const unsigned long long rows = (unsigned long long)n_pages * nkv * PAGE;
     if ((rc = tma::make_map_bf16(&tk, k_pool, rows, d, d, PAGE)) != 0) return rc;
-    if ((rc = tma::make_map_bf16(&tv, v_pool, rows, d, d, PAGE)) != 0) return rc;
+    if ((rc = tma::make_map_bf16(&tv, v_pool, rows, dv, dv, PAGE)) != 0) return rc;
     const float scale_log2 = scale * 1.4426950408889634f;
-    dim3 grid(nq, max_tiles);
-    if (d == 128) {
-        constexpr int smem = 2 * 16384 + 2 * 16384 + 2 * 16384 + 256;   // Q, K x 2, V x 2, barriers
-        static bool cfg = false;
-        if (!cfg) {
-            cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-            if (e != cudaSuccess) return (int)e;
-            cfg = true;
-        }
-        return gg_launch(attn_prefill_tc_kernel<128>, grid, dim3(192), smem, stream, 1, tq, tk, tv, (bf16*)out, cu_seqlens,
-                         ctx_lens, seq_of_token, page_table, max_pages, n_seqs, nq, nkv, scale_log2, window, sink, out_scale, n_pages,
-                         status);
-    }
-    constexpr int smem = 16384 + 2 * 8192 + 2 * 8192 + 256;
-    static bool cfg64 = false;
-    if (!cfg64) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e != cudaSuccess) return (int)e;
-        cfg64 = true;
-    }
-    return gg_launch(attn_prefill_tc_kernel<64>, grid, dim3(192), smem, stream, 1, tq, tk, tv, (bf16*)out, cu_seqlens,
-                     ctx_lens, seq_of_token, page_table, max_pages, n_seqs, nq, nkv, scale_log2, window, sink, out_scale,
-                     n_pages, status);
+    const AttnShape sh = {d, dv, chunk, (const bf16*)gate, ldg};
+    GG_ATTN_SIZES(launch_attn_prefill_tc, tq, tk, tv, dim3(nq, max_tiles), out, cu_seqlens, ctx_lens, seq_of_token, page_table,
+                  max_pages, n_seqs, nq, nkv, scale_log2, window, sink, out_scale, n_pages, status, sh, stream);
 }
 
 // 1 if this library was built with checked page tables (the debug build), else 0.

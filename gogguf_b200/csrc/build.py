@@ -61,6 +61,7 @@ MODULES: Dict[str, str] = {
     "diag_recurrence": "diag_recurrence.cu",
     "selective_scan": "selective_scan.cu",
     "matrix_memory": "matrix_memory.cu",
+    "matrix_memory_chunks": "matrix_memory_chunks.cu",
     "diff_attention": "diff_attention.cu",
     "mixed_head_attention": "mixed_head_attention.cu",
     "mixed_head_prompt": "mixed_head_prompt.cu",

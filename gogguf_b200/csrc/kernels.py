@@ -1019,6 +1019,36 @@ def memory_scan(x: torch.Tensor, off, zi: torch.Tensor, zf: torch.Tensor, out: t
         int(dv), float(q_scale), float(cap), float(eps), _stream())
 
 
+MEMORY_CHUNK = 64             # tokens per chunk (MC_PC in csrc/matrix_memory_chunks.cu)
+
+
+def memory_chunks_takes(d: int, dv: int) -> bool:
+    """Does the chunked form (bfloat16 rows, tensor cores) take these head sizes?"""
+    return all(0 < n <= 128 and n % 8 == 0 for n in (d, dv))
+
+
+def memory_chunks_scratch(n_tokens: int, n_seqs: int, heads: int, d: int, dv: int) -> int:
+    """Floats of scratch `memory_chunks` needs: a state, its sums and maxima per chunk and head."""
+    return (n_tokens // MEMORY_CHUNK + n_seqs) * heads * (d * dv + d + 3)
+
+
+def memory_chunks(x: torch.Tensor, off, zi: torch.Tensor, zf: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, states,
+                  cu_seqlens: torch.Tensor, slots: torch.Tensor, seq_of_token: torch.Tensor, weight: torch.Tensor, n_tokens: int,
+                  n_seqs: int, heads: int, d: int, dv: int, q_scale: float, cap: float, eps: float) -> None:
+    """`memory_scan` for prompts of bfloat16 rows, in chunks of 64 tokens on the tensor cores."""
+    _memory_check(x, off, zi, zf, out, states, weight, heads, d, dv)
+    if x.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+        raise KernelError("memory_chunks takes bfloat16 rows")
+    _need(scratch, torch.float32, "scratch")
+    if scratch.numel() < memory_chunks_scratch(n_tokens, n_seqs, heads, d, dv):
+        raise KernelError("memory_chunks: the scratch is too small")
+    S, n, m = states
+    kernel("matrix_memory_chunks", "gg_memory_chunks")(
+        _p(x), x.stride(0), *(int(o) for o in off), _p(zi), _p(zf), zi.stride(0), _p(out), _p(S), _p(n), _p(m), _p(cu_seqlens),
+        _p(slots), _p(seq_of_token), _p(weight), int(n_tokens), int(n_seqs), int(heads), int(d), int(dv), float(q_scale), float(cap),
+        float(eps), _p(scratch), _stream())
+
+
 # ------------------------------------------------------------------------------- vector-state recurrences
 def rglru_gates(u: torch.Tensor, wa_t: torch.Tensor, wi_t: torch.Tensor, ba: torch.Tensor, bi: torch.Tensor,
                 c: torch.Tensor, a: torch.Tensor, b: torch.Tensor, seq_of_token: torch.Tensor, n_tokens: int) -> None:

@@ -46,12 +46,15 @@ def _block_parts(b: BlockSpec) -> List[Tuple[str, PartSpec, type]]:
 
     The arrangement class says which roles a block of its kind has and which family (registry) each
     role's part comes from; the block spec must name exactly those (roles listed in the arrangement's
-    `optional_roles` may be left out)."""
+    `optional_roles` may be left out, those of a tuple in `roles_together` all or none)."""
     acls = R.lookup(R.ARRANGEMENTS, b.arrangement, "block arrangement")
     roles = getattr(acls, "roles", None)
     if roles is None:
         raise TypeError(f"block arrangement {b.arrangement!r} declares no `roles` (role -> family)")
     optional = set(getattr(acls, "optional_roles", ()))
+    for group in getattr(acls, "roles_together", ()):
+        if any(r in b.parts for r in group):
+            optional -= set(group)
     missing = [r for r in roles if r not in b.parts and r not in optional]
     extra = [r for r in b.parts if r not in roles]
     if missing or extra:

@@ -22,14 +22,13 @@ class PreNormBlock:
     # role -> family: what a block of this arrangement is made of (the builder builds exactly these)
     roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm"}
     optional_roles = ("feed_forward", "feed_forward_norm")
+    roles_together = (("feed_forward", "feed_forward_norm"),)
     keeps_row_stats = True      # clears RowStats.fresh itself before each write to the residual
 
     def __init__(self, spec: BlockSpec, parts: Dict[str, object], rt: Runtime):
         self.parts = dict(parts)
         mixer, feed_forward = parts["mixer"], parts.get("feed_forward")
         mixer_norm, feed_forward_norm = parts["mixer_norm"], parts.get("feed_forward_norm")
-        if (feed_forward is None) != (feed_forward_norm is None):
-            raise ValueError("pre_norm: a feed-forward and feed_forward_norm come together")
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
         self.rt = rt

@@ -284,6 +284,12 @@ class MatrixMemoryMixer:
             gates = ctx.ws.get("mlstm_gates", (T, self.proj_gates.out_features), torch.float32)
             self.proj_gates(h, gates, ws=ctx.ws)
         y = ctx.ws.get("mlstm_out", (T, H * dv), self.rt.dtype)
+        if self._chunked and ctx.max_new >= CHUNKED_FROM and K.memory_chunks_takes(d, dv):
+            scratch = ctx.ws.get("mlstm_chunk_states", (K.memory_chunks_scratch(T, ctx.n_seqs, H, d, dv),), torch.float32)
+            K.memory_chunks(row, self.off, gates[:, :H], gates[:, H:2 * H], y, scratch, states, ctx.cu_seqlens, ctx.slots,
+                            ctx.seq_of_token, self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
+            self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
+            return
         K.memory_scan(row, self.off, gates[:, :H], gates[:, H:2 * H], y, states, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
                       self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
         self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))

@@ -120,8 +120,9 @@ def softmax_attention(q, k, v, scale, mask):
 # ----------------------------------------------------------------------------------------------- mixers
 def chunked_attention(m: dict, w: Dict[str, torch.Tensor], p: str, h: torch.Tensor) -> torch.Tensor:
     n, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = rotate_halves(linear(h, w, p + "q", True).reshape(n, H, d), m["rot"])
-    k = rotate_halves(linear(h, w, p + "k", True).reshape(n, G, d), m["rot"])
+    q, k = linear(h, w, p + "q", True).reshape(n, H, d), linear(h, w, p + "k", True).reshape(n, G, d)
+    if m.get("rot"):
+        q, k = rotate_halves(q, m["rot"]), rotate_halves(k, m["rot"])
     v = linear(h, w, p + "v", True).reshape(n, G, dv)
     o = softmax_attention(q, k, v, m["scale"], unseen(n, h.dtype, m["mask"]["size"])).reshape(n, H * dv)
     return linear(o * sigmoid(linear(h, w, p + "g")), w, p + "o")
