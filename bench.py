@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L] [--impl ours|reference]
                     [--shape 8b|14b|32b] [--workload] [--prefill-lengths 256,1024] [--decode-contexts 16384,32768]
-    python bench.py --compare gigopel|sokirax|felolorn|dinuzen|kulesun [--compare-sizes 2k,4k]   (another workload, see the end of this text)
+    python bench.py --compare gigopel|sokirax|felolorn|dinuzen|kulesun|niresun [--compare-sizes 2k,4k]   (another workload, see the end of this text)
 
 A "step" is one decode step of a batch: every sequence goes on by one token, sampled greedily on the
 device.  The timed region is exactly K steps after W warm-up steps, timed with CUDA events on the
@@ -52,6 +52,12 @@ the heads' outputs, and attention whose heads' weights are mixed; gated dense fe
 layers cycle through two latent layers and one attention layer, beside the dense Sokirax model (the same arrangement
 of norms and the same feed-forward around other mixers), the dense Gigopel model (latent attention of the same sizes)
 and the same Qwen3.  It prints {"compare": "kulesun", "sizes": {...}}.
+
+`--compare niresun` measures the Niresun design (dynamic tanh norms; a selective scan without a feed-forward, attention
+in chunks behind a gate, convolved attention beside a matrix memory; gelu gated units): one model per size whose layers
+cycle through scan, parallel layer, scan and attention, beside the dense Sokirax model (its closest relative: attention
+with a partial, stretched rotation, and attention beside a matrix state of the same sizes), the all-experts Dinuzen model
+(a state space behind a convolution) and the same Qwen3.  It prints {"compare": "niresun", "sizes": {...}}.
 
 Peaks come from MEASURED_PEAKS.json beside this file when the driver wrote it, else from the
 fallback figures of an earlier measurement on this pool.  The weights (16 GB) are far larger than
@@ -320,6 +326,32 @@ def kulesun_config(z):
                         for i in range(z["layers"])])
 
 
+# Niresun at the same widths and depths: Sokirax's attention and matrix-state sizes, a selective scan twice as wide as the
+# stream with 16 states a channel, Sokirax's dense feed-forward in the layers that have one
+NIRESUN_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=8, chunk=1024, mem_heads=8, inner=4096, state=16, dt_rank=128, taps=4, ff=8192,
+               layers=8, vocab=65536),
+    "4k": dict(width=4096, heads=32, kv_heads=8, chunk=2048, mem_heads=16, inner=8192, state=16, dt_rank=256, taps=4, ff=16384,
+               layers=8, vocab=65536),
+}
+
+
+def niresun_config(z):
+    """Layers cycle through selective scan, parallel layer, selective scan and attention in chunks; scans have no
+    feed-forward."""
+    H, G = z["heads"], z["kv_heads"]
+    ssm = dict(inner=z["inner"], state=z["state"], dt_rank=z["dt_rank"], conv=z["taps"])
+    att = dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=z["chunk"]),
+               rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
+    par = dict(left=dict(heads=H, kv_heads=G, dim=64, vdim=64, scale=0.125, conv=z["taps"], q_temp=dict(coef=0.1, every=4096)),
+               right=dict(heads=z["mem_heads"], dim=128, vdim=128, gate_cap=15.0))
+    mlp = dict(kind="dense", ff=(2 * z["ff"] // 3) // 128 * 128)
+    kinds = [dict(type="mamba1", mixer=ssm, mlp=None), dict(type="parallel", mixer=par, mlp=mlp), dict(type="mamba1", mixer=ssm, mlp=None),
+             dict(type="attention", mixer=att, mlp=mlp)]
+    return dict(architecture="Niresun", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), initializer_range=0.02,
+                layers=[kinds[i % 4] for i in range(z["layers"])])
+
+
 def qwen3_like(z):
     """Qwen3 at the same width, depth, head count and feed-forward parameter count (3 matrices instead of 2), with
     full attention (its cache of a 2,048-token context is read whole; Gigopel reads its window)."""
@@ -488,12 +520,33 @@ def compare_run(a):
         per_seq = t * 2 * (n_lat * (R + r) + n_att * 2 * AG * ad)
         return flops, wbytes, per_seq
 
+    def nir_numbers(z, t):
+        """The same figures for a Niresun model whose layers cycle through scan, parallel layer, scan and attention."""
+        W, H, G, R, C, N, D = (z[k] for k in ("width", "heads", "kv_heads", "mem_heads", "inner", "state", "dt_rank"))
+        n = z["layers"] // 4
+        ssm = 2 * C * W + (D + 2 * N) * C + C * D + W * C
+        par = (H * 64 + 2 * G * 64) * W + W * H * 64 + 4 * R * 128 * W + 2 * R * W + W * R * 128
+        att = (2 * H + 2 * G) * 128 * W + W * H * 128              # q, k, v, the gate and the output matrix
+        ff = 3 * W * ((2 * z["ff"] // 3) // 128 * 128)
+        keys, near = t * (t + 1) // 2, sum(i % z["chunk"] + 1 for i in range(t))
+        mix = 2 * n * ssm + n * (par + att + 2 * ff)
+        flops = 2 * t * mix + n * (2 * 2 * H * 64 * keys + 2 * 2 * H * 128 * near + t * (R * 2 * 2 * 128 * 128 + 2 * 6 * C * N))
+        flops += 2 * z["vocab"] * W
+        wbytes = mix * 2 + z["vocab"] * W * 2
+        held = (t - 1) % z["chunk"] + 1
+        per_seq = n * (t * 2 * G * 64 * 2 + held * 2 * G * 128 * 2 + 2 * R * 128 * 128 * 4 + 2 * 2 * C * N * 4)
+        return flops, wbytes, per_seq
+
     out = {}
     T = PROMPT_LEN
     design = a.compare
     for name in [x for x in a.compare_sizes.split(",") if x.strip()]:
         z = GIGOPEL_SIZES[name]
-        if design == "kulesun":
+        if design == "niresun":
+            zs, zd, zn = SOKIRAX_SIZES[name], DINUZEN_SIZES[name], NIRESUN_SIZES[name]
+            arms = [("niresun_dense", niresun_config(zn)), ("sokirax_dense", sokirax_config(zs, "dense")),
+                    ("dinuzen_experts", dinuzen_config(zd)), ("qwen3_like", qwen3_like(z))]
+        elif design == "kulesun":
             zs, zk = SOKIRAX_SIZES[name], KULESUN_SIZES[name]
             arms = [("kulesun_dense", kulesun_config(zk)), ("sokirax_dense", sokirax_config(zs, "dense")),
                     ("gigopel_dense", gigopel_config(z, "dense")), ("qwen3_like", qwen3_like(z))]
@@ -520,6 +573,8 @@ def compare_run(a):
             per_seq = 0
             if arm == "qwen3_like":
                 flops, wbytes = qwen_numbers(cd, z, T)
+            elif arm == "niresun_dense":
+                flops, wbytes, per_seq = nir_numbers(zn, T)
             elif arm == "kulesun_dense":
                 flops, wbytes, per_seq = kul_numbers(zk, T)
             elif arm == "gigopel_dense" and design == "kulesun":
@@ -529,7 +584,7 @@ def compare_run(a):
                 flops, wbytes, per_seq = din_numbers(zd, T)
             elif arm == "felolorn_experts":
                 flops, wbytes, per_seq = fel_numbers(zf, T)
-            elif design in ("sokirax", "felolorn", "kulesun"):
+            elif design in ("sokirax", "felolorn", "kulesun", "niresun"):
                 flops, wbytes, per_seq = sok_numbers(zs, "dense" if arm.endswith("dense") else "moe", T)
             else:
                 flops, wbytes = gig_numbers(z, "dense" if arm.endswith("dense") else "moe", T)
@@ -547,7 +602,7 @@ def compare_run(a):
                     rb -= z["layers"] * (z["experts"] - used) * 3 * z["width"] * z["expert_ff"] * 2
                 if arm == "qwen3_like":
                     rb += b * T * 2 * z["layers"] * 8 * 128 * 2
-                elif design in ("sokirax", "felolorn", "dinuzen", "kulesun"):
+                elif design in ("sokirax", "felolorn", "dinuzen", "kulesun", "niresun"):
                     rb += b * per_seq
                 else:
                     rb += b * min(T, z["window"]) * z["layers"] * (z["kv_rank"] + z["rot_dim"]) * 2
@@ -586,7 +641,7 @@ def main():
                     "decode_by_context)")
     ap.add_argument("--prefill-lengths", default="", help="comma separated prompt lengths: time one prefill step of each "
                     "(printed on stderr, added to the line as prefill_sweep)")
-    ap.add_argument("--compare", default="", choices=["", "gigopel", "sokirax", "felolorn", "dinuzen", "kulesun"],
+    ap.add_argument("--compare", default="", choices=["", "gigopel", "sokirax", "felolorn", "dinuzen", "kulesun", "niresun"],
                     help="another workload: the named design beside Qwen3 at equal size (prefill and decode), see the top")
     ap.add_argument("--compare-sizes", default="2k,4k", help="which of the comparison's layer sizes to run")
     a = ap.parse_args()

@@ -1,4 +1,4 @@
-"""Kernel micro-benchmarks: python -m gogguf_b200.csrc.microbench [gemm|gemm_layer|attn|prefill_attn|sample|latent|retention|recurrence|dinuzen] [--m 1,8,64] [--ctx 2048,8192]
+"""Kernel micro-benchmarks: python -m gogguf_b200.csrc.microbench [gemm|gemm_layer|attn|prefill_attn|sample|latent|retention|recurrence|dinuzen|kulesun|niresun] [--m 1,8,64] [--ctx 2048,8192]
 
 Times single kernels the way a decode step runs them: forty launches captured in a CUDA graph and
 replayed, so that host launch cost is out of the picture and dependent launches overlap as they do
@@ -589,6 +589,125 @@ def kulesun(sizes=((16, 4, 128, 128, 2048), (32, 8, 128, 128, 4096))) -> None:
         torch.cuda.empty_cache()
 
 
+def niresun(sizes=((2048, 4096, 16, 16, 8, 8), (4096, 8192, 16, 32, 8, 16))) -> None:
+    """The kernels of the Niresun design alone, per size (width, inner, state, heads, kv heads, memory heads)."""
+    from . import fast_attention as FA
+    from . import kernels as K
+    from . import tcgen05_gemm as TG
+    dev = "cuda:0"
+    hbm, tfl, src = _peaks()
+    print(f"peaks ({src}): {hbm:.0f} GB/s copy, {tfl:.0f} TFLOP/s bf16", flush=True)
+    bf = torch.bfloat16
+    ints = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+
+    def say(what, us, nbytes=None, flops=None):
+        txt = f"{what:60s} {us:8.1f} us"
+        if nbytes is not None:
+            txt += f"  {nbytes / us / 1e3:8.1f} GB/s ({nbytes / us / 1e3 / hbm:.2f} of the copy bandwidth)"
+        if flops is not None:
+            txt += f"  {flops / us / 1e6:7.1f} TFLOP/s ({flops / us / 1e6 / tfl:.3f} of the bf16 peak)"
+        print(txt, flush=True)
+
+    for W, C, N, H, G, R in sizes:
+        T = 2048
+        cu1, sot1, slot1, ends = ints([0, T]), ints([0] * T), ints([0]), ints([T])
+        # ---- selective scan and the convolution before it
+        A, D = -torch.exp(torch.randn(C, N, device=dev) * 0.5), torch.randn(C, device=dev)
+        xz, x = torch.randn(T, 2 * C, device=dev).to(bf), torch.randn(T, C, device=dev).to(bf)
+        bc, xdt = torch.randn(T, 128 + 2 * N, device=dev).to(bf), torch.randn(T, C, device=dev) - 2
+        out = torch.empty(T, C, device=dev, dtype=bf)
+        cw, cb, tail = torch.randn(4, C, device=dev), torch.randn(C, device=dev), torch.zeros(64, 3, C, device=dev)
+        state = torch.zeros(64, C, N, device=dev)
+        for chunk in (0, 64):
+            scr = torch.empty(K.selective_scan_scratch(T, 1, C, N, chunk), device=dev) if chunk else None
+            us = _time_graph(lambda i: K.selective_scan(x, xz[:, C:], bc, 128, 128 + N, xdt, out, state, cu1, slot1, sot1, A, D, T, 1,
+                                                        chunk=chunk, scratch=scr), 10)
+            say(f"selective scan, prompt, {C} x {N}, T={T}" + (", in chunks" if chunk else ""), us, T * C * 10)
+        us = _time_graph(lambda i: K.column_conv(xz[:, :C], x, cw, cb, None, tail, cu1, slot1, sot1, T, 1, act=1, max_new=T), 10)
+        say(f"convolution of projection columns, T={T}", us, T * C * 4)
+        for B in (8, 64):
+            cu, sot, sl = ints(list(range(B + 1))), ints(list(range(B))), ints(list(range(B)))
+            us = _time_graph(lambda i: K.selective_scan(x[:B], xz[:B, C:], bc[:B], 128, 128 + N, xdt[:B], out[:B], state, cu, sl, sot, A, D,
+                                                        B, B))
+            say(f"selective scan, decode, batch {B}", us, B * C * (2 * N * 4 + 10) + C * N * 4)
+            us = _time_graph(lambda i: K.column_conv(xz[:B, :C], x[:B], cw, cb, None, tail, cu, sl, sot, B, B, act=1, max_new=1))
+            say(f"convolution of projection columns, batch {B}", us, B * C * (4 + 6 * 4))
+        # ---- matrix memory
+        d = dv = 128
+        off = (0, R * d, 2 * R * d, R * (2 * d + dv))
+        row, gates = torch.randn(T, 2 * R * (d + dv), device=dev).to(bf), torch.randn(T, 2 * R, device=dev)
+        st = tuple(torch.zeros(64, *s, device=dev) for s in ((R, d, dv), (R, d), (R,)))
+        y, w = torch.empty(T, R * dv, device=dev, dtype=bf), torch.randn(R * dv, device=dev)
+        scr = torch.empty(K.memory_chunks_scratch(T, 1, R, d, dv), device=dev)
+        us = _time_graph(lambda i: K.memory_chunks(row, off, gates[:, :R], gates[:, R:], y, scr, st, cu1, slot1, sot1, w, T, 1, R, d, dv,
+                                                   d ** -0.5, 15.0, 1e-6), 10)
+        say(f"matrix memory, prompt, {R} heads of {d} x {dv}, T={T}", us, T * R * (2 * d + 3 * dv) * 2, T * R * 2 * 2 * d * dv)
+        for B in (8, 64):
+            cu, sot, sl = ints(list(range(B + 1))), ints(list(range(B))), ints(list(range(B)))
+            rf = torch.randn(B, row.shape[1] + 2 * R, device=dev)
+            us = _time_graph(lambda i: K.memory_scan(rf, off, rf[:, -2 * R:-R], rf[:, -R:], y[:B], st, cu, sl, sot, w, B, B, R, d, dv,
+                                                     d ** -0.5, 15.0, 1e-6))
+            say(f"matrix memory, decode, batch {B}", us, B * R * 2 * d * dv * 4)
+        del st, scr
+        # ---- attention: prompts and decode steps, preparation
+        table = ints([list(range(b * 33, b * 33 + 33)) for b in range(64)])
+        for what, hd, hv, chunk, gated in (("left", 64, 64, 0, False), ("chunked, gated", 128, 128, 1024, True),
+                                           ("plain", 128, 128, 0, False), ("plain", 96, 112, 0, False)):
+            kp, vp = (torch.randn(64 * 33, G, 64, e, device=dev).to(bf) for e in (hd, hv))
+            q, o = torch.randn(T, H * hd, device=dev).to(bf), torch.empty(T, H * hv, device=dev, dtype=bf)
+            gt = torch.randn(T, H * hv, device=dev).to(bf) if gated else None
+            kw = dict(dv=hv, chunk=chunk, gate=gt)
+            keys = sum((i % chunk if chunk else i) + 1 for i in range(T))
+            us = _time_graph(lambda i: FA.attn_prefill_tc(q, kp, vp, o, cu1, ends, sot1, table[:1], 64, T, 1, T // 128 + 1, H, G, hd,
+                                                          hd ** -0.5, 0, **kw), 10)
+            say(f"attention {what} {hd}/{hv}, prompt, T={T}", us, flops=2 * H * (hd + hv) * keys)
+            for B in (8, 64):
+                pos, sot = ints([T - 1] * B), ints(list(range(B)))
+                held = (T - 1) % chunk + 1 if chunk else T
+                ns = min(8, FA.decode_tma_splits(B, G, held, cluster=True))
+                us = _time_graph(lambda i: FA.attn_decode_tma(q[:B], kp, vp, o[:B], pos, sot, table[:B], 64, B, H, G, hd, hd ** -0.5, 0, ns,
+                                                              cluster=True, dv=hv, chunk=chunk, gate=gt[:B] if gated else None))
+                say(f"attention {what} {hd}/{hv}, decode, batch {B}, {held} keys", us, B * held * G * (hd + hv) * 2)
+            if what != "plain":
+                cols = (H + G) * hd + G * hv
+                rows = torch.randn(T, cols, device=dev).to(bf)
+                conv = torch.randn(4, cols, device=dev) if what == "left" else None
+                ct = torch.zeros(64, 3, cols, device=dev)
+                cos, sin = torch.randn(T, 32, device=dev), torch.randn(T, 32, device=dev)
+                for B in (T, 8):
+                    cu, sot, sl = (cu1, sot1, slot1) if B == T else (ints(list(range(B + 1))), ints(list(range(B))), ints(list(range(B))))
+                    pos = ints(list(range(T))) if B == T else ints([T] * B)
+                    us = _time_graph(lambda i: K.qkv_prep(
+                        rows[:B], q[:B], None, None, 1e-6, 1 if conv is not None else 0, cos[:B], sin[:B], pos, sot, table, 64, kp, vp, B, H,
+                        G, hd, hv, 0 if conv is not None else 64, conv=conv, conv_state=ct if conv is not None else None, cu_seqlens=cu,
+                        slots=sl, n_seqs=1 if B == T else B, max_new=T if B == T else 1, coef=0.1 if conv is not None else 0.0), 10)
+                    say(f"preparation of q, k, v ({what}), {B} rows", us, B * cols * 4)
+            del kp, vp
+        # ---- norms, products
+        for m in (8, T):
+            xr, h = torch.randn(m, W, device=dev), torch.empty(m, W, device=dev, dtype=bf)
+            nw, nb = torch.randn(W, device=dev), torch.randn(W, device=dev)
+            us = _time_graph(lambda i: K.dynamic_tanh(xr, 0.5, nw, nb, h))
+            say(f"dynamic tanh, {m} rows of {W}", us, m * W * 6)
+            yy = torch.randn(2, m, W, device=dev)
+            yw = torch.stack([nw, nb])
+            us = _time_graph(lambda i: K.normed_sum(xr, yy, yw, [1e-6, 1e-6], h, (0.5, nw, nb)))
+            say(f"sum of two normed parts + dynamic tanh, {m} rows", us, m * W * (4 * 2 + 2 * 8 + 2))
+            a = torch.randn(m, W, device=dev).to(bf)
+            wm = (torch.randn(W, W, device=dev) * 0.02).to(bf)
+            ssq = torch.empty(m, W // 128, device=dev)
+            t = [_time_graph(lambda i: TG.gemm_tc_norm(a, wm, xr, accumulate=True, **kw)) for kw in
+                 (dict(), dict(out_ssq=ssq, out_xhat=h), dict(out_xhat=h, out_norm=(0.5, nw, nb)))]
+            print(f"product {W} x {W}, {m} rows, added: {t[0]:6.1f} us, with row statistics {t[1]:6.1f} us, with the next dynamic tanh "
+                  f"{t[2]:6.1f} us", flush=True)
+            I = 2 * W
+            wg = (torch.randn(2 * I, W, device=dev) * 0.02).to(bf)
+            act = torch.empty(m, I, device=dev, dtype=bf)
+            t = [_time_graph(lambda i: TG.gemm_tc_norm(a, wg, act, swiglu=True, glu_act=k)) for k in (0, 1)]
+            print(f"gated unit {I} x {W}, {m} rows: silu {t[0]:6.1f} us, gelu {t[1]:6.1f} us", flush=True)
+        torch.cuda.empty_cache()
+
+
 def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps, value_heads=None):
     """A callable that runs attention with mixed heads as the mixer would for a step of those sizes; scratch is made on
     the first call of a size, so that the calls can be captured."""
@@ -616,7 +735,7 @@ def mixed_head_runner(H, G, d, dv, g_off, talk, kw, ps, value_heads=None):
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "gemm_layer", "attn", "prefill_attn", "sample", "latent", "retention", "recurrence", "dinuzen", "kulesun"])
+    ap.add_argument("what", choices=["gemm", "gemm_layer", "attn", "prefill_attn", "sample", "latent", "retention", "recurrence", "dinuzen", "kulesun", "niresun"])
     ap.add_argument("--m", default="1,8,64", help="token counts (gemm), batch sizes (attn) or prompt lengths (prefill_attn)")
     ap.add_argument("--ctx", default="2048", help="attn: cached positions per sequence (comma separated)")
     ap.add_argument("--scratch", action="store_true", help="attn: splits merged by a second kernel instead of inside clusters")
@@ -631,8 +750,8 @@ def main() -> None:
     if a.what == "recurrence":
         recurrence()
         return
-    if a.what in ("dinuzen", "kulesun"):
-        {"dinuzen": dinuzen, "kulesun": kulesun}[a.what]()
+    if a.what in ("dinuzen", "kulesun", "niresun"):
+        {"dinuzen": dinuzen, "kulesun": kulesun, "niresun": niresun}[a.what]()
         return
     if a.what == "attn":
         for c in a.ctx.split(","):
