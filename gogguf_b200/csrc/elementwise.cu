@@ -192,52 +192,77 @@ GG_API gg_dynamic_tanh(const float* x, const int* rows, float alpha, const float
 
 // ----------------------------------------------------------------------------- a sum of normed parts, added
 // x[r, :] += sum_k y_k[r, :] / sqrt(mean(y_k[r, :]^2) + eps_k) * w_k for up to NORMED_MAX parts (y [parts][rows][H],
-// w [parts][H] with any factor of a part's already in it), all float32; y is left zeroed.  With hout the updated row's
-// dynamic tanh (alpha, nw, nb) is left there in the compute dtype too, so the norm that comes next needs no kernel of
-// its own.  One block per row.
+// w [parts][H] with any factor of a part's already in it), all float32; zero_y: y is left zeroed.  With hout the updated
+// row's dynamic tanh (alpha, nw, nb) is left there in the compute dtype too, so the norm that comes next needs no kernel of
+// its own.  One block per row.  KEEP > 0: at most KEEP groups of V columns a thread, whose y (of up to two parts) stay in
+// registers between the sums of squares and the add.
 #define NORMED_MAX 4
 struct NormedEps { float v[NORMED_MAX]; };
 
-template <typename TO, int V>
+template <typename TO, int V, int KEEP>
 __global__ void __launch_bounds__(256) normed_sum_kernel(float* x, float* y, const float* __restrict__ w, int parts, int H,
                                                          long long part_stride, const NormedEps eps, TO* __restrict__ hout,
-                                                         float alpha, const float* __restrict__ nw, const float* __restrict__ nb) {
+                                                         float alpha, const float* __restrict__ nw, const float* __restrict__ nb,
+                                                         int zero_y) {
     pdl_launch();
     pdl_wait();
     __shared__ float red[33];
     const size_t r = blockIdx.x;
-    float f[NORMED_MAX];
-    for (int k = 0; k < parts; ++k) {
+    constexpr int KP = KEEP > 0 ? 2 : NORMED_MAX, KK = KEEP > 0 ? KEEP : 1;
+    float f[KP], kept[KEEP > 0 ? 2 : 1][KK][V];
+#pragma unroll
+    for (int k = 0; k < KP; ++k) {
+        f[k] = 0.f;
+        if (k >= parts) continue;
         const float* yr = y + k * part_stride + r * H;
         float ss = 0.f;
-        for (int i = V * threadIdx.x; i < H; i += V * blockDim.x) {
-            float v[V];
-            load_row_v<V>(yr + i, v);
+        if (KEEP > 0) {
 #pragma unroll
-            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+            for (int j = 0; j < KK; ++j) {
+                const int i = V * (threadIdx.x + j * 256);
+                float* v = kept[KEEP > 0 ? k : 0][j];
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] = 0.f;
+                if (i < H) load_row_v<V>(yr + i, v);
+            }
+#pragma unroll
+            for (int j = 0; j < KK; ++j)
+#pragma unroll
+                for (int e = 0; e < V; ++e) { const float v = kept[KEEP > 0 ? k : 0][j][e]; ss = fmaf(v, v, ss); }
+        } else {
+            for (int i = V * threadIdx.x; i < H; i += V * 256) {
+                float v[V];
+                load_row_v<V>(yr + i, v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+            }
         }
-        ss = block_sum(ss, red);
-        const float g = 1.0f / sqrtf(ss / (float)H + eps.v[k]);
-#pragma unroll
-        for (int j = 0; j < NORMED_MAX; ++j)
-            if (j == k) f[j] = g;
+        f[k] = ss;
     }
+#pragma unroll
+    for (int k = 0; k < KP; ++k)
+        if (k < parts) f[k] = 1.0f / sqrtf(block_sum(f[k], red) / (float)H + eps.v[k]);
     float zero[V];
 #pragma unroll
     for (int e = 0; e < V; ++e) zero[e] = 0.f;
-    for (int i = V * threadIdx.x; i < H; i += V * blockDim.x) {
+    auto finish = [&](int i, int j) {
         float a[V];
         load_row_v<V>(x + r * H + i, a);
 #pragma unroll
-        for (int k = 0; k < NORMED_MAX; ++k) {
+        for (int k = 0; k < KP; ++k) {
             if (k < parts) {
                 float v[V], ww[V];
                 float* yr = y + k * part_stride + r * H + i;
-                load_row_v<V>(yr, v);
+                if (KEEP > 0) {
+#pragma unroll
+                    for (int e = 0; e < V; ++e) v[e] = kept[KEEP > 0 ? k : 0][KEEP > 0 ? j : 0][e];
+                } else {
+                    load_row_v<V>(yr, v);
+                }
                 load_row_v<V>(w + (size_t)k * H + i, ww);
 #pragma unroll
                 for (int e = 0; e < V; ++e) a[e] = fmaf(v[e] * f[k], ww[e], a[e]);
-                store_row_v<float, V>(yr, zero);
+                if (zero_y) store_row_v<float, V>(yr, zero);
             }
         }
         store_row_v<float, V>(x + r * H + i, a);
@@ -249,23 +274,38 @@ __global__ void __launch_bounds__(256) normed_sum_kernel(float* x, float* y, con
             for (int e = 0; e < V; ++e) a[e] = fmaf(tanhf(alpha * a[e]), ww[e], bb[e]);
             store_row_v<TO, V>(hout + r * H + i, a);
         }
+    };
+    if (KEEP > 0) {
+#pragma unroll
+        for (int j = 0; j < KK; ++j) {
+            const int i = V * (threadIdx.x + j * 256);
+            if (i < H) finish(i, j);
+        }
+    } else {
+        for (int i = V * threadIdx.x; i < H; i += V * 256) finish(i, 0);
     }
 }
 
 // hout (rows of H numbers in `out_dtype`) may be null, and nw and nb with it.
 GG_API gg_normed_sum(float* x, float* y, const float* w, int parts, int rows, int H, long long part_stride, float eps0,
                      float eps1, float eps2, float eps3, void* hout, int out_dtype, float alpha, const float* nw, const float* nb,
-                     cudaStream_t stream) {
+                     int zero_y, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (H <= 0 || parts < 1 || parts > NORMED_MAX || (hout != nullptr && (nw == nullptr || nb == nullptr))) return GG_ERR_ARG;
     const NormedEps eps = {{eps0, eps1, eps2, eps3}};
     const bool vec = H % 4 == 0 && part_stride % 4 == 0 &&
                      (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)hout | (uintptr_t)nw | (uintptr_t)nb) & 15) == 0;
+    const int keep = vec && parts <= 2 ? (H <= 1024 ? 1 : H <= 2048 ? 2 : H <= 4096 ? 4 : 0) : 0;
+#define GG_NS(TO_, V_, K_)                                                                                                \
+    gg_launch(normed_sum_kernel<TO_, V_, K_>, dim3(rows), dim3(256), 0, stream, 1, x, y, w, parts, H, part_stride, eps, (TO_*)hout, \
+              alpha, nw, nb, zero_y)
     GG_DISPATCH_DTYPE(out_dtype, TO,
-        if (vec) gg_launch(normed_sum_kernel<TO, 4>, dim3(rows), dim3(256), 0, stream, 1, x, y, w, parts, H, part_stride, eps, (TO*)hout,
-                           alpha, nw, nb);
-        else gg_launch(normed_sum_kernel<TO, 1>, dim3(rows), dim3(256), 0, stream, 1, x, y, w, parts, H, part_stride, eps, (TO*)hout,
-                       alpha, nw, nb));
+        if (keep == 1) GG_NS(TO, 4, 1);
+        else if (keep == 2) GG_NS(TO, 4, 2);
+        else if (keep == 4) GG_NS(TO, 4, 4);
+        else if (vec) GG_NS(TO, 4, 0);
+        else GG_NS(TO, 1, 0));
+#undef GG_NS
     return gg_last_error();
 }
 
@@ -538,6 +578,14 @@ GG_API gg_qk_norm_rope_cache(const void* qkv, int dtype, void* q_out, const floa
 //   then the rotation of the pairs (i, i + rot/2) of the first `rot` elements of every q and k head;
 //   q to q_out[T, nq, d], k into the paged key pool [page][kv_head][page_size][d], v into the paged value pool
 //   [page][kv_head][page_size][dv].  The key and value head sizes may differ.  All arithmetic float32.
+__device__ __forceinline__ void load_elems4(const float* p, float* v) { load_row_v<4>(p, v); }
+__device__ __forceinline__ void load_elems4(const bf16* p, float* v) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x));
+    const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+    v[0] = f0.x; v[1] = f0.y; v[2] = f1.x; v[3] = f1.y;
+}
+
 struct QkvConv {
     const float* w;              // [taps][columns]
     float* state;                // [slots][taps - 1][columns]
@@ -561,6 +609,124 @@ __device__ __forceinline__ float qkv_column(const T* qkv, long long ld, int t, i
         if (cv.one_each) { st[(size_t)j * cols + c] = carry; carry = v; }
     }
     return acc;
+}
+
+// (the quotient in double: where p + 1 is a multiple of `every` the step must not be missed by a rounding)
+__device__ __forceinline__ float qkv_temperature(int pos, float coef, double every) {
+    return coef != 0.f ? 1.f + coef * logf((float)floor(((double)pos + 1.0) / every) + 1.f) : 1.f;
+}
+
+// The same with a warp a head (grid: token, groups of eight of the nq + 2 nkv heads) and four neighbouring elements a
+// lane: heads of up to 128 elements, everything a multiple of four, no norm over the whole projection.
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_prep_head_kernel(
+    const T* qkv, long long ld, T* __restrict__ q_out, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
+    int norm_mode, const float* cosv, const float* sinv, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
+    const int* __restrict__ page_table, int max_pages, int page_size, T* __restrict__ k_pool, T* __restrict__ v_pool, int nq, int nkv,
+    int d, int dv, int rot, const QkvConv cv, float coef, double every, const PageBounds pb) {
+    pdl_launch();
+    pdl_wait();
+    __shared__ float rows[8][128];
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y * 8 + warp;
+    if (head >= nq + 2 * nkv) return;
+    const bool is_q = head < nq, is_v = head >= nq + nkv;
+    const int n = is_v ? dv : d, e = 4 * lane;
+    const bool on = e < n;
+    const int b = seq_of_token[t];
+    T* qd = q_out + ((size_t)t * nq + head) * d + e;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (b < 0) {
+        if (is_q && on) store_row_v<T, 4>(qd, v);
+        return;
+    }
+    const int pos = positions[t];
+    const int cols = (nq + nkv) * d + nkv * dv;
+    const int c = (is_v ? (nq + nkv) * d + (head - nq - nkv) * dv : head * d) + e;
+    if (on) {
+        load_elems4(qkv + (size_t)t * ld + c, v);
+        if (cv.taps) {
+            const int R = cv.taps - 1, start = cv.cu_seqlens[b];
+            float* st = R ? cv.state + (size_t)cv.slots[b] * R * cols + c : nullptr;
+            float w4[4], carry[4], u[4];
+            load_row_v<4>(cv.w + (size_t)R * cols + c, w4);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { carry[i] = v[i]; v[i] *= w4[i]; }
+            if (R > 0 && R <= 3) {             // (the rows are asked for together)
+                float uu[3][4], ww[3][4];
+#pragma unroll
+                for (int k = 0; k < 3; ++k) {
+                    const int j = R - 1 - k, s = t - 1 - k;
+                    if (k < R) {
+                        if (s >= start) load_elems4(qkv + (size_t)s * ld + c, uu[k]);
+                        else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, uu[k]);
+                        load_row_v<4>(cv.w + (size_t)j * cols + c, ww[k]);
+                    }
+                }
+#pragma unroll
+                for (int k = 0; k < 3; ++k)
+                    if (k < R) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) v[i] = fmaf(ww[k][i], uu[k][i], v[i]);
+                        if (cv.one_each) {
+                            store_row_v<float, 4>(st + (size_t)(R - 1 - k) * cols, carry);
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) carry[i] = uu[k][i];
+                        }
+                    }
+            } else for (int j = R - 1; j >= 0; --j) {
+                const int s = t - R + j;
+                if (s >= start) load_elems4(qkv + (size_t)s * ld + c, u);
+                else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, u);
+                load_row_v<4>(cv.w + (size_t)j * cols + c, w4);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[i] = fmaf(w4[i], u[i], v[i]);
+                if (cv.one_each) {
+                    store_row_v<float, 4>(st + (size_t)j * cols, carry);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) carry[i] = u[i];
+                }
+            }
+        }
+    }
+    if (!is_v) {
+        float f = is_q ? qkv_temperature(pos, coef, every) : 1.f;
+        if (norm_mode) {
+            const float ss = warp_sum(v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3]);
+            f /= sqrtf(ss / (float)d + eps);
+            const float* w = is_q ? qw : kw;
+            if (w != nullptr && on) {
+                float w4[4];
+                load_row_v<4>(w + e, w4);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[i] *= w4[i];
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] *= f;
+        if (rot) {
+            const int half = rot >> 1;
+            if (on) store_row_v<float, 4>(&rows[warp][e], v);
+            __syncwarp();
+            if (e < rot) {
+                const float* cs = cosv + (size_t)t * half;
+                const float* sn = sinv + (size_t)t * half;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int k = e + i;
+                    if (k < half) v[i] = v[i] * cs[k] - rows[warp][k + half] * sn[k];
+                    else if (k < rot) v[i] = rows[warp][k - half] * sn[k - half] + v[i] * cs[k - half];
+                }
+            }
+        }
+    }
+    if (!on) return;
+    if (is_q) { store_row_v<T, 4>(qd, v); return; }
+    if (k_pool == nullptr) return;
+    const int page = gg_page_w(page_table + (size_t)b * max_pages, pos / page_size, max_pages, pb, 46);
+    if (page < 0) return;
+    const size_t slot_row = ((size_t)page * nkv + (is_v ? head - nq - nkv : head - nq)) * page_size + pos % page_size;
+    store_row_v<T, 4>((is_v ? v_pool : k_pool) + slot_row * n + e, v);
 }
 
 template <typename T>
@@ -589,7 +755,7 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(
     const int pos = positions[t];
     const int start = cv.taps ? cv.cu_seqlens[b] : 0;
     float* st = cv.taps > 1 ? cv.state + (size_t)cv.slots[b] * (cv.taps - 1) * row : nullptr;
-    if (threadIdx.x == 0) q_factor = coef != 0.f ? 1.f + coef * (float)log(floor(((double)pos + 1.0) / every) + 1.0) : 1.f;
+    if (threadIdx.x == 0) q_factor = qkv_temperature(pos, coef, every);
     const bool write_kv = k_pool != nullptr;
     for (int i = threadIdx.x; i < nqk; i += blockDim.x) buf[i] = qkv_column<T>(qkv, ld, t, start, st, row, i, cv);
     __syncthreads();
@@ -670,12 +836,22 @@ GG_API gg_qkv_prep(const void* qkv, int dtype, long long ld, void* q_out, const 
     const size_t smem = ((size_t)(nq + nkv) * d + nq + nkv + 33) * sizeof(float);
     if (smem > 200 * 1024) return GG_ERR_ARG;
     const QkvConv cv = {conv_w, conv_state, cu_seqlens, slots, conv_w != nullptr ? taps : 0, max_new == 1 ? 1 : 0};
+    const bool heads = norm_mode != 2 && d % 4 == 0 && dv % 4 == 0 && d <= 128 && dv <= 128 && ld % 4 == 0 &&
+                       (((uintptr_t)qkv) & (dtype == GG_BF16 ? 7 : 15)) == 0 &&
+                       (((uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)qw | (uintptr_t)kw | (uintptr_t)conv_w |
+                         (uintptr_t)conv_state) & 15) == 0;
     GG_DISPATCH_DTYPE(dtype, T,
+        if (heads) {
+            gg_launch(qkv_prep_head_kernel<T>, dim3(ntok, (nq + 2 * nkv + 7) / 8), dim3(256), 0, stream, 1, (const T*)qkv, ld, (T*)q_out, qw,
+                      kw, eps, norm_mode, cosv, sinv, positions, seq_of_token, page_table, max_pages, page_size, (T*)k_pool, (T*)v_pool, nq,
+                      nkv, d, dv, rot, cv, coef, (double)every, PageBounds{n_pages, status});
+        } else {
         if (smem > 47 * 1024)
             cudaFuncSetAttribute(qkv_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         gg_launch(qkv_prep_kernel<T>, dim3(ntok), dim3(256), smem, stream, 1,
             (const T*)qkv, ld, (T*)q_out, qw, kw, eps, norm_mode, cosv, sinv, positions, seq_of_token, page_table, max_pages,
             page_size, (T*)k_pool, (T*)v_pool, nq, nkv, d, dv, rot, cv, coef, (double)every, PageBounds{n_pages, status});
+        }
         if (cv.taps > 1 && !cv.one_each)
             gg_launch(column_conv_state_kernel<T>, dim3(n_seqs, (row + 255) / 256), dim3(256), 0, stream, 1, (const T*)qkv, ld,
                       (const float*)nullptr, conv_state, cu_seqlens, slots, seq_of_token, row, taps));
@@ -1592,7 +1768,8 @@ __global__ void __launch_bounds__(256) column_conv_state_kernel(const T* h, long
 // The same for up to eight taps, a thread walking TT consecutive rows of one channel with the window of earlier values
 // in registers, so that a row of h is read once instead of once per tap; the window is filled again (from the
 // step's rows or the sequence's state) where a new sequence starts among the rows.  Blocks (TT rows, 256 channels).
-template <typename T, typename TO, int TAPS, int TT>
+// V = 4: four neighbouring channels a thread (8- or 16-byte accesses).
+template <typename T, typename TO, int TAPS, int TT, int V>
 __global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long long ldh, TO* out, long long ldo,
                                                                const float* __restrict__ w, const float* __restrict__ bias,
                                                                const float* __restrict__ in_bias, float* state,
@@ -1603,42 +1780,67 @@ __global__ void __launch_bounds__(256) column_conv_tile_kernel(const T* h, long 
     pdl_launch();
     pdl_wait();
     constexpr int R = TAPS - 1;
-    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    const int c = V * (blockIdx.y * blockDim.x + threadIdx.x);
     if (c >= C) return;
-    float wr[TAPS];
+    float wr[TAPS][V], ob[V], ib[V], win[R > 0 ? R : 1][V];
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) wr[j] = w[(size_t)j * C + c];
-    const float ob = bias != nullptr ? bias[c] : 0.f, ib = in_bias != nullptr ? in_bias[c] : 0.f;
-    float win[R > 0 ? R : 1];
+    for (int k = 0; k < V; ++k) { ob[k] = 0.f; ib[k] = 0.f; }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_row_v<V>(w + (size_t)j * C + c, wr[j]);
+    if (bias != nullptr) load_row_v<V>(bias + c, ob);
+    if (in_bias != nullptr) load_row_v<V>(in_bias + c, ib);
+    auto row = [&](int s, float* v) {
+        if (V == 4) load_elems4(h + (size_t)s * ldh + c, v);
+        else v[0] = to_f<T>(h[(size_t)s * ldh + c]);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] += ib[k];
+    };
     const int t0 = blockIdx.x * TT;
     int prev_b = -2;
+    // the rows and whose they are are asked for together
+    float fetched[TT][V];
+    int whose[TT];
+#pragma unroll
+    for (int tt = 0; tt < TT; ++tt) {
+        const int t = min(t0 + tt, ntok - 1);
+        whose[tt] = seq_of_token[t];
+        row(t, fetched[tt]);
+    }
 #pragma unroll
     for (int tt = 0; tt < TT; ++tt) {
         const int t = t0 + tt;
         if (t >= ntok) break;
-        const int b = seq_of_token[t];
-        if (b < 0) { out[(size_t)t * ldo + c] = from_f<TO>(0.f); prev_b = -2; continue; }
+        const int b = whose[tt];
+        float acc[V];
+        const float* cur = fetched[tt];
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc[k] = 0.f;
+        if (b < 0) { store_row_v<TO, V>(out + (size_t)t * ldo + c, acc); prev_b = -2; continue; }
         float* st = state + (size_t)slots[b] * R * C + c;
         if (b != prev_b) {
             const int start = cu_seqlens[b];
 #pragma unroll
             for (int j = 0; j < R; ++j) {
                 const int s = t - R + j;
-                win[j] = s >= start ? to_f<T>(h[(size_t)s * ldh + c]) + ib : st[(size_t)(R + (s - start)) * C];
+                if (s >= start) row(s, win[j]);
+                else load_row_v<V>(st + (size_t)(R + (s - start)) * C, win[j]);
             }
             prev_b = b;
         }
-        const float cur = to_f<T>(h[(size_t)t * ldh + c]) + ib;
-        float acc = fmaf(wr[R], cur, ob);
 #pragma unroll
-        for (int j = 0; j < R; ++j) acc = fmaf(wr[j], win[j], acc);
-        out[(size_t)t * ldo + c] = from_f<TO>(act == 1 ? acc / (1.0f + expf(-acc)) : acc);
+        for (int k = 0; k < V; ++k) {
+            acc[k] = fmaf(wr[R][k], cur[k], ob[k]);
 #pragma unroll
-        for (int j = 0; j + 1 < R; ++j) win[j] = win[j + 1];
-        if (R > 0) win[R - 1] = cur;
+            for (int j = 0; j < R; ++j) acc[k] = fmaf(wr[j][k], win[j][k], acc[k]);
+            if (act == 1) acc[k] = acc[k] / (1.0f + expf(-acc[k]));
+#pragma unroll
+            for (int j = 0; j + 1 < R; ++j) win[j][k] = win[j + 1][k];
+            if (R > 0) win[R - 1][k] = cur[k];
+        }
+        store_row_v<TO, V>(out + (size_t)t * ldo + c, acc);
         if (one_each) {                                   // the sequence's only row of the step: its state moves on
 #pragma unroll
-            for (int j = 0; j < R; ++j) st[(size_t)j * C] = win[j];
+            for (int j = 0; j < R; ++j) store_row_v<float, V>(st + (size_t)j * C, win[j]);
         }
     }
 }
@@ -1647,12 +1849,23 @@ template <typename T, typename TO, int TAPS>
 static int column_conv_tile_launch(const T* h, long long ldh, TO* out, long long ldo, const float* w, const float* bias,
                                    const float* in_bias, float* state, const int* cu_seqlens, const int* slots,
                                    const int* seq_of_token, int ntok, int C, int act, int one_each, cudaStream_t stream) {
-    const unsigned cb = (unsigned)((C + 255) / 256);
-    if (ntok < 1024 || one_each)       // few rows, or a row a sequence: a row a thread, so that the step fills more of the GPU
-        return gg_launch(column_conv_tile_kernel<T, TO, TAPS, 1>, dim3((unsigned)ntok, cb), dim3(256), 0, stream, 1, h, ldh, out, ldo,
-                         w, bias, in_bias, state, cu_seqlens, slots, seq_of_token, C, ntok, act, one_each);
-    return gg_launch(column_conv_tile_kernel<T, TO, TAPS, 8>, dim3((unsigned)((ntok + 7) / 8), cb), dim3(256), 0, stream, 1, h, ldh,
-                     out, ldo, w, bias, in_bias, state, cu_seqlens, slots, seq_of_token, C, ntok, act, one_each);
+    const bool vec = TAPS <= 4 && C % 4 == 0 && ldh % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)h) & (4 * sizeof(T) - 1)) == 0 &&
+                     (((uintptr_t)out) & (4 * sizeof(TO) - 1)) == 0 &&
+                     (((uintptr_t)w | (uintptr_t)bias | (uintptr_t)in_bias | (uintptr_t)state) & 15) == 0;
+    // few rows, or a row a sequence: a row a thread, so that the step fills more of the GPU
+    const bool rows1 = ntok < 1024 || one_each;
+    const int V = vec ? 4 : 1;
+    const dim3 grid((unsigned)(rows1 ? ntok : (ntok + 7) / 8), (unsigned)((C + 256 * V - 1) / (256 * V)));
+#define CC_GO(TT_, V_)                                                                                                     \
+    return gg_launch(column_conv_tile_kernel<T, TO, TAPS, TT_, V_>, grid, dim3(256), 0, stream, 1, h, ldh, out, ldo, w, bias,   \
+                     in_bias, state, cu_seqlens, slots, seq_of_token, C, ntok, act, one_each)
+    if constexpr (TAPS <= 4) {
+        if (vec && rows1) CC_GO(1, 4);
+        if (vec) CC_GO(8, 4);
+    }
+    if (rows1) CC_GO(1, 1);
+    CC_GO(8, 1);
+#undef CC_GO
 }
 
 template <typename T, typename TO>

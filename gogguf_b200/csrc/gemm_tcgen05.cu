@@ -106,9 +106,16 @@ struct NormIO {
     int glu_act;             // the gated unit's activation (SwiGLU mode): 0 silu, 1 gelu in its tanh form
 };
 
+// tanh(x) in float32: 1 - 2 / (e^2x + 1), its Taylor polynomial where that would cancel (|x| < 1/8: an error below 3e-8)
+__device__ __forceinline__ float emit_tanh(float x) {
+    const float x2 = x * x;
+    const float small = x * fmaf(x2, fmaf(x2, fmaf(x2, -0.053968254f, 0.13333333f), -0.33333333f), 1.0f);
+    const float large = 1.0f - __fdividef(2.0f, __expf(2.0f * x) + 1.0f);
+    return fabsf(x) < 0.125f ? small : large;
+}
 // What goes to out_xhat for an updated residual value v of column c.
 __device__ __forceinline__ float emit_value(const NormIO& nio, float v, int c) {
-    return nio.t_w != nullptr ? fmaf(tanhf(nio.t_alpha * v), __ldg(nio.t_w + c), __ldg(nio.t_b + c)) : v;
+    return nio.t_w != nullptr ? fmaf(emit_tanh(nio.t_alpha * v), __ldg(nio.t_w + c), __ldg(nio.t_b + c)) : v;
 }
 
 // Bias values of `n` consecutive columns from c0 on (columns at or beyond N get 0), added to v.

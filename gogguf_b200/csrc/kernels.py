@@ -106,8 +106,8 @@ NORMED_MAX = 4                # parts that `normed_sum` takes (csrc/elementwise.
 
 
 def normed_sum(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps, out: Optional[torch.Tensor] = None,
-               norm=None) -> None:
-    """x[r] += sum_k y[k, r] / sqrt(mean(y[k, r]^2) + eps[k]) * weight[k], all float32 (y [parts, rows, H], left zeroed).
+               norm=None, zero_y: bool = False) -> None:
+    """x[r] += sum_k y[k, r] / sqrt(mean(y[k, r]^2) + eps[k]) * weight[k], all float32 (y [parts, rows, H]; zero_y: left zeroed).
     norm (alpha, weight, bias): the updated rows' dynamic tanh goes to `out` as well."""
     _need(x, torch.float32, "x")
     _need(y, torch.float32, "y")
@@ -124,7 +124,7 @@ def normed_sum(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps, out:
     e = list(eps) + [1.0] * (NORMED_MAX - parts)
     kernel("elementwise", "gg_normed_sum")(_p(x), _p(y), _p(weight), parts, x.numel() // H, H, x.numel(), *(float(v) for v in e),
                                             _p(out), dtype_code(out.dtype) if out is not None else F32, float(alpha), _p(nw), _p(nb),
-                                            _stream())
+                                            int(zero_y), _stream())
 
 
 def rope_tables(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor,
@@ -964,11 +964,12 @@ def selective_scan_scratch(n_tokens: int, n_seqs: int, inner: int, N: int, chunk
 def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, xdt: torch.Tensor,
                    out: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
                    seq_of_token: torch.Tensor, a: torch.Tensor, skip: torch.Tensor, n_tokens: int, n_seqs: int, chunk: int = 0,
-                   scratch: Optional[torch.Tensor] = None) -> None:
+                   scratch: Optional[torch.Tensor] = None, max_new: int = 0) -> None:
     """dt = softplus(xdt); S[c, n] <- exp(dt a[c, n]) S[c, n] + dt x_c B_n; out_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c)
     per channel, from and into state [slots, inner, N] (float32).  x, z [T, inner] and B, C (columns b_off and c_off of bc)
     in the dtype of out, xdt [T, inner] float32 (all may be column ranges of wider rows); a [inner, N], skip [inner]
-    float32.  chunk > 0: in chunks of that many rows (prompts with few channels)."""
+    float32.  chunk > 0: in chunks of that many rows (prompts).  max_new: the most tokens one sequence brings, where the
+    caller knows it (1: the form for a token each)."""
     inner, N = a.shape
     for t, n in ((xdt, "xdt"), (state, "state"), (a, "a"), (skip, "skip")):
         if t.dtype != torch.float32:
@@ -988,7 +989,7 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, b_off: in
     kernel("selective_scan", "gg_selective_scan")(
         _p(x), x.stride(0), _p(z), z.stride(0), _p(bc), bc.stride(0), int(b_off), int(c_off), _p(xdt), xdt.stride(0), _p(out),
         dtype_code(out.dtype), _p(state), _p(cu_seqlens), _p(slots), _p(seq_of_token), _p(a), _p(skip), int(n_tokens), int(n_seqs),
-        inner, N, int(chunk), _p(scratch), _stream())
+        inner, N, int(chunk), int(max_new), _p(scratch), _stream())
 
 
 # ------------------------------------------------------------------------------- matrix memory

@@ -618,17 +618,17 @@ def niresun(sizes=((2048, 4096, 16, 16, 8, 8), (4096, 8192, 16, 32, 8, 16))) -> 
         out = torch.empty(T, C, device=dev, dtype=bf)
         cw, cb, tail = torch.randn(4, C, device=dev), torch.randn(C, device=dev), torch.zeros(64, 3, C, device=dev)
         state = torch.zeros(64, C, N, device=dev)
-        for chunk in (0, 64):
+        for chunk in (0, 32, 64, 128, 256, 512):
             scr = torch.empty(K.selective_scan_scratch(T, 1, C, N, chunk), device=dev) if chunk else None
             us = _time_graph(lambda i: K.selective_scan(x, xz[:, C:], bc, 128, 128 + N, xdt, out, state, cu1, slot1, sot1, A, D, T, 1,
                                                         chunk=chunk, scratch=scr), 10)
-            say(f"selective scan, prompt, {C} x {N}, T={T}" + (", in chunks" if chunk else ""), us, T * C * 10)
+            say(f"selective scan, prompt, {C} x {N}, T={T}" + (f", in chunks of {chunk}" if chunk else ""), us, T * C * 10)
         us = _time_graph(lambda i: K.column_conv(xz[:, :C], x, cw, cb, None, tail, cu1, slot1, sot1, T, 1, act=1, max_new=T), 10)
         say(f"convolution of projection columns, T={T}", us, T * C * 4)
         for B in (8, 64):
             cu, sot, sl = ints(list(range(B + 1))), ints(list(range(B))), ints(list(range(B)))
             us = _time_graph(lambda i: K.selective_scan(x[:B], xz[:B, C:], bc[:B], 128, 128 + N, xdt[:B], out[:B], state, cu, sl, sot, A, D,
-                                                        B, B))
+                                                        B, B, max_new=1))
             say(f"selective scan, decode, batch {B}", us, B * C * (2 * N * 4 + 10) + C * N * 4)
             us = _time_graph(lambda i: K.column_conv(xz[:B, :C], x[:B], cw, cb, None, tail, cu, sl, sot, B, B, act=1, max_new=1))
             say(f"convolution of projection columns, batch {B}", us, B * C * (4 + 6 * 4))

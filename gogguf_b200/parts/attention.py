@@ -42,6 +42,8 @@ MAX_HEAD_DIM = 256
 
 @register_mixer("attention")
 class AttentionMixer:
+    overwrites = True           # stores its output instead of adding it where ctx.shared["output_empty"] is set
+
     @classmethod
     def _names(cls, spec: PartSpec) -> Dict[str, str]:
         n = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight",
@@ -229,4 +231,4 @@ class AttentionMixer:
             K.attention_plain(q, cache.k, cache.v, o, ctx.positions, ctx.seq_of_token, table,
                               cache.page_size, T, nq, nkv, d, self.scale, self.window, dv=dv, sink=self.sink,
                               out_scale=self.out_scale, chunk=self.chunk, gate=gate)
-        self.o(o, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
+        self.o(o, residual, accumulate=not ctx.shared.get("output_empty", False), ws=ctx.ws, emit=ctx.shared.get("row_stats"))

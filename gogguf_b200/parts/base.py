@@ -196,7 +196,9 @@ class Linear:
         elif isinstance(x, RowStats):
             raise TypeError("Linear: RowStats given to a projection without a folded norm")
         if isinstance(emit, NormedRows):
-            if (emit.norm is not None and accumulate and self._fast is not None and x.dtype == torch.bfloat16
+            # (measured: in products of more rows the norm's arithmetic lengthens the epilogue by more than a norm kernel takes)
+            rows = x.shape[0] if m is None else m
+            if (emit.norm is not None and rows <= 128 and accumulate and self._fast is not None and x.dtype == torch.bfloat16
                     and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and out.is_contiguous()
                     and out.shape[-1] == emit.rows.shape[-1] and x.data_ptr() != emit.rows.data_ptr()):
                 kw.update(out_xhat=emit.rows, out_norm=emit.norm.emit)

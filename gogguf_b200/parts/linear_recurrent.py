@@ -281,17 +281,17 @@ class Mamba1Mixer:
         if chunk:
             scratch = ctx.ws.get("mamba1_chunk_states", (K.selective_scan_scratch(T, ctx.n_seqs, C, N, chunk),), torch.float32)
         K.selective_scan(x, p[:, C:], low, self.R, self.R + N, step, y, st.state, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
-                         self.a, self.skip, T, ctx.n_seqs, chunk=chunk, scratch=scratch)
+                         self.a, self.skip, T, ctx.n_seqs, chunk=chunk, scratch=scratch, max_new=int(ctx.max_new))
         self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
 
 
 def selective_chunk(max_new: int, n_seqs: int, channels: int, states: int) -> int:
     """Rows per chunk of a selective scan (0: every sequence walked whole).  The chunked form computes every row's decays
-    twice, so it pays only where the channels alone leave most of the GPU idle and the prompts are long."""
+    twice, so it pays where the channels alone leave the multiprocessors few warps and the prompts are long."""
     lanes = 1
     while 4 * lanes < states and lanes < 32:
         lanes *= 2
     warps = n_seqs * channels * lanes // 32
-    if max_new < CHUNKED_FROM or warps * 3 >= 148 * 4:
+    if max_new < CHUNKED_FROM or warps >= 148 * 16:
         return 0
-    return 64
+    return 128 if max_new >= 1024 else 64

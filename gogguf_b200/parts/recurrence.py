@@ -219,6 +219,8 @@ class MatrixMemoryMixer:
 
     Spec parameters: hidden_size, num_heads, head_dim, value_dim, gate_cap, eps, names."""
 
+    overwrites = True           # stores its output instead of adding it where ctx.shared["output_empty"] is set
+
     @classmethod
     def _names(cls, spec: PartSpec) -> Dict[str, str]:
         n = dict(q="q", k="k", v="v", g="g", i="i", i_bias="i.b", f="f", f_bias="f.b", norm="norm", o="o")
@@ -288,8 +290,7 @@ class MatrixMemoryMixer:
             scratch = ctx.ws.get("mlstm_chunk_states", (K.memory_chunks_scratch(T, ctx.n_seqs, H, d, dv),), torch.float32)
             K.memory_chunks(row, self.off, gates[:, :H], gates[:, H:2 * H], y, scratch, states, ctx.cu_seqlens, ctx.slots,
                             ctx.seq_of_token, self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
-            self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
-            return
-        K.memory_scan(row, self.off, gates[:, :H], gates[:, H:2 * H], y, states, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
-                      self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
-        self.o(y, residual, accumulate=True, ws=ctx.ws, emit=ctx.shared.get("row_stats"))
+        else:
+            K.memory_scan(row, self.off, gates[:, :H], gates[:, H:2 * H], y, states, ctx.cu_seqlens, ctx.slots, ctx.seq_of_token,
+                          self.norm_weight, T, ctx.n_seqs, H, d, dv, d ** -0.5, self.cap, self.eps)
+        self.o(y, residual, accumulate=not ctx.shared.get("output_empty", False), ws=ctx.ws, emit=ctx.shared.get("row_stats"))

@@ -6,8 +6,9 @@ member's output, default 1) and `out_norm` {tensor, size, eps} (optional: the me
 square over the row and multiplied by that stored vector, named under the member's prefix, before it is added).  Each member keeps a cache or state of its own: the part's cache request is the tuple
 of its members' requests and it is handed the tuple of their views.  A member that takes its factor into its own
 last step (`scale_output(w) -> bool`) adds straight into the output; any other member writes into a zeroed buffer
-that is added with its factor.  Members with a norm write into zeroed buffers side by side; one kernel norms, weighs and
-adds them, and leaves the rows behind the block's next norm where that works element by element (`NormedRows`).
+that is added with its factor.  Members with a norm write into buffers side by side, zeroed unless the member says
+(`overwrites`) that it stores its output where ctx.shared["output_empty"] is set; one kernel norms, weighs and adds
+them, and leaves the rows behind the block's next norm where that works element by element (`NormedRows`).
 """
 from __future__ import annotations
 
@@ -72,6 +73,8 @@ class SideBySideMixer:
             self.members.append((part, w, direct))
         if len(weights_n) > K.NORMED_MAX:
             raise ValueError(f"side_by_side: at most {K.NORMED_MAX} members have a norm")
+        # do all members with a norm store their outputs, so that nobody has to clear the buffers?
+        self.overwrites = all(getattr(p, "overwrites", False) for p, _, direct in self.members if direct is None)
         self.norm_weight = torch.stack(weights_n).contiguous() if weights_n else None
 
     def absorb_norm(self, norm) -> bool:
@@ -100,12 +103,15 @@ class SideBySideMixer:
         parts_out = None
         if self.norm_weight is not None:
             parts_out = ctx.ws.get("side_by_side_normed", (len(self.norm_eps),) + tuple(residual.shape), torch.float32)
-            if ctx.shared.get(self.ZEROED) != (parts_out.data_ptr(), parts_out.numel()):
+            if not self.overwrites and ctx.shared.get(self.ZEROED) != (parts_out.data_ptr(), parts_out.numel()):
                 parts_out.zero_()
         k = 0
         for (part, w, direct), view in zip(self.members, cache):
             if direct is None:
+                if self.overwrites:
+                    ctx.shared["output_empty"] = True
                 part.forward(h, parts_out[k], ctx, view, writes_cache)
+                ctx.shared.pop("output_empty", None)
                 k += 1
                 continue
             if direct:
@@ -120,7 +126,10 @@ class SideBySideMixer:
         if parts_out is not None:
             emit = isinstance(ahead, NormedRows) and ahead.norm is not None and ahead.rows.shape == residual.shape
             K.normed_sum(residual, parts_out, self.norm_weight, self.norm_eps, ahead.rows if emit else None,
-                         ahead.norm.emit if emit else None)
+                         ahead.norm.emit if emit else None, zero_y=not self.overwrites)
             if emit:
                 ahead.fresh = True
-            ctx.shared[self.ZEROED] = (parts_out.data_ptr(), parts_out.numel())
+            if self.overwrites:
+                ctx.shared.pop(self.ZEROED, None)
+            else:
+                ctx.shared[self.ZEROED] = (parts_out.data_ptr(), parts_out.numel())

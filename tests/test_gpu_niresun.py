@@ -65,6 +65,7 @@ def test_dynamic_tanh(T, H):
 def test_a_product_leaves_the_rows_behind_the_next_norm(N, K_):
     """Every form of the product (decode with and without a K split, prompts with and without one, few columns): it adds
     into the residual and leaves the dynamic tanh of the updated rows."""
+    from gogguf_b200.csrc import tcgen05_gemm as TG
     from gogguf_b200.parts.base import Linear, NormedRows, Runtime, Workspace
     g = _gen(N + K_)
     w = (torch.randn(N, K_, generator=g) * 0.1).to(torch.bfloat16)
@@ -84,7 +85,12 @@ def test_a_product_leaves_the_rows_behind_the_next_norm(N, K_):
         assert not ahead.fresh and float((ahead.rows - 7.0).abs().max()) == 0.0       # nobody's turn: nothing is written
         acc, ahead.norm = res.to(DEV), Norm
         lin(x.to(DEV), acc, accumulate=True, ws=ws, emit=ahead)
-        assert ahead.fresh and rel_err(acc, want) < 3e-5, m
+        assert ahead.fresh == (m <= 128) and rel_err(acc, want) < 3e-5, m
+        if m > 128:                                  # the product can, a norm kernel is faster
+            acc = res.to(DEV)
+            scratch = torch.empty(max(1, TG.pair_scratch_elems(m, N, K_)), device=DEV)
+            TG.gemm_tc_norm(x.to(DEV), w.to(DEV), acc, accumulate=True, out_xhat=ahead.rows, out_norm=Norm.emit, scratch=scratch)
+            assert rel_err(acc, want) < 3e-5, m
         assert rel_err(ahead.rows, torch.tanh(0.6 * want) * nw.double().cpu() + nb.double().cpu()) < 5e-3, m
     _check_status()
 
@@ -117,7 +123,8 @@ def test_gelu_gated_unit(I, W):
             assert rel_err(out, want) < (3e-6 if dt == torch.float32 else 1e-2), (dt, fast, T)
 
 
-@pytest.mark.parametrize("P,T,H", [(2, 5, 64), (1, 3, 77), (3, 130, 320), (4, 2, 2052)])
+@pytest.mark.parametrize("P,T,H", [(2, 5, 64), (1, 3, 77), (3, 130, 320), (4, 2, 2052), (2, 9, 2048), (2, 3, 4096), (1, 2, 1500),
+                                   (2, 2, 4104), (2, 3, 50)])
 def test_sum_of_normed_parts(P, T, H):
     K = _K()
     g = _gen(P * H)
@@ -129,8 +136,9 @@ def test_sum_of_normed_parts(P, T, H):
     for dt in (None, torch.float32, torch.bfloat16):
         xd, yd = x.to(DEV), y.to(DEV)
         out = None if dt is None else torch.empty(T, H, dtype=dt, device=DEV)
-        K.normed_sum(xd, yd, w.to(DEV), eps, out, None if dt is None else (0.4, nw.to(DEV), nb.to(DEV)))
-        assert rel_err(xd, want) < 2e-6 and float(yd.abs().max()) == 0.0
+        zero = dt != torch.bfloat16
+        K.normed_sum(xd, yd, w.to(DEV), eps, out, None if dt is None else (0.4, nw.to(DEV), nb.to(DEV)), zero_y=zero)
+        assert rel_err(xd, want) < 2e-6 and (float(yd.abs().max()) == 0.0 if zero else torch.equal(yd.cpu(), y))
         if dt is not None:
             assert rel_err(out, torch.tanh(0.4 * want) * nw.double() + nb.double()) < (2e-6 if dt == torch.float32 else 5e-3)
 
@@ -325,7 +333,7 @@ def test_selective_scan(dt, C, N):
                 out = torch.full((T, C), 9.0, dtype=dt, device=DEV)
                 scratch = torch.full((K.selective_scan_scratch(T, 2, C, N, chunk),), 1e30, device=DEV) if chunk else None
                 K.selective_scan(xz[:, :C], xz[:, C:], bc, off, off + N, part("dt").to(DEV), out, state, cu, _i32(slots), sot, A.to(DEV),
-                                 skip.to(DEV), T, 2, chunk=chunk, scratch=scratch)
+                                 skip.to(DEV), T, 2, chunk=chunk, scratch=scratch, max_new=max(new))
                 ref = torch.cat([w[a:a + n] for w, a, n in zip(want, at, new)])
                 assert rel_err(out, ref) < tol, (new, chunk, rel_err(out, ref))
                 at = [a + n for a, n in zip(at, new)]
@@ -337,6 +345,13 @@ def test_selective_scan(dt, C, N):
     K.selective_scan(xz[:2, :C], xz[:2, C:], bc[:2], off, off + N, D[0]["dt"][:2].to(DEV), out, state, cu, _i32([3, 0]), sot,
                      A.to(DEV), skip.to(DEV), 2, 2)
     assert float(out[1].abs().max()) == 0.0 and torch.equal(state[[0, 1, 2]], before[[0, 1, 2]]) and not torch.equal(state[3], before[3])
+    after, out1 = state.clone(), out.clone()                       # the form for a token each
+    state.copy_(before)
+    out.fill_(9.0)
+    K.selective_scan(xz[:2, :C], xz[:2, C:], bc[:2], off, off + N, D[0]["dt"][:2].to(DEV), out, state, cu, _i32([3, 0]), sot,
+                     A.to(DEV), skip.to(DEV), 2, 2, max_new=1)
+    assert rel_err(out, out1.double()) < tol and rel_err(state, after.double()) < 1e-5 and torch.equal(state[[0, 1, 2]], before[[0, 1, 2]])
+    assert float(out[1].abs().max()) == 0.0
 
 
 @pytest.mark.parametrize("H,d,dv,cap,shift", [(3, 10, 14, 6.0, 0.0), (1, 16, 16, 1.0, 0.0), (4, 64, 128, 12.0, 0.0), (2, 128, 128, 15.0, 3.0),

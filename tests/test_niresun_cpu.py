@@ -205,6 +205,6 @@ def test_drawn_configurations_are_valid(seed):
 
 def test_rows_per_chunk_of_a_selective_scan():
     from gogguf_b200.parts.linear_recurrent import selective_chunk
-    assert selective_chunk(2048, 1, 4096, 16) == 0            # enough channels to fill the GPU
-    assert selective_chunk(2048, 1, 256, 16) == 64 and selective_chunk(2048, 64, 256, 16) == 0
+    assert selective_chunk(2048, 1, 4096, 16) == 128 and selective_chunk(2048, 8, 4096, 16) == 0      # enough to fill the GPU
+    assert selective_chunk(200, 1, 256, 16) == 64 and selective_chunk(2048, 64, 256, 24) == 0
     assert selective_chunk(1, 1, 256, 16) == 0 and selective_chunk(100, 1, 256, 16) == 0
