@@ -1142,6 +1142,15 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
             __syncwarp();
             if (lane == 0) tma::mbar_arrive(&p_ready[j & 1]);
         }
+        // the gates of the row's next 32 columns, asked for ahead
+        uint4 gates[4];
+        const bf16* grow = sh.gate != nullptr && row < rows ? sh.gate + (size_t)(tok0 + row0 + row) * sh.ldg + h * dv : nullptr;
+        auto ask = [&](int c0) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (grow != nullptr && c0 + 8 * k < dv) gates[k] = *reinterpret_cast<const uint4*>(grow + c0 + 8 * k);
+        };
+        ask(0);
         // The last P V, on a barrier of its own that completes once: a warp that comes late to a wait by parity could find
         // two phases gone, which looks like none.
         if (ok && tma::mbar_wait(o_done, 0, abort_flag, status, 28)) {
@@ -1154,21 +1163,21 @@ __global__ void __launch_bounds__(192) attn_prefill_tc_kernel(
                 uint32_t orow[32];
                 tc5::ld32(O_t + lane_off + c0, orow);
                 tc5::wait_ld();
+                if (grow != nullptr) {
+#pragma unroll
+                    for (int c = 0; c < 32; c += 2) {
+                        const uint32_t word = c % 8 == 0 ? gates[c / 8].x : c % 8 == 2 ? gates[c / 8].y : c % 8 == 4 ? gates[c / 8].z
+                                                                                                      : gates[c / 8].w;
+                        const float2 gf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&word));
+                        orow[c] = __float_as_uint(__fdividef(__uint_as_float(orow[c]), 1.0f + __expf(-gf.x)));
+                        orow[c + 1] = __float_as_uint(__fdividef(__uint_as_float(orow[c + 1]), 1.0f + __expf(-gf.y)));
+                    }
+                    ask(c0 + 32);
+                }
                 if (row < rows) {
 #pragma unroll
                     for (int c = 0; c < 32; c += 8) {
                         if (!EXACT && c0 + c >= dv) break;
-                        if (sh.gate != nullptr) {
-                            const uint4 gv = *reinterpret_cast<const uint4*>(sh.gate + (size_t)(tok0 + row0 + row) * sh.ldg +
-                                                                             h * dv + c0 + c);
-                            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
-#pragma unroll
-                            for (int e = 0; e < 4; ++e) {
-                                const float2 gf = __bfloat1622float2(g2[e]);
-                                orow[c + 2 * e] = __float_as_uint(__uint_as_float(orow[c + 2 * e]) / (1.0f + __expf(-gf.x)));
-                                orow[c + 2 * e + 1] = __float_as_uint(__uint_as_float(orow[c + 2 * e + 1]) / (1.0f + __expf(-gf.y)));
-                            }
-                        }
                         uint32_t pk[4];
 #pragma unroll
                         for (int e = 0; e < 4; ++e)

@@ -616,117 +616,159 @@ __device__ __forceinline__ float qkv_temperature(int pos, float coef, double eve
     return coef != 0.f ? 1.f + coef * logf((float)floor(((double)pos + 1.0) / every) + 1.f) : 1.f;
 }
 
-// The same with a warp a head (grid: token, groups of eight of the nq + 2 nkv heads) and four neighbouring elements a
-// lane: heads of up to 128 elements, everything a multiple of four, no norm over the whole projection.
-template <typename T>
+// The same with LPH lanes a head (16 where heads have at most 64 elements, else 32), four neighbouring elements a lane, and
+// TT consecutive tokens a thread (grid: groups of TT tokens, groups of 256 / LPH of the nq + 2 nkv heads): heads of up to 128
+// elements, everything a multiple of four, no norm over the whole projection.  The convolution's window stays in registers
+// from token to token and is filled again where another sequence starts.
+template <typename T, int LPH, int TT>
 __global__ void __launch_bounds__(256) qkv_prep_head_kernel(
     const T* qkv, long long ld, T* __restrict__ q_out, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
     int norm_mode, const float* cosv, const float* sinv, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
-    const int* __restrict__ page_table, int max_pages, int page_size, T* __restrict__ k_pool, T* __restrict__ v_pool, int nq, int nkv,
-    int d, int dv, int rot, const QkvConv cv, float coef, double every, const PageBounds pb) {
+    const int* __restrict__ page_table, int max_pages, int page_size, T* __restrict__ k_pool, T* __restrict__ v_pool, int ntok, int nq,
+    int nkv, int d, int dv, int rot, const QkvConv cv, float coef, double every, const PageBounds pb) {
     pdl_launch();
     pdl_wait();
-    __shared__ float rows[8][128];
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y * 8 + warp;
-    if (head >= nq + 2 * nkv) return;
+    constexpr int HPB = 256 / LPH;
+    __shared__ __align__(16) float rows[HPB][4 * LPH];
+    const int slot_h = threadIdx.x / LPH, e = 4 * (threadIdx.x % LPH);
+    const int head = blockIdx.y * HPB + slot_h;
+    const bool have = head < nq + 2 * nkv;
     const bool is_q = head < nq, is_v = head >= nq + nkv;
-    const int n = is_v ? dv : d, e = 4 * lane;
-    const bool on = e < n;
-    const int b = seq_of_token[t];
-    T* qd = q_out + ((size_t)t * nq + head) * d + e;
-    float v[4] = {0.f, 0.f, 0.f, 0.f};
-    if (b < 0) {
-        if (is_q && on) store_row_v<T, 4>(qd, v);
-        return;
-    }
-    const int pos = positions[t];
+    const int n = is_v ? dv : d;
+    const bool on = have && e < n;
     const int cols = (nq + nkv) * d + nkv * dv;
     const int c = (is_v ? (nq + nkv) * d + (head - nq - nkv) * dv : head * d) + e;
-    if (on) {
-        load_elems4(qkv + (size_t)t * ld + c, v);
-        if (cv.taps) {
-            const int R = cv.taps - 1, start = cv.cu_seqlens[b];
-            float* st = R ? cv.state + (size_t)cv.slots[b] * R * cols + c : nullptr;
-            float w4[4], carry[4], u[4];
-            load_row_v<4>(cv.w + (size_t)R * cols + c, w4);
+    const int t0 = blockIdx.x * TT, R = cv.taps - 1;
+    const bool window = cv.taps > 0 && R <= 3;
+    // the rows and whose they are are asked for together
+    float fetched[TT][4], win[3][4], wt[4][4];
+    int whose[TT], posn[TT];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { carry[i] = v[i]; v[i] *= w4[i]; }
-            if (R > 0 && R <= 3) {             // (the rows are asked for together)
-                float uu[3][4], ww[3][4];
+    for (int tt = 0; tt < TT; ++tt) {
+        const int t = min(t0 + tt, ntok - 1);
+        whose[tt] = seq_of_token[t];
+        posn[tt] = positions[t];
 #pragma unroll
-                for (int k = 0; k < 3; ++k) {
-                    const int j = R - 1 - k, s = t - 1 - k;
-                    if (k < R) {
-                        if (s >= start) load_elems4(qkv + (size_t)s * ld + c, uu[k]);
-                        else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, uu[k]);
-                        load_row_v<4>(cv.w + (size_t)j * cols + c, ww[k]);
-                    }
-                }
+        for (int i = 0; i < 4; ++i) fetched[tt][i] = 0.f;
+        if (on) load_elems4(qkv + (size_t)t * ld + c, fetched[tt]);
+    }
 #pragma unroll
-                for (int k = 0; k < 3; ++k)
-                    if (k < R) {
+    for (int j = 0; j < 4; ++j) {
 #pragma unroll
-                        for (int i = 0; i < 4; ++i) v[i] = fmaf(ww[k][i], uu[k][i], v[i]);
-                        if (cv.one_each) {
-                            store_row_v<float, 4>(st + (size_t)(R - 1 - k) * cols, carry);
+        for (int i = 0; i < 4; ++i) wt[j][i] = 0.f;
+        if (window && on && j < cv.taps) load_row_v<4>(cv.w + (size_t)(R - j) * cols + c, wt[j]);      // j tokens back
+    }
+    int prev_b = -2;
 #pragma unroll
-                            for (int i = 0; i < 4; ++i) carry[i] = uu[k][i];
+    for (int tt = 0; tt < TT; ++tt) {
+        const int t = t0 + tt;
+        if (t >= ntok) break;
+        const int b = whose[tt];
+        T* qd = q_out + ((size_t)t * nq + head) * d + e;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (b < 0) {                         // padding row: nothing reads its q, the caches are not touched
+            if (is_q && on) store_row_v<T, 4>(qd, v);
+            prev_b = -2;
+            continue;
+        }
+        const int pos = posn[tt];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] = fetched[tt][i];
+        if (cv.taps && on) {
+            const int start = cv.cu_seqlens[b];
+            float* st = R > 0 ? cv.state + (size_t)cv.slots[b] * R * cols + c : nullptr;
+            if (window) {
+                if (b != prev_b) {
+#pragma unroll
+                    for (int k = 0; k < 3; ++k) {              // win[k]: the row k + 1 tokens back
+                        const int s = t - 1 - k;
+                        if (k < R) {
+                            if (s >= start) load_elems4(qkv + (size_t)s * ld + c, win[k]);
+                            else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, win[k]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) win[k][i] = 0.f;
                         }
                     }
-            } else for (int j = R - 1; j >= 0; --j) {
-                const int s = t - R + j;
-                if (s >= start) load_elems4(qkv + (size_t)s * ld + c, u);
-                else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, u);
-                load_row_v<4>(cv.w + (size_t)j * cols + c, w4);
+                    prev_b = b;
+                }
+                float cur[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) v[i] = fmaf(w4[i], u[i], v[i]);
+                for (int i = 0; i < 4; ++i) {
+                    cur[i] = v[i];
+                    v[i] = fmaf(wt[3][i], win[2][i], fmaf(wt[2][i], win[1][i], fmaf(wt[1][i], win[0][i], wt[0][i] * cur[i])));
+                    win[2][i] = win[1][i]; win[1][i] = win[0][i]; win[0][i] = cur[i];
+                }
                 if (cv.one_each) {
-                    store_row_v<float, 4>(st + (size_t)j * cols, carry);
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) carry[i] = u[i];
+                    for (int k = 0; k < 3; ++k)
+                        if (k < R) store_row_v<float, 4>(st + (size_t)(R - 1 - k) * cols, win[k]);
+                }
+            } else {
+                float w4[4], carry[4], u[4];
+                load_row_v<4>(cv.w + (size_t)R * cols + c, w4);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) { carry[i] = v[i]; v[i] *= w4[i]; }
+                for (int j = R - 1; j >= 0; --j) {
+                    const int s = t - R + j;
+                    if (s >= start) load_elems4(qkv + (size_t)s * ld + c, u);
+                    else load_row_v<4>(st + (size_t)(R + (s - start)) * cols, u);
+                    load_row_v<4>(cv.w + (size_t)j * cols + c, w4);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) v[i] = fmaf(w4[i], u[i], v[i]);
+                    if (cv.one_each) {
+                        store_row_v<float, 4>(st + (size_t)j * cols, carry);
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) carry[i] = u[i];
+                    }
                 }
             }
         }
-    }
-    if (!is_v) {
-        float f = is_q ? qkv_temperature(pos, coef, every) : 1.f;
-        if (norm_mode) {
-            const float ss = warp_sum(v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3]);
-            f /= sqrtf(ss / (float)d + eps);
-            const float* w = is_q ? qw : kw;
-            if (w != nullptr && on) {
-                float w4[4];
-                load_row_v<4>(w + e, w4);
+        // (all lanes of a warp take part in the sums; what a head of values or no head has there is not used)
+        if (norm_mode || coef != 0.f) {
+            float f = is_q ? qkv_temperature(pos, coef, every) : 1.f;
+            if (norm_mode) {
+                float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) v[i] *= w4[i];
+                for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+                f /= sqrtf(ss / (float)d + eps);
+                const float* w = is_q ? qw : kw;
+                if (w != nullptr && on && !is_v) {
+                    float w4[4];
+                    load_row_v<4>(w + e, w4);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) v[i] *= w4[i];
+                }
+            }
+            if (!is_v) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[i] *= f;
             }
         }
-#pragma unroll
-        for (int i = 0; i < 4; ++i) v[i] *= f;
         if (rot) {
             const int half = rot >> 1;
-            if (on) store_row_v<float, 4>(&rows[warp][e], v);
+            __syncwarp();                    // the token before has read its partners
+            if (on && !is_v) store_row_v<float, 4>(&rows[slot_h][e], v);
             __syncwarp();
-            if (e < rot) {
+            if (on && !is_v && e < rot) {
                 const float* cs = cosv + (size_t)t * half;
                 const float* sn = sinv + (size_t)t * half;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const int k = e + i;
-                    if (k < half) v[i] = v[i] * cs[k] - rows[warp][k + half] * sn[k];
-                    else if (k < rot) v[i] = rows[warp][k - half] * sn[k - half] + v[i] * cs[k - half];
+                    if (k < half) v[i] = v[i] * cs[k] - rows[slot_h][k + half] * sn[k];
+                    else if (k < rot) v[i] = rows[slot_h][k - half] * sn[k - half] + v[i] * cs[k - half];
                 }
             }
         }
+        if (!on) continue;
+        if (is_q) { store_row_v<T, 4>(qd, v); continue; }
+        if (k_pool == nullptr) continue;
+        const int page = gg_page_w(page_table + (size_t)b * max_pages, pos / page_size, max_pages, pb, 46);
+        if (page < 0) continue;
+        const size_t slot_row = ((size_t)page * nkv + (is_v ? head - nq - nkv : head - nq)) * page_size + pos % page_size;
+        store_row_v<T, 4>((is_v ? v_pool : k_pool) + slot_row * n + e, v);
     }
-    if (!on) return;
-    if (is_q) { store_row_v<T, 4>(qd, v); return; }
-    if (k_pool == nullptr) return;
-    const int page = gg_page_w(page_table + (size_t)b * max_pages, pos / page_size, max_pages, pb, 46);
-    if (page < 0) return;
-    const size_t slot_row = ((size_t)page * nkv + (is_v ? head - nq - nkv : head - nq)) * page_size + pos % page_size;
-    store_row_v<T, 4>((is_v ? v_pool : k_pool) + slot_row * n + e, v);
 }
 
 template <typename T>
@@ -835,6 +877,10 @@ GG_API gg_qkv_prep(const void* qkv, int dtype, long long ld, void* q_out, const 
         return GG_ERR_ARG;
     const size_t smem = ((size_t)(nq + nkv) * d + nq + nkv + 33) * sizeof(float);
     if (smem > 200 * 1024) return GG_ERR_ARG;
+#define GG_PREP(LPH_, TT_)                                                                                                 \
+    gg_launch(qkv_prep_head_kernel<T, LPH_, TT_>, grid, dim3(256), 0, stream, 1, (const T*)qkv, ld, (T*)q_out, qw, kw, eps, norm_mode,  \
+              cosv, sinv, positions, seq_of_token, page_table, max_pages, page_size, (T*)k_pool, (T*)v_pool, ntok, nq, nkv, d, dv, rot, cv, \
+              coef, (double)every, PageBounds{n_pages, status})
     const QkvConv cv = {conv_w, conv_state, cu_seqlens, slots, conv_w != nullptr ? taps : 0, max_new == 1 ? 1 : 0};
     const bool heads = norm_mode != 2 && d % 4 == 0 && dv % 4 == 0 && d <= 128 && dv <= 128 && ld % 4 == 0 &&
                        (((uintptr_t)qkv) & (dtype == GG_BF16 ? 7 : 15)) == 0 &&
@@ -842,9 +888,12 @@ GG_API gg_qkv_prep(const void* qkv, int dtype, long long ld, void* q_out, const 
                          (uintptr_t)conv_state) & 15) == 0;
     GG_DISPATCH_DTYPE(dtype, T,
         if (heads) {
-            gg_launch(qkv_prep_head_kernel<T>, dim3(ntok, (nq + 2 * nkv + 7) / 8), dim3(256), 0, stream, 1, (const T*)qkv, ld, (T*)q_out, qw,
-                      kw, eps, norm_mode, cosv, sinv, positions, seq_of_token, page_table, max_pages, page_size, (T*)k_pool, (T*)v_pool, nq,
-                      nkv, d, dv, rot, cv, coef, (double)every, PageBounds{n_pages, status});
+            const bool small = d <= 64 && dv <= 64, rows1 = ntok < 512 || cv.taps < 2;      // (several tokens a thread share a window)
+            const dim3 grid(rows1 ? ntok : (ntok + 3) / 4, (nq + 2 * nkv + (small ? 15 : 7)) / (small ? 16 : 8));
+            if (small && rows1) GG_PREP(16, 1);
+            else if (small) GG_PREP(16, 4);
+            else if (rows1) GG_PREP(32, 1);
+            else GG_PREP(32, 4);
         } else {
         if (smem > 47 * 1024)
             cudaFuncSetAttribute(qkv_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -855,6 +904,7 @@ GG_API gg_qkv_prep(const void* qkv, int dtype, long long ld, void* q_out, const 
         if (cv.taps > 1 && !cv.one_each)
             gg_launch(column_conv_state_kernel<T>, dim3(n_seqs, (row + 255) / 256), dim3(256), 0, stream, 1, (const T*)qkv, ld,
                       (const float*)nullptr, conv_state, cu_seqlens, slots, seq_of_token, row, taps));
+#undef GG_PREP
     return gg_last_error();
 }
 

@@ -692,7 +692,7 @@ def niresun(sizes=((2048, 4096, 16, 16, 8, 8), (4096, 8192, 16, 32, 8, 16))) -> 
             yy = torch.randn(2, m, W, device=dev)
             yw = torch.stack([nw, nb])
             us = _time_graph(lambda i: K.normed_sum(xr, yy, yw, [1e-6, 1e-6], h, (0.5, nw, nb)))
-            say(f"sum of two normed parts + dynamic tanh, {m} rows", us, m * W * (4 * 2 + 2 * 8 + 2))
+            say(f"sum of two normed parts + dynamic tanh, {m} rows", us, m * W * (4 * 2 + 2 * 4 + 2))
             a = torch.randn(m, W, device=dev).to(bf)
             wm = (torch.randn(W, W, device=dev) * 0.02).to(bf)
             ssq = torch.empty(m, W // 128, device=dev)

@@ -154,7 +154,8 @@ def test_preparation_of_q_k_and_v(dt, nq, nkv, d, dv, taps, rdims, unit, temp):
     K = _K()
     g = _gen(nq * d + dv)
     cols, eps = (nq + nkv) * d + nkv * dv, 1e-4
-    lens = (150, 7)
+    long = nq in (4, 8)                            # steps of many rows take the form with several tokens a thread
+    lens = (700, 7) if long else (150, 7)
     rows = [torch.randn(n, cols, generator=g).to(dt) for n in lens]
     cw = torch.randn(cols, taps, generator=g) if taps else None
     coef, every = temp or (0.0, 1.0)
@@ -174,12 +175,13 @@ def test_preparation_of_q_k_and_v(dt, nq, nkv, d, dv, taps, rdims, unit, temp):
         want.append((q.reshape(n, -1), k, v.reshape(n, nkv, dv)))
     slots = [2, 0]
     state = torch.zeros(3, max(taps - 1, 1), cols, device=DEV) if taps > 1 else None
-    table = [[4, 1, 6], [3, 5, 0]]
-    kp = torch.full((8, nkv, PS, d), 7.0, dtype=dt, device=DEV)
-    vp = torch.full((8, nkv, PS, dv), 7.0, dtype=dt, device=DEV)
+    order = torch.randperm(24, generator=g).tolist()
+    table = [order[:11], order[11:22]]
+    kp = torch.full((24, nkv, PS, d), 7.0, dtype=dt, device=DEV)
+    vp = torch.full((24, nkv, PS, dv), 7.0, dtype=dt, device=DEV)
     tol = 3e-6 if dt == torch.float32 else 6e-3
     at = [0, 0]
-    for new in ((70, 1), (2, 3), (1, 1), (1, 1), (76, 1)):
+    for new in ((lens[0] - 80, 1), (2, 3), (1, 1), (1, 1), (76, 1)):
         cu, sot = _batch(new)
         T = sum(new)
         pos = [at[b] + i for b, n in enumerate(new) for i in range(n)]
@@ -198,7 +200,7 @@ def test_preparation_of_q_k_and_v(dt, nq, nkv, d, dv, taps, rdims, unit, temp):
         ref = torch.cat([want[b][0][at[b]:at[b] + n] for b, n in enumerate(new)])
         assert rel_err(q_out, ref) < tol, (new, rel_err(q_out, ref))
         at = [a + n for a, n in zip(at, new)]
-    seen = torch.zeros(8, PS, dtype=torch.bool)
+    seen = torch.zeros(24, PS, dtype=torch.bool)
     for b, n in enumerate(lens):
         for p in range(n):
             pg, sl = table[b][p // PS], p % PS
@@ -220,6 +222,39 @@ def test_preparation_of_q_k_and_v(dt, nq, nkv, d, dv, taps, rdims, unit, temp):
                    2, nq, nkv, d, dv, rdims, conv=cw.t().contiguous().to(DEV), conv_state=state, cu_seqlens=cu, slots=_i32([0, 0]),
                    n_seqs=2, max_new=1, coef=coef, every=every)
         assert all(torch.equal(a, b) for a, b in zip(before, (kp, vp, state))) and float(q_out[:2].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("dt,odt", [(torch.float32, torch.float32), (torch.bfloat16, torch.float32), (torch.bfloat16, torch.bfloat16)])
+@pytest.mark.parametrize("C,taps", [(64, 4), (36, 2), (260, 3), (33, 4), (40, 6), (24, 1)])
+def test_convolution_of_columns(dt, odt, C, taps):
+    """Short and long steps (a row, or eight, a thread; one channel or four), sequences that start inside a group of rows,
+    single tokens that move the state on themselves, silu or not, both output types."""
+    K = _K()
+    g = _gen(C + taps)
+    lens, slots = (1090, 3, 40), [1, 3, 0]
+    rows = [torch.randn(n, C, generator=g).to(dt) for n in lens]
+    w, b = torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
+    for act in (0, 1):
+        want = [plain.causal_conv(r.double(), w.double(), b) for r in rows]
+        want = [plain.silu(v) for v in want] if act else want
+        state = torch.zeros(4, taps - 1, C, device=DEV) if taps > 1 else None
+        at = [0, 0, 0]
+        for new in ((1061, 1, 6), (1, 1, 1), (27, 0, 32), (1, 1, 1)):
+            own = [i for i in range(3) if new[i]]
+            cu, sot = _batch([new[i] for i in own])
+            T = sum(new)
+            wide = torch.full((T, C + 16), 3.0, dtype=dt)
+            wide[:, 8:8 + C] = torch.cat([rows[i][at[i]:at[i] + new[i]] for i in own])
+            out = torch.full((T, C), 9.0, dtype=odt, device=DEV)
+            K.column_conv(wide.to(DEV)[:, 8:8 + C], out, w.t().contiguous().to(DEV), b.to(DEV), None, state, cu, _i32([slots[i] for i in own]),
+                          sot, T, len(own), act=act, max_new=max(new))
+            ref = torch.cat([want[i][at[i]:at[i] + new[i]] for i in own])
+            assert rel_err(out, ref) < (2e-6 if odt == torch.float32 else 6e-3), (new, act)
+            at = [a + n for a, n in zip(at, new)]
+        for i in range(3):
+            if taps > 1:
+                assert torch.equal(state[slots[i]].cpu(), rows[i].float()[-(taps - 1):] if lens[i] >= taps - 1 else torch.cat(
+                    [torch.zeros(taps - 1 - lens[i], C), rows[i].float()]))
 
 
 def _attention_reference(q, k, v, gate, pos, lens, scale, chunk, window, out_scale=1.0):
