@@ -965,7 +965,7 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, b_off: in
                    out: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
                    seq_of_token: torch.Tensor, a: torch.Tensor, skip: torch.Tensor, n_tokens: int, n_seqs: int, chunk: int = 0,
                    scratch: Optional[torch.Tensor] = None, max_new: int = 0) -> None:
-    """dt = softplus(xdt); S[c, n] <- exp(dt a[c, n]) S[c, n] + dt x_c B_n; out_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c)
+    """h = softplus(xdt); S_cj becomes e^(h a_cj) S_cj + h x_c B_j; out_c = (sum_j S_cj C_j + skip_c x_c) silu(z_c)
     per channel, from and into state [slots, inner, N] (float32).  x, z [T, inner] and B, C (columns b_off and c_off of bc)
     in the dtype of out, xdt [T, inner] float32 (all may be column ranges of wider rows); a [inner, N], skip [inner]
     float32.  chunk > 0: in chunks of that many rows (prompts).  max_new: the most tokens one sequence brings, where the

@@ -1,7 +1,7 @@
 // The selective scan: a diagonal state per channel, its decay and its input made from the token.
 //
 //     dt = softplus(xdt_c)                                                  xdt: a projection with its bias, float32
-//     S[c, n] <- exp(dt A[c, n]) S[c, n] + dt x_c B_n,   y_c = sum_n S[c, n] C_n + D_c x_c,   out_c = y_c silu(z_c)
+//     S_cj becomes e^(dt a_cj) S_cj + dt x_c B_j,     out_c = (sum_j S_cj C_j + D_c x_c) silu(z_c)
 //
 // S [inner][N] (float32, zero at a sequence's start) lives in the cache's per-slot state.  x, z, B and C come in the
 // compute dtype (columns of wider rows), xdt in float32; everything from there to the store is float32.

@@ -14,9 +14,8 @@
 `mamba1` (a selective scan: a diagonal state per channel, its decay, input and read-out made from the token; state: a
 matrix [inner, state]):
     W_in h = [x: inner | z: inner],  x <- silu(conv(x));   W_x x = [r: dt_rank | B: state | C: state]
-    dt = softplus(W_dt r + b_dt),  A = -exp(A_log) [inner, state]
-    S_t[c, n] = exp(dt_c A[c, n]) S_(t-1)[c, n] + dt_c x_c B_n,   y_c = sum_n S_t[c, n] C_n + D_c x_c
-    out = W_o (y * silu(z))
+    h = softplus(W_dt r + b_dt),  a = -e^A_log [inner, state]
+    S_t,cj = e^(h_c a_cj) S_(t-1),cj + h_c x_c B_j,   y_c = sum_j S_t,cj C_j + D_c x_c,   out = W_o (y * silu(z))
 
 conv(v)_t = bias + sum_j c[:, j] v_(t - taps + 1 + j) inside a sequence (the last tap meets the token itself, zeros
 before the start).  What a layer keeps per sequence is the convolution's last taps - 1 inputs and S (two

@@ -76,10 +76,10 @@ class RotaryYarn(RotaryNeoX):
 
 @register_position("rope_banded")
 class RotaryBanded(RotaryNeoX):
-    """NeoX pairing with frequencies scaled by bands of wavelength, for contexts beyond the trained length: with l = 2 pi /
-    f_i the positions a pair needs for one turn, pairs with l < original / high keep f_i, pairs with l > original / low are
-    slowed to f_i / factor, and between the two s = (original / l - low) / (high - low) mixes them, (1 - s) f_i / factor +
-    s f_i.  Parameters: theta, rotary_dim, factor, low, high, original."""
+    """NeoX pairing with frequencies scaled by bands of wavelength, for contexts beyond the trained length: with n_i
+    the turns that pair i makes in `original` positions, pairs of more than `high` turns keep their frequency, pairs of fewer
+    than `low` are slowed by `factor`, and the others take a mean of the two, weighted by how far n_i lies from low to
+    high.  Parameters: theta, rotary_dim, factor, low, high, original."""
 
     def __init__(self, params: Dict[str, Any], rt: Runtime):
         super().__init__(params, rt)
@@ -88,7 +88,7 @@ class RotaryBanded(RotaryNeoX):
             raise ValueError("rope_banded: factor, low, high and original must be positive")
         scaled = []
         for f in self.inv_freq.tolist():
-            turns = original * f / (2.0 * math.pi)          # original / l
+            turns = original * f / (2.0 * math.pi)
             if turns > high:
                 scaled.append(f)
             elif turns < low:

@@ -3,7 +3,8 @@
 Spec parameters: `members`, a list of dicts with `kind` (a registered mixer kind), `params` (that mixer's own
 parameters), `prefix` (added to the part's prefix for the member's tensors), `weight` (the factor on the
 member's output, default 1) and `out_norm` {tensor, size, eps} (optional: the member's output is divided by its root mean
-square over the row and multiplied by that stored vector, named under the member's prefix, before it is added).  Each member keeps a cache or state of its own: the part's cache request is the tuple
+square over the row and multiplied by that stored vector, named under the member's prefix, before it is added).  Each
+member keeps a cache or state of its own: the part's cache request is the tuple
 of its members' requests and it is handed the tuple of their views.  A member that takes its factor into its own
 last step (`scale_output(w) -> bool`) adds straight into the output; any other member writes into a zeroed buffer
 that is added with its factor.  Members with a norm write into buffers side by side, zeroed unless the member says

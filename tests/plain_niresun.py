@@ -74,14 +74,14 @@ def frequencies(rot: dict) -> torch.Tensor:
     factor, low, high, original = (float(sc[k]) for k in ("factor", "low", "high", "original"))
     out = []
     for v in f.tolist():
-        wavelength = 2.0 * math.pi / v
-        if wavelength < original / high:
+        turns = original * v / (2.0 * math.pi)               # in `original` positions
+        if turns > high:
             out.append(v)
-        elif wavelength > original / low:
+        elif turns < low:
             out.append(v / factor)
         else:
-            s = (original / wavelength - low) / (high - low)
-            out.append((1.0 - s) * v / factor + s * v)
+            s = (turns - low) / (high - low) if high != low else 1.0
+            out.append(v / factor + s * (v - v / factor))
     return torch.tensor(out, dtype=torch.float64)
 
 

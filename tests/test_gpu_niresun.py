@@ -274,7 +274,7 @@ def _attention_reference(q, k, v, gate, pos, lens, scale, chunk, window, out_sca
 
 
 @pytest.mark.parametrize("H,G,d,dv,chunk,window,gated", [
-    (6, 2, 72, 48, 100, 0, True), (4, 1, 128, 128, 70, 0, True), (8, 2, 64, 64, 0, 0, False), (8, 1, 64, 80, 96, 0, True),
+    (6, 2, 72, 48, 100, 0, True), (4, 1, 128, 128, 70, 0, True), (8, 2, 64, 64, 0, 0, False), (7, 1, 64, 88, 90, 0, True),
     (4, 4, 40, 128, 64, 0, False), (3, 3, 8, 8, 1, 0, True), (16, 1, 96, 104, 33, 50, True), (2, 1, 120, 24, 1000, 0, True),
     (6, 2, 12, 20, 37, 0, True), (5, 1, 14, 26, 50, 0, False), (20, 1, 64, 64, 90, 0, True)])
 def test_attention_of_other_sizes_in_chunks_behind_a_gate(H, G, d, dv, chunk, window, gated):
